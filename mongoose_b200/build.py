@@ -5,10 +5,11 @@ The counterpart of the reference's kernel provisioning
 host side opens with dlopen.  Unlike the reference it never probes the GPU for
 an architecture (the target is fixed) and never installs a toolkit.
 
-    python -m mongoose_b200.build [--force] [--verbose]
+    python -m mongoose_b200.build [--force] [--verbose] [--family=layered]
 """
 from __future__ import annotations
 
+import glob
 import os
 import shutil
 import subprocess
@@ -20,8 +21,16 @@ CSRC = os.path.join(HERE, "csrc")
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 LIB_NAME = "libmongoose_kernels.so"
 LIB_PATH = os.path.join(HERE, LIB_NAME)
-SOURCES = ["legacy_ops.cu", "block_ops.cu", "engine.cu"]
-HEADERS = ["mg_common.cuh", "decode_kernels.cuh", "mega_kernel.cuh"]
+# translation unit -> what it serves: "abi" the reference's C symbols, "core" the engine's host code,
+# "dense" the fixed seven-matrix decode block, "layered" models described layer by layer
+UNITS = {
+    "engine.cu": "core",
+    "legacy_ops.cu": "abi", "block_ops.cu": "abi",
+    "dense_phases.cu": "dense", "mega_single.cu": "dense", "mega_tp.cu": "dense",
+}
+# A family of models can be served by a library of its own, compiled from what that family needs (the
+# persistent kernel of the dense family alone takes two minutes); the whole library serves every family.
+FAMILIES = {"layered": ("core", "layered")}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -46,15 +55,38 @@ def _stale(target: str, deps: list[str]) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
+def family_lib(family: str) -> str:
+    """Path of the library that serves one family only."""
+    return os.path.join(HERE, f"libmongoose_{family}.so")
+
+
+def headers() -> list[str]:
+    return sorted(glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h")) +
+                  [os.path.join(INCLUDE, "mongoose_kernels.h"), os.path.abspath(__file__)])
+
+
+def fresh(lib: str) -> bool:
+    """Is `lib` newer than every source it may have been built from?"""
+    return not _stale(lib, [os.path.join(CSRC, u) for u in UNITS] + headers())
+
+
+def ensure(family: str) -> str:
+    """A library that serves `family`: the whole one where it is up to date, else the family's own,
+    compiled if need be."""
+    return LIB_PATH if fresh(LIB_PATH) else build(family=family)
+
+
+def build(force: bool = False, verbose: bool = False, family: str | None = None) -> str:
     nvcc = _nvcc()
     objdir = os.path.join(HERE, "build")
     os.makedirs(objdir, exist_ok=True)
-    common = [os.path.join(CSRC, h) for h in HEADERS] + [os.path.join(INCLUDE, "mongoose_kernels.h"),
-                                                         os.path.abspath(__file__)]
+    common = headers()
+    parts = FAMILIES[family] if family else None
+    sources = [u for u, part in UNITS.items() if parts is None or part in parts]
+    lib_path = family_lib(family) if family else LIB_PATH
     jobs = []
     objs = []
-    for src in SOURCES:
+    for src in sources:
         s = os.path.join(CSRC, src)
         o = os.path.join(objdir, src.replace(".cu", ".o"))
         objs.append(o)
@@ -73,18 +105,21 @@ def build(force: bool = False, verbose: bool = False) -> str:
         if verbose:
             sys.stderr.write(r.stderr)
 
-    with ThreadPoolExecutor(max_workers=len(SOURCES)) as ex:
+    with ThreadPoolExecutor(max_workers=len(sources)) as ex:
         list(ex.map(compile_one, jobs))
 
-    if force or jobs or _stale(LIB_PATH, objs):
-        cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", LIB_PATH, *objs,
+    if force or jobs or _stale(lib_path, objs):
+        part = f"{lib_path}.{os.getpid()}"
+        cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", part, *objs,
                "-Xcompiler", "-fPIC", "-cudart", "static"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-    return LIB_PATH
+        os.replace(part, lib_path)
+    return lib_path
 
 
 if __name__ == "__main__":
-    p = build(force="--force" in sys.argv, verbose="--verbose" in sys.argv)
+    p = build(force="--force" in sys.argv, verbose="--verbose" in sys.argv,
+              family=next((a.split("=", 1)[1] for a in sys.argv if a.startswith("--family=")), None))
     print(p)

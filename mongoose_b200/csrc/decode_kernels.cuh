@@ -95,7 +95,7 @@ __device__ __forceinline__ long long xchg_deadline(const XchgStatus* st) {
     return ld_l2_u32(reinterpret_cast<const unsigned int*>(&st->error)) ? 0ll : clock64() + 2000000000ll;
 }
 
-__device__ __noinline__ void xchg_timeout(const GatherArgs& g, int sender, unsigned int want, unsigned int seen) {
+static __device__ __noinline__ void xchg_timeout(const GatherArgs& g, int sender, unsigned int want, unsigned int seen) {
     if (atomicCAS(&g.status->error, 0, 1) == 0) {
         g.status->slot = g.slot; g.status->sender = sender; g.status->want = want; g.status->seen = seen;
     }
@@ -620,7 +620,7 @@ __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
 
 // Sum of the received rows into a plain vector (the hidden state a layer range hands back to the
 // host when no kernel of the same step consumes it).
-__global__ void __launch_bounds__(256) xchg_reduce_kernel(const GatherArgs g, float* out, int K) {
+static __global__ void __launch_bounds__(256) xchg_reduce_kernel(const GatherArgs g, float* out, int K) {
     pdl_wait();
     const unsigned int want = ld_l2_u32(g.count);
     const long long deadline = xchg_deadline(g.status);
@@ -629,7 +629,7 @@ __global__ void __launch_bounds__(256) xchg_reduce_kernel(const GatherArgs g, fl
 }
 
 // Cursor update after the running argmax has been combined over tensor-parallel ranks.
-__global__ void finalize_step_kernel(StepState* s, int* out_tokens) {
+static __global__ void finalize_step_kernel(StepState* s, int* out_tokens) {
     pdl_wait();
     const unsigned long long key = s->best;
     const int tok = (int)(0xffffffffu - (unsigned int)(key & 0xffffffffull));

@@ -28,6 +28,7 @@
 
 #include "../../include/mongoose_kernels.h"
 #include "decode_kernels.cuh"
+#include "kernel_table.h"
 #include "mega_kernel.cuh"
 
 using namespace mg;
@@ -469,25 +470,10 @@ int upload_planes(mg_engine* e, int idx, int fmt, int rows, int K, const std::ve
 // ------------------------------------------------------------------
 // Kernel selection and launch
 // ------------------------------------------------------------------
-typedef void (*phase_fn_t)(const PhaseArgs);
+phase_fn_t phase_fn(int fmt, int epi, int R) { return dense_kernels()->phase(fmt, epi, R); }
 
-template <int FMT>
-phase_fn_t phase_fn_fmt(int epi, int R) {
-    switch (epi) {
-        case EPI_QKV: return phase_kernel<FMT, EPI_QKV, 2, 4>;
-        case EPI_SWIGLU: return R == 4 ? phase_kernel<FMT, EPI_SWIGLU, 4, 2> : phase_kernel<FMT, EPI_SWIGLU, 2, 4>;
-        case EPI_LOGITS: return phase_kernel<FMT, EPI_LOGITS, 4, 2>;
-        default:
-            return R == 4 ? phase_kernel<FMT, EPI_RESID, 4, 2>
-                 : R == 2 ? phase_kernel<FMT, EPI_RESID, 2, 4>
-                          : phase_kernel<FMT, EPI_RESID, 1, 8>;
-    }
-}
-
-phase_fn_t phase_fn(int fmt, int epi, int R) {
-    return fmt == FMT_Q8_0 ? phase_fn_fmt<FMT_Q8_0>(epi, R)
-         : fmt == FMT_Q4_0 ? phase_fn_fmt<FMT_Q4_0>(epi, R)
-                           : phase_fn_fmt<FMT_F16>(epi, R);
+const void* mega_fn(const mg_engine* e) {
+    return e->sh.size > 1 ? dense_kernels()->mega_tp() : dense_kernels()->mega();
 }
 
 const int kMaxDynSmem = 120 * 1024;
@@ -498,12 +484,9 @@ int set_kernel_attrs(mg_engine* e) {
             for (int R = 1; R <= 4; R *= 2)
                 MG_CUDA(e, cudaFuncSetAttribute((const void*)phase_fn(fmt, epi, R),
                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem));
-    MG_CUDA(e, cudaFuncSetAttribute((const void*)attn_decode_kernel<64>,
-                                    cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem));
-    MG_CUDA(e, cudaFuncSetAttribute((const void*)attn_decode_kernel<128>,
-                                    cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem));
-    MG_CUDA(e, cudaFuncSetAttribute((const void*)attn_decode_kernel<32>,
-                                    cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem));
+    for (int hd = 32; hd <= 128; hd *= 2)
+        MG_CUDA(e, cudaFuncSetAttribute((const void*)dense_kernels()->attn(hd),
+                                        cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem));
     return MG_OK;
 }
 
@@ -641,20 +624,9 @@ int enqueue_step(mg_engine* e, cudaStream_t s, int ls, int le, int mode, int hea
         {   // attention
             const size_t smem = ((size_t)c.head_dim + 40 + 512 + c.max_seq) * sizeof(float);
             if (smem > (size_t)kMaxDynSmem) return fail(e, MG_ERR_UNSUPPORTED, "max_seq %d too large", c.max_seq);
-            cudaError_t ce;
-            if (c.head_dim == 64)
-                ce = launch(e, s, attn_decode_kernel<64>, n_heads, 256, smem, (const float*)e->q,
-                            (const __half*)(e->kc + kvoff), (const __half*)(e->vc + kvoff), e->attn,
-                            (const StepState*)e->st, kv_dim, n_heads, n_kv);
-            else if (c.head_dim == 128)
-                ce = launch(e, s, attn_decode_kernel<128>, n_heads, 256, smem, (const float*)e->q,
-                            (const __half*)(e->kc + kvoff), (const __half*)(e->vc + kvoff), e->attn,
-                            (const StepState*)e->st, kv_dim, n_heads, n_kv);
-            else
-                ce = launch(e, s, attn_decode_kernel<32>, n_heads, 256, smem, (const float*)e->q,
-                            (const __half*)(e->kc + kvoff), (const __half*)(e->vc + kvoff), e->attn,
-                            (const StepState*)e->st, kv_dim, n_heads, n_kv);
-            MG_CUDA(e, ce);
+            MG_CUDA(e, launch(e, s, dense_kernels()->attn(c.head_dim), n_heads, 256, smem, (const float*)e->q,
+                              (const __half*)(e->kc + kvoff), (const __half*)(e->vc + kvoff), e->attn,
+                              (const StepState*)e->st, kv_dim, n_heads, n_kv));
         }
         {   // wo + residual: h2 = h + Wo attn (a partial sum over this rank's heads under tensor parallelism)
             PhaseArgs a{};
@@ -891,7 +863,7 @@ int build_mega(mg_engine* e) {
     bool ok = mega_feasible(e, &why);
     if (ok) {
         int per_sm = 0;
-        const void* kern = e->sh.size > 1 ? (const void*)mega_decode_kernel<true> : (const void*)mega_decode_kernel<false>;
+        const void* kern = mega_fn(e);
         if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->mk_smem) != cudaSuccess ||
             cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kern, MK_THREADS, e->mk_smem) != cudaSuccess ||
             per_sm < 1) {
@@ -1156,7 +1128,7 @@ int launch_mega(mg_engine* e, int ls, int le, int mode, int head, int n_steps) {
     a.trace = e->trace_next ? e->mk_trace : nullptr;
     e->trace_next = false;
     void* params[] = {&a};
-    const void* kern = e->sh.size > 1 ? (const void*)mega_decode_kernel<true> : (const void*)mega_decode_kernel<false>;
+    const void* kern = mega_fn(e);
     MG_CUDA(e, cudaLaunchCooperativeKernel(kern, dim3(e->num_sms), dim3(MK_THREADS), params,
                                            e->mk_smem, e->stream));
     e->launches += 1;
@@ -1280,6 +1252,7 @@ int mg_create(const mg_config* cfg, mg_engine** out) {
         return MG_ERR_ARG;
     if (c.layer_fmt < 0 || c.layer_fmt > 2 || c.head_fmt < 0 || c.head_fmt > 2) return MG_ERR_ARG;
     if (c.max_batch > 1) return MG_ERR_UNSUPPORTED;
+    if (!dense_kernels) return MG_ERR_UNSUPPORTED;      // a library built without this family
 
     mg_engine* e = new mg_engine();
     e->cfg = c;

@@ -390,7 +390,7 @@ struct MkCtx {
     __device__ __forceinline__ int nslot() const { return a.nslot; }
 };
 
-__device__ __noinline__ void mk_fail_impl(volatile int* abort_flag, MegaStatus* status, int code, int where, int who = -1) {
+static __device__ __noinline__ void mk_fail_impl(volatile int* abort_flag, MegaStatus* status, int code, int where, int who = -1) {
     *abort_flag = 1;
     if (atomicCAS(&status->error, 0, code) == 0) {
         status->where = where;
@@ -417,7 +417,7 @@ __device__ __forceinline__ void mk_trace(const MegaArgs& a, int step, int ev) {
 // in ONE out-of-line copy per kind of wait, so that the many places that wait add a handful of
 // instructions each to the code a phase runs through (the kernel's speed is bounded by the length
 // of the instruction stream of a phase as much as by its data).  All waits are bounded.
-__device__ __noinline__ void mk_wait_bar_slow(volatile int* abort_flag, MegaStatus* status, long long limit,
+static __device__ __noinline__ void mk_wait_bar_slow(volatile int* abort_flag, MegaStatus* status, long long limit,
                                               uint32_t bar_s, uint32_t parity, int code, int where) {
     if (*abort_flag) return;
     const long long t0 = global_ns();
@@ -443,7 +443,7 @@ __device__ __forceinline__ void mk_wait_bar(MkCtx& c, unsigned long long* bar, u
 
 // Re-read a pair of exchange words (16-byte aligned) until both carry `tag`; sys = the words may be
 // written by another GPU.  Returns the raw words: x, z = values, y, w = tags.
-__device__ __noinline__ uint4 mk_poll16_slow(volatile int* abort_flag, MegaStatus* status, long long limit,
+static __device__ __noinline__ uint4 mk_poll16_slow(volatile int* abort_flag, MegaStatus* status, long long limit,
                                              const Tagged* p, unsigned int tag, int sys, int who = -1) {
     uint4 r = make_uint4(0u, tag, 0u, tag);
     if (*abort_flag) return r;
@@ -1028,7 +1028,7 @@ __device__ __forceinline__ void red_add_s64(long long* p, long long v) {
     asm volatile("red.relaxed.gpu.global.add.u64 [%0], %1;" ::"l"(p), "l"(v) : "memory");
 }
 // Re-read a pair of accumulator words (16-byte aligned) until both have received n additions.
-__device__ __noinline__ uint4 mk_pollacc_slow(volatile int* abort_flag, MegaStatus* status, long long limit,
+static __device__ __noinline__ uint4 mk_pollacc_slow(volatile int* abort_flag, MegaStatus* status, long long limit,
                                               const Tagged* p, unsigned int n) {
     uint4 r = make_uint4(0u, 0u, 0u, 0u);
     if (*abort_flag) return r;
@@ -1063,7 +1063,7 @@ struct StageSrc {
 #endif
 
 // The first token's hidden state does not come through an exchange buffer: embedding row or plain vector.
-__device__ __noinline__ float2 mk_direct_pair(const MegaArgs& a, int kind, int token, int i) {
+static __device__ __noinline__ float2 mk_direct_pair(const MegaArgs& a, int kind, int token, int i) {
     if (kind == SRC_EMBED)
         return make_float2(embed_value(a.embed_w, a.head_fmt, a.dim, token, i), embed_value(a.embed_w, a.head_fmt, a.dim, token, i + 1));
     return make_float2(a.h_in[i], a.h_in[i + 1]);
