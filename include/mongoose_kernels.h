@@ -160,7 +160,7 @@ enum {
 };
 
 /* Weight storage formats. */
-enum { MG_FMT_Q8_0 = 0, MG_FMT_Q4_0 = 1, MG_FMT_F16 = 2 };
+enum { MG_FMT_Q8_0 = 0, MG_FMT_Q4_0 = 1, MG_FMT_F16 = 2, MG_FMT_BF16 = 3 /* layer-described models */ };
 
 /* Model description: the positional arguments of NewCUDAFusedInference
  * (cuda_fused_infer.go:144) plus what the reference hard-codes. */
@@ -315,6 +315,64 @@ MG_API int mg_wait_mailbox(mg_engine* e, int timeout_ms);
 MG_API int mg_queue_hidden_to_l3(mg_engine* e);
 MG_API int mg_wait_l3(mg_engine* e, int timeout_ms);
 MG_API const float* mg_l3_hidden(mg_engine* e);
+
+/* ---- models described layer by layer ----------------------------------------------------------------
+ * mg_create builds the reference's one block (the seven matrices of every layer alike).  The calls below
+ * build a decoder whose layers are listed one by one, each with its mixer and feed-forward sizes; the
+ * engine they return takes the same stepping calls (mg_step_token, mg_generate, mg_enqueue_greedy,
+ * mg_partial_step, mg_graph_launch, ...) and keeps its sequence state - cached keys and recurrent state -
+ * in the same arena.  Portions of a prompt go through mg_forward.  No counterpart in the reference.
+ *
+ * A layer: x += norm(mixer(x)); x += norm(ff(x)), norms with their weights stored around zero.  The mixer
+ * MG_MIXER_PARALLEL runs two branches on the same input and takes half the sum of their normed outputs:
+ *   attention - grouped query heads, per-head query and key norms, query temperature
+ *     1 + temp_coef * ln(floor((p + 1) / temp_every) + 1), score * scale minus slope_h * distance with
+ *     slope_h = 2^(-8 (h + 1) / heads), weights sigmoid(score + bias_h) not normalised over keys and mixed
+ *     over heads by a matrix, values = raw keys;
+ *   matrix memory - per head a [dim][vdim] state with exponential gates (caps gate_cap), 32-bit. */
+enum { MG_MATH_BF16 = 0,      /* matrix products and activations of prompts in bf16, fp32 accumulation */
+       MG_MATH_F32 = 1 };     /* everything in 32-bit */
+enum { MG_MIXER_PARALLEL = 0 };
+typedef struct mg_gate_attn_config {
+    int heads, kv_heads, dim;
+    float scale, temp_coef;
+    int temp_every;
+} mg_gate_attn_config;
+typedef struct mg_mat_mem_config {
+    int heads, dim, vdim;
+    float gate_cap;
+} mg_mat_mem_config;
+typedef struct mg_layer_config {
+    int mixer;                /* MG_MIXER_* */
+    mg_gate_attn_config attn;
+    mg_mat_mem_config mem;
+    int ffn_dim;              /* inner width of the gelu feed-forward; 0 = the layer has none */
+} mg_layer_config;
+typedef struct mg_model_config {
+    int width, vocab, n_layers, max_seq;
+    float norm_eps;
+    int math;                 /* MG_MATH_* */
+    int device;
+} mg_model_config;
+/* Weight slots of a layer-described model: index layer * MG_LAYER_SLOTS + slot; after the layers
+ * n_layers * MG_LAYER_SLOTS + {0 embedding, 1 final norm (around zero), 2 output head}.  Matrices are
+ * [out][in]; mg_set_weight takes fp32 (stored as bf16), mg_set_weight_raw takes bf16 for any slot. */
+enum {
+    MG_SLOT_NORM1 = 0, MG_SLOT_NORM2 = 1,
+    MG_SLOT_AT_Q = 2, MG_SLOT_AT_K = 3, MG_SLOT_AT_QNORM = 4, MG_SLOT_AT_KNORM = 5, MG_SLOT_AT_TALK = 6, MG_SLOT_AT_BIAS = 7,
+    MG_SLOT_AT_O = 8, MG_SLOT_AT_OUT = 9,
+    MG_SLOT_MEM_Q = 10, MG_SLOT_MEM_K = 11, MG_SLOT_MEM_V = 12, MG_SLOT_MEM_G = 13, MG_SLOT_MEM_O = 14, MG_SLOT_MEM_NORM = 15,
+    MG_SLOT_MEM_I = 16, MG_SLOT_MEM_IB = 17, MG_SLOT_MEM_F = 18, MG_SLOT_MEM_FB = 19, MG_SLOT_MEM_OUT = 20,
+    MG_SLOT_UP = 21, MG_SLOT_DOWN = 22,
+    MG_LAYER_SLOTS = 32
+};
+MG_API int mg_create_layered(const mg_model_config* cfg, const mg_layer_config* layers, mg_engine** out);
+/* n tokens at positions pos .. pos + n - 1 of the engine's sequence, from the cache and state that
+ * earlier calls left: pos is 0 (a new sequence; nothing of the old one is read) or the number of tokens
+ * seen so far.  logits_out (HOST, [n_want][vocab]) receives the logits after the tokens want[0..n_want)
+ * (ascending places among the n).  One token takes the decode path, more the prompt path; an engine
+ * made by mg_create feeds them one by one, as its mg_generate does. */
+MG_API int mg_forward(mg_engine* e, const int* tokens, int n, int pos, const int* want, int n_want, float* logits_out);
 
 /* ---- tensor-parallel decode over 2/4/8 GPUs of one node, one process per GPU ----------------------
  * The reference has no tensor parallelism (multigpu.go:32-82, 496-623 manages per-device handles and

@@ -30,6 +30,26 @@ class MgTpShard(C.Structure):
                 ("ffn0", ci), ("ffn1", ci), ("vocab0", ci), ("vocab1", ci)]
 
 
+class MgGateAttnConfig(C.Structure):
+    """struct mg_gate_attn_config of include/mongoose_kernels.h."""
+    _fields_ = [("heads", ci), ("kv_heads", ci), ("dim", ci), ("scale", cf), ("temp_coef", cf), ("temp_every", ci)]
+
+
+class MgMatMemConfig(C.Structure):
+    """struct mg_mat_mem_config of include/mongoose_kernels.h."""
+    _fields_ = [("heads", ci), ("dim", ci), ("vdim", ci), ("gate_cap", cf)]
+
+
+class MgLayerConfig(C.Structure):
+    """struct mg_layer_config of include/mongoose_kernels.h."""
+    _fields_ = [("mixer", ci), ("attn", MgGateAttnConfig), ("mem", MgMatMemConfig), ("ffn_dim", ci)]
+
+
+class MgModelConfig(C.Structure):
+    """struct mg_model_config of include/mongoose_kernels.h."""
+    _fields_ = [("width", ci), ("vocab", ci), ("n_layers", ci), ("max_seq", ci), ("norm_eps", cf), ("math", ci), ("device", ci)]
+
+
 # name -> (restype, argtypes): every symbol include/mongoose_kernels.h declares.
 SIGNATURES = {
     # reference ABI (stream is the last argument everywhere)
@@ -63,6 +83,8 @@ SIGNATURES = {
     "mongoose_partial_step_q4_fused_graph": (None, [vp] * 25 + [ci] * 10 + [vp]),
     # engine
     "mg_create": (ci, [C.POINTER(MgConfig), C.POINTER(vp)]),
+    "mg_create_layered": (ci, [C.POINTER(MgModelConfig), C.POINTER(MgLayerConfig), C.POINTER(vp)]),
+    "mg_forward": (ci, [vp, vp, ci, ci, vp, ci, vp]),
     "mg_destroy": (None, [vp]),
     "mg_num_weights": (ci, [vp]),
     "mg_set_weight": (ci, [vp, ci, vp, sz]),
@@ -120,28 +142,52 @@ SIGNATURES = {
 _lib = None
 
 
-def load(path: str | None = None) -> C.CDLL:
+def load(path: str | None = None, family: str | None = None) -> C.CDLL:
     """Open the library and bind every declared symbol.  Raises with the
-    reason when the file is absent or a symbol is missing."""
+    reason when the file is absent or a symbol is missing.  With `family`, the
+    library that serves only that family of models (build.py) does where the
+    whole one has not been built; it holds the engine, not the mongoose_* symbols."""
     global _lib
     if _lib is not None and path is None:
         return _lib
     p = path or LIB_PATH
+    partial = False
+    if path is None and family and not os.path.exists(p):
+        p = os.path.join(_HERE, f"libmongoose_{family}.so")
+        partial = True
+    lib = _open(p, partial)
+    if path is None and not partial:
+        _lib = lib
+    return lib
+
+
+def provision(family: str) -> C.CDLL:
+    """Compile what `family` needs, unless an up-to-date library is there, and open it
+    (the counterpart of the reference's kernel provisioning, kernel_provision.go:28-88)."""
+    global _lib
+    from . import build
+    p = build.ensure(family)
+    if p == LIB_PATH:
+        return load()
+    _lib = _open(p, True)
+    return _lib
+
+
+def _open(p: str, partial: bool) -> C.CDLL:
     if not os.path.exists(p):
         raise RuntimeError(
             f"{p} not found: build it with `python -m mongoose_b200.build` "
             "(there is no CPU or PyTorch fallback for this path)")
-    lib = C.CDLL(p, mode=C.RTLD_GLOBAL)
+    lib = C.CDLL(p, mode=C.RTLD_LOCAL if partial else C.RTLD_GLOBAL)
     missing = []
     for name, (res, args) in SIGNATURES.items():
         try:
             fn = getattr(lib, name)
         except AttributeError:
-            missing.append(name)
+            if not (partial and name.startswith("mongoose_")):
+                missing.append(name)
             continue
         fn.restype, fn.argtypes = res, args
     if missing:
         raise RuntimeError(f"{p} does not export: {', '.join(missing)}")
-    if path is None:
-        _lib = lib
     return lib

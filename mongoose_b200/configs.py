@@ -13,6 +13,7 @@ from dataclasses import dataclass, replace
 FMT_Q8_0 = 0
 FMT_Q4_0 = 1
 FMT_F16 = 2
+FMT_BF16 = 3    # layer-described models (layered.py)
 
 # slots of the reference's weight index scheme, idx = layer*12 + slot
 # (cuda_fused_infer.go:241-272)

@@ -34,8 +34,13 @@ struct StepState {
     unsigned int pad;
 };
 
-enum : int { PRO_PLAIN = 0, PRO_RMS = 1, PRO_RMS_EMBED = 2 };
-enum : int { EPI_QKV = 0, EPI_RESID = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3 };
+enum : int { PRO_PLAIN = 0, PRO_RMS = 1, PRO_RMS_EMBED = 2,
+             // layer-described models (stage_layered): the residual sum is formed where it is next read
+             PRO_X = 3,            // x as it is
+             PRO_EMBED_POS = 4,    // embedding row + position vector
+             PRO_POST = 5,         // x + norm(z)
+             PRO_POST_PAIR = 6 };  // x + norm(half the sum of two normed vectors)
+enum : int { EPI_QKV = 0, EPI_RESID = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_STORE = 4, EPI_GELU = 5 };
 
 // ---------------------------------------------------------------------
 // Tensor-parallel exchange fused into the phase kernels.  A rank's wo / down kernel writes its
@@ -146,8 +151,17 @@ struct PhaseArgs {
     int row_base;         // LOGITS: global index of local row 0 (vocab-sharded lm_head)
     int defer_finalize;   // LOGITS: leave the cursor update to finalize_step_kernel (argmax still to be reduced over ranks)
     PushArgs push;        // RESID: send the output rows to every rank instead of (or besides) `out`
+    // layer-described models: K is the padded row length of the matrix, k_valid the vector's own length
+    int k_valid;
+    const float* pos_tab; // EMBED_POS: [max_seq][k_valid]
+    const float* z[2];    // POST: the sublayer's output; POST_PAIR: its two branches
+    const float* z_w[2];  // POST_PAIR: plain norm weights of the branches
+    const float* post_w;  // weight of the norm on the sublayer's output, stored around zero
+    const float* last_w;  // not NULL: a norm (weight around zero) of the sum follows (the model's last)
     GatherArgs gather;    // RMS prologue: the hidden state is the sum of the received rows; CTA 0 keeps it in h_store
 };
+
+typedef void (*phase_fn_t)(const PhaseArgs);
 
 __device__ __forceinline__ unsigned long long pack_best(float v, unsigned int idx) {
     unsigned int u = __float_as_uint(v);
@@ -169,9 +183,68 @@ __device__ __forceinline__ float embed_value(const WeightView& e, int fmt, int K
         const int nib = j < 16 ? (byte & 0xF) : (byte >> 4);
         const float d = half_bits_to_float(e.ds[(size_t)token * (K / 32) + b]);
         return d * (float)(nib - 8);
+    } else if (fmt == FMT_BF16) {
+        return __uint_as_float((uint32_t)reinterpret_cast<const unsigned short*>(e.qs)[(size_t)token * K + i] << 16);
     } else {
         return half_bits_to_float(reinterpret_cast<const unsigned short*>(e.qs)[(size_t)token * K + i]);
     }
+}
+
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+// Prologue of layer-described models.  xs gets K floats, zero from k_valid on; with `keep` the residual
+// sum goes to h_store (never the buffer x_src names: other CTAs still read that one).
+__device__ __forceinline__ void stage_layered(const PhaseArgs& a, float* xs, float* red, bool keep) {
+    const int K = a.K, n = a.k_valid, nt = blockDim.x;
+    const float inv_n = 1.0f / (float)n;
+    for (int i = n + threadIdx.x; i < K; i += nt) xs[i] = 0.f;
+    if (a.pro == PRO_X || a.pro == PRO_EMBED_POS) {
+        const int token = a.pro == PRO_EMBED_POS ? a.st->token : 0, pos = a.pro == PRO_EMBED_POS ? a.st->pos : 0;
+        for (int i = threadIdx.x; i < n; i += nt) {
+            const float v = a.pro == PRO_X ? a.x_src[i]
+                                           : embed_value(a.embed, a.embed_fmt, K, token, i) + a.pos_tab[(size_t)pos * n + i];
+            xs[i] = v;
+            if (keep) a.h_store[i] = v;
+        }
+    } else {
+        float ss = 0.f;
+        if (a.pro == PRO_POST) {
+            for (int i = threadIdx.x; i < n; i += nt) {
+                const float v = a.z[0][i];
+                xs[i] = v;
+                ss = fmaf(v, v, ss);
+            }
+        } else {
+            float s0 = 0.f, s1 = 0.f;
+            for (int i = threadIdx.x; i < n; i += nt) {
+                const float u = a.z[0][i], v = a.z[1][i];
+                s0 = fmaf(u, u, s0);
+                s1 = fmaf(v, v, s1);
+            }
+            const float r0 = 0.5f / sqrtf(block_sum(s0, red) * inv_n + a.eps);
+            const float r1 = 0.5f / sqrtf(block_sum(s1, red) * inv_n + a.eps);
+            for (int i = threadIdx.x; i < n; i += nt) {
+                const float v = a.z[0][i] * r0 * a.z_w[0][i] + a.z[1][i] * r1 * a.z_w[1][i];
+                xs[i] = v;
+                ss = fmaf(v, v, ss);
+            }
+        }
+        const float r = 1.0f / sqrtf(block_sum(ss, red) * inv_n + a.eps);
+        for (int i = threadIdx.x; i < n; i += nt) {
+            const float v = a.x_src[i] + xs[i] * r * (1.0f + a.post_w[i]);
+            xs[i] = v;
+            if (keep) a.h_store[i] = v;
+        }
+    }
+    if (a.last_w) {
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < n; i += nt) ss = fmaf(xs[i], xs[i], ss);
+        const float r = 1.0f / sqrtf(block_sum(ss, red) * inv_n + a.eps);
+        for (int i = threadIdx.x; i < n; i += nt) xs[i] = xs[i] * r * (1.0f + a.last_w[i]);
+    }
+    __syncthreads();
 }
 
 __device__ __forceinline__ void stage_x(const PhaseArgs& a, float* xs, float* red) {
@@ -385,7 +458,7 @@ __device__ __forceinline__ void load_stage(const Tile<EPI, R>& t, int c, bool va
 // Dynamic shared memory: K floats (x) + 40 floats (reductions).
 // ---------------------------------------------------------------------
 template <int FMT, int EPI, int R, int D>
-__global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
+__device__ __forceinline__ void phase_body(const PhaseArgs& a, const int bid, const int nblocks) {
     using C = Chunk<FMT>;
     extern __shared__ __align__(16) float smem[];
     float* xs = smem;
@@ -393,8 +466,8 @@ __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
 
     const int lane = threadIdx.x & 31;
     const int wpc = blockDim.x >> 5;
-    const int gw = blockIdx.x * wpc + (threadIdx.x >> 5);   // global warp index
-    const int nwarps = gridDim.x * wpc;
+    const int gw = bid * wpc + (threadIdx.x >> 5);   // global warp index
+    const int nwarps = nblocks * wpc;
     const int nchunks = a.K / C::kWeights;
     const int steps = (nchunks + 31) >> 5;
     const int my_items = gw < a.nitems ? (a.nitems - gw + nwarps - 1) / nwarps : 0;
@@ -421,9 +494,10 @@ __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
     pdl_launch_dependents();
     pdl_wait();
 
-    constexpr bool kInt = (FMT != FMT_F16);          // int8 / 4-bit weights: integer dot products
+    constexpr bool kInt = (FMT != FMT_F16 && FMT != FMT_BF16);          // int8 / 4-bit weights: integer dot products
     float rms = 1.0f;
     if (kInt) rms = stage_xq(a, reinterpret_cast<uint8_t*>(smem), red, FMT == FMT_Q4_0);
+    else if (FMT == FMT_BF16) stage_layered(a, xs, red, bid == 0 && a.h_store != nullptr);
     else stage_x(a, xs, red);
     const uint8_t* P0 = reinterpret_cast<const uint8_t*>(smem);
     const uint8_t* P1 = P0 + a.K;
@@ -551,6 +625,14 @@ __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
                                 }
                             }
                         }
+                    } else if (EPI == EPI_STORE || EPI == EPI_GELU) {
+                        if (lane == 0) {
+#pragma unroll
+                            for (int r = 0; r < R; r++) {
+                                const int row = it * R + r;
+                                if (row < a.rows[0]) a.out[row] = EPI == EPI_GELU ? gelu_tanh(acc[r]) : acc[r];
+                            }
+                        }
                     } else {  // EPI_LOGITS
                         if (lane == 0) {
 #pragma unroll
@@ -580,7 +662,7 @@ __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
             __syncthreads();
             if (threadIdx.x == 0) {
                 const unsigned int ticket = atomicAdd(a.push.ticket, 1u);
-                if (ticket == gridDim.x - 1) {
+                if (ticket == nblocks - 1) {
                     *a.push.ticket = 0u;
                     *a.push.count = ld_l2_u32(a.push.count) + 1u;
                 }
@@ -601,9 +683,9 @@ __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
             if (b) atomicMax(&s->best, b);
             __threadfence();
             const unsigned int ticket = atomicAdd(&s->done, 1u);
-            if (ticket == gridDim.x - 1 && a.defer_finalize) {
+            if (ticket == (unsigned)nblocks - 1 && a.defer_finalize) {
                 s->done = 0u;
-            } else if (ticket == gridDim.x - 1) {
+            } else if (ticket == (unsigned)nblocks - 1) {
                 __threadfence();
                 const unsigned long long key = atomicMax(&s->best, 0ull);
                 const int tok = (int)(0xffffffffu - (unsigned int)(key & 0xffffffffull));
@@ -616,6 +698,18 @@ __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
             }
         }
     }
+}
+
+template <int FMT, int EPI, int R, int D>
+__global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
+    phase_body<FMT, EPI, R, D>(a, blockIdx.x, gridDim.x);
+}
+
+// Two independent matrices in one launch: the first `split` CTAs multiply a's, the others b's.
+template <int FMT, int EPI, int R, int D>
+__global__ void __launch_bounds__(256) phase_pair_kernel(const PhaseArgs a, const PhaseArgs b, int split) {
+    const bool first = (int)blockIdx.x < split;
+    phase_body<FMT, EPI, R, D>(first ? a : b, first ? blockIdx.x : blockIdx.x - split, first ? split : gridDim.x - split);
 }
 
 // Sum of the received rows into a plain vector (the hidden state a layer range hands back to the

@@ -28,7 +28,9 @@
 
 #include "../../include/mongoose_kernels.h"
 #include "decode_kernels.cuh"
+#include "gemm_tc.h"
 #include "kernel_table.h"
+#include "layered.h"
 #include "mega_kernel.cuh"
 
 using namespace mg;
@@ -153,6 +155,7 @@ struct Arena {
 
 }  // namespace
 
+struct Layered;
 struct mg_engine {
     mg_config cfg{};
     int num_sms = 148;
@@ -229,6 +232,9 @@ struct mg_engine {
     uint8_t* xchg = nullptr;            // [2 slots][size][dim] tagged words, then this rank's counters
     uint8_t* xchg_peer[kMaxRanks] = {}; // rank p's buffer as seen from here (own entry = xchg)
     XchgStatus* xchg_status = nullptr;
+    // a model described layer by layer (layered_host.cuh), NULL for the one block mg_create builds
+    Layered* lm = nullptr;
+    int cursor = 0;                     // host mirror of the device-side position (layer-described models)
     std::string err;
 };
 
@@ -581,7 +587,10 @@ enum { HEAD_NONE = 0, HEAD_ARGMAX = 1, HEAD_LOGITS = 2 };
 
 // One token through layers [ls, le) (+ head).  The op order is PartialStep's
 // (cuda_fused_infer.go:414-451) with its 17 launches per layer fused into 5.
+int enqueue_layered_step(mg_engine* e, cudaStream_t s, int ls, int le, int mode, int head);
+
 int enqueue_step(mg_engine* e, cudaStream_t s, int ls, int le, int mode, int head) {
+    if (e->lm) return enqueue_layered_step(e, s, ls, le, mode, head);
     const mg_config& c = e->cfg;
     const Shard& sh = e->sh;
     const int L = c.n_layers;
@@ -700,6 +709,18 @@ int enqueue_step(mg_engine* e, cudaStream_t s, int ls, int le, int mode, int hea
     return MG_OK;
 }
 
+
+void drop_graphs(mg_engine* e) {
+    for (auto& kv : e->graphs)
+        if (kv.second.exec) cudaGraphExecDestroy(kv.second.exec);
+    e->graphs.clear();
+}
+
+}  // namespace
+
+#include "layered_host.cuh"
+
+namespace {
 
 // ------------------------------------------------------------------
 // Persistent-kernel path: tape construction and launch
@@ -1143,6 +1164,7 @@ int check_mega_status(mg_engine* e) {
     XchgStatus* hx = reinterpret_cast<XchgStatus*>(e->pin_i + e->pin_i_cap + 8);
     static_assert(sizeof(MegaStatus) <= 32 && sizeof(XchgStatus) <= 32, "status words must fit their pinned slots");
     if (e->tp_fused) MG_CUDA(e, cudaMemcpyAsync(hx, e->xchg_status, sizeof(XchgStatus), cudaMemcpyDeviceToHost, e->stream));
+    if (e->lm) MG_CUDA(e, cudaMemcpyAsync(hs, e->lm->status, 4, cudaMemcpyDeviceToHost, e->stream));
     if (e->mega_ok) MG_CUDA(e, cudaMemcpyAsync(hs, e->mk_status, sizeof(MegaStatus), cudaMemcpyDeviceToHost, e->stream));
     MG_CUDA(e, cudaStreamSynchronize(e->stream));
     if (e->tp_fused) {
@@ -1152,6 +1174,10 @@ int check_mega_status(mg_engine* e) {
             return fail(e, MG_ERR_TIMEOUT, "tensor-parallel exchange: rows of rank %d never arrived (slot %d, exchange %u, last seen %u)",
                         x.sender, x.slot, x.want, x.seen);
         }
+    }
+    if (e->lm && *reinterpret_cast<int*>(hs)) {
+        cudaMemset(e->lm->status, 0, 4);
+        return fail(e, MG_ERR_TIMEOUT, "tensor-core kernel: a wait for its own copies or products ran out");
     }
     if (!e->mega_ok) return MG_OK;
     const MegaStatus s = *hs;
@@ -1186,6 +1212,11 @@ int run_step(mg_engine* e, int ls, int le, int mode, int head) {
         if (e->sh.size > 1 && e->comm && head == HEAD_LOGITS && le >= e->cfg.n_layers)   // every rank gets every rank's slice
             MG_NCCL(e, g_nccl.AllGather(e->logits, e->logits_all, (size_t)e->sh.v_stride, ncclFloat, e->comm, e->stream));
         return MG_OK;
+    }
+    if (e->lm) {
+        // what is captured does not depend on the position; what may run does
+        if (int rc = layered_advance(e, ls, std::min(le, e->cfg.n_layers), e->cursor, 1)) return rc;
+        if (le >= e->cfg.n_layers && head != HEAD_NONE) e->cursor += 1;      // lm_head's last CTA moves the device's
     }
     if (!e->use_graph) {
         int rc = enqueue_step(e, e->stream, ls, le, mode, head);
@@ -1225,10 +1256,61 @@ int check_engine(mg_engine* e) {
     return MG_OK;
 }
 
-void drop_graphs(mg_engine* e) {
-    for (auto& kv : e->graphs)
-        if (kv.second.exec) cudaGraphExecDestroy(kv.second.exec);
-    e->graphs.clear();
+// What every engine has: the device, its streams and events.
+int create_common(mg_engine* e) {
+    const mg_config& c = e->cfg;
+    cudaError_t ce = cudaSetDevice(c.device);
+    if (ce != cudaSuccess) return MG_ERR_CUDA;
+    cudaDeviceProp prop{};
+    if (cudaGetDeviceProperties(&prop, c.device) != cudaSuccess) return MG_ERR_CUDA;
+    if (prop.major != 10) {
+        fprintf(stderr, "[mongoose-b200] device %d is sm_%d%d; this library is built for sm_100a only\n", c.device,
+                prop.major, prop.minor);
+        return MG_ERR_UNSUPPORTED;
+    }
+    e->num_sms = prop.multiProcessorCount;
+    if (cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking) != cudaSuccess) return MG_ERR_CUDA;
+
+    e->own_ls = 0; e->own_le = c.n_layers;
+    if (cudaEventCreateWithFlags(&e->sent_event, cudaEventDisableTiming) != cudaSuccess ||
+        cudaEventCreateWithFlags(&e->mail_event, cudaEventDisableTiming) != cudaSuccess ||
+        cudaEventCreateWithFlags(&e->compute_done, cudaEventDisableTiming) != cudaSuccess ||
+        cudaEventCreateWithFlags(&e->l3_done, cudaEventDisableTiming) != cudaSuccess ||
+        cudaStreamCreateWithFlags(&e->copy_stream, cudaStreamNonBlocking) != cudaSuccess ||
+        cudaMallocHost((void**)&e->l3, (size_t)c.dim * sizeof(float)) != cudaSuccess)
+        return MG_ERR_CUDA;
+    e->out_cap = c.max_seq > 4096 ? c.max_seq : 4096;
+    return MG_OK;
+}
+
+// The device-side cursor, the generated tokens and their pinned mirror.
+int create_cursor(mg_engine* e) {
+    int rc;
+    if ((rc = dev_alloc(e, &e->st, (size_t)1))) return rc;
+    if ((rc = dev_alloc(e, &e->out_tokens, (size_t)e->out_cap))) return rc;
+    if (cudaMemset(e->out_tokens, 0, (size_t)e->out_cap * 4) != cudaSuccess) return MG_ERR_CUDA;
+    StepState s0{};
+    s0.out_cap = e->out_cap;
+    if (cudaMemcpy(e->st, &s0, sizeof s0, cudaMemcpyHostToDevice) != cudaSuccess) return MG_ERR_CUDA;
+
+    e->pin_i_cap = 8 + e->out_cap;
+    if (cudaMallocHost((void**)&e->pin_i, (size_t)(e->pin_i_cap + 16) * sizeof(int)) != cudaSuccess) return MG_ERR_NOMEM;
+    return MG_OK;
+}
+
+void read_env(mg_engine* e) {
+    { const char* zc = getenv("MG_ZERO_COPY"); e->zero_copy = !(zc && zc[0] == '0'); }
+    const char* env = getenv("MG_NO_GRAPH");
+    if (env && env[0] == '1') e->use_graph = false;
+    env = getenv("MG_NO_MEGA");
+    if (env && env[0] == '1') e->use_mega = false;
+    env = getenv("MG_NO_PDL");
+    if (env && env[0] == '1') e->use_pdl = false;
+    // L2 prefetch distance of the persistent kernel's weight stream; 64 KiB measured best on
+    // 7B-class widths (layer time 85 -> 75 us), neutral on the 0.5 B model, 384 KiB thrashes L2
+    env = getenv("MG_PREFETCH_KB");
+    e->mk_prefetch = (env ? atoi(env) : 64) * 1024;
+    if (e->mk_prefetch < 0 || e->mk_prefetch > (1 << 20)) e->mk_prefetch = 0;
 }
 
 }  // namespace
@@ -1261,35 +1343,15 @@ int mg_create(const mg_config* cfg, mg_engine** out) {
     int rc = MG_OK;
     auto bail = [&](int code) { mg_destroy(e); return code; };
 
-    cudaError_t ce = cudaSetDevice(c.device);
-    if (ce != cudaSuccess) return bail(MG_ERR_CUDA);
-    cudaDeviceProp prop{};
-    if (cudaGetDeviceProperties(&prop, c.device) != cudaSuccess) return bail(MG_ERR_CUDA);
-    if (prop.major != 10) {
-        fprintf(stderr, "[mongoose-b200] device %d is sm_%d%d; this library is built for sm_100a only\n", c.device,
-                prop.major, prop.minor);
-        return bail(MG_ERR_UNSUPPORTED);
-    }
-    e->num_sms = prop.multiProcessorCount;
-    if (cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking) != cudaSuccess) return bail(MG_ERR_CUDA);
-
     {
         std::string why;
         if (!make_shard(c, 0, 1, &e->sh, &why)) return bail(MG_ERR_ARG);
     }
-    e->own_ls = 0; e->own_le = c.n_layers;
-    if (cudaEventCreateWithFlags(&e->sent_event, cudaEventDisableTiming) != cudaSuccess ||
-        cudaEventCreateWithFlags(&e->mail_event, cudaEventDisableTiming) != cudaSuccess ||
-        cudaEventCreateWithFlags(&e->compute_done, cudaEventDisableTiming) != cudaSuccess ||
-        cudaEventCreateWithFlags(&e->l3_done, cudaEventDisableTiming) != cudaSuccess ||
-        cudaStreamCreateWithFlags(&e->copy_stream, cudaStreamNonBlocking) != cudaSuccess ||
-        cudaMallocHost((void**)&e->l3, (size_t)c.dim * sizeof(float)) != cudaSuccess)
-        return bail(MG_ERR_CUDA);
+    if ((rc = create_common(e))) return bail(rc);
     const int nw = c.n_layers * 12 + 2;
     e->mats.resize(nw);
     e->vecs.assign(nw, nullptr);
 
-    e->out_cap = c.max_seq > 4096 ? c.max_seq : 4096;
     const int half = c.head_dim / 2;
     const size_t kv_elems = (size_t)c.n_layers * c.max_seq * c.kv_dim;
     {
@@ -1319,8 +1381,7 @@ int mg_create(const mg_config* cfg, mg_engine** out) {
     if ((rc = dev_alloc(e, &e->attn, (size_t)c.dim))) return bail(rc);
     if ((rc = dev_alloc(e, &e->mid, (size_t)c.ffn_dim))) return bail(rc);
     if ((rc = dev_alloc(e, &e->logits, (size_t)c.vocab))) return bail(rc);
-    if ((rc = dev_alloc(e, &e->st, (size_t)1))) return bail(rc);
-    if ((rc = dev_alloc(e, &e->out_tokens, (size_t)e->out_cap))) return bail(rc);
+    if ((rc = create_cursor(e))) return bail(rc);
 
     // RoPE tables in float64 on the host, narrowed to fp32 (cuda_fused_infer.go:181-190).
     {
@@ -1337,28 +1398,73 @@ int mg_create(const mg_config* cfg, mg_engine** out) {
             return bail(MG_ERR_CUDA);
     }
     if (cudaMemset(e->kc, 0, kv_elems * 2) != cudaSuccess || cudaMemset(e->vc, 0, kv_elems * 2) != cudaSuccess ||
-        cudaMemset(e->h, 0, (size_t)c.dim * 4) != cudaSuccess || cudaMemset(e->out_tokens, 0, (size_t)e->out_cap * 4) != cudaSuccess)
+        cudaMemset(e->h, 0, (size_t)c.dim * 4) != cudaSuccess)
         return bail(MG_ERR_CUDA);
-    StepState s0{};
-    s0.out_cap = e->out_cap;
-    if (cudaMemcpy(e->st, &s0, sizeof s0, cudaMemcpyHostToDevice) != cudaSuccess) return bail(MG_ERR_CUDA);
-
-    e->pin_i_cap = 8 + e->out_cap;
-    if (cudaMallocHost((void**)&e->pin_i, (size_t)(e->pin_i_cap + 16) * sizeof(int)) != cudaSuccess) return bail(MG_ERR_NOMEM);
-    { const char* zc = getenv("MG_ZERO_COPY"); e->zero_copy = !(zc && zc[0] == '0'); }
 
     if ((rc = set_kernel_attrs(e))) return bail(rc);
-    const char* env = getenv("MG_NO_GRAPH");
-    if (env && env[0] == '1') e->use_graph = false;
-    env = getenv("MG_NO_MEGA");
-    if (env && env[0] == '1') e->use_mega = false;
-    env = getenv("MG_NO_PDL");
-    if (env && env[0] == '1') e->use_pdl = false;
-    // L2 prefetch distance of the persistent kernel's weight stream; 64 KiB measured best on
-    // 7B-class widths (layer time 85 -> 75 us), neutral on the 0.5 B model, 384 KiB thrashes L2
-    env = getenv("MG_PREFETCH_KB");
-    e->mk_prefetch = (env ? atoi(env) : 64) * 1024;
-    if (e->mk_prefetch < 0 || e->mk_prefetch > (1 << 20)) e->mk_prefetch = 0;
+    read_env(e);
+    *out = e;
+    return MG_OK;
+}
+
+int mg_create_layered(const mg_model_config* cfg, const mg_layer_config* layers, mg_engine** out) {
+    if (!cfg || !layers || !out) return MG_ERR_ARG;
+    *out = nullptr;
+    mg_engine* e = new mg_engine();
+    e->lm = new Layered();
+    Layered& m = *e->lm;
+    m.c = *cfg;
+    auto bail = [&](int code, const char* why) {
+        if (why && why[0]) fprintf(stderr, "[mongoose-b200] mg_create_layered: %s\n", why);
+        mg_destroy(e);
+        return code;
+    };
+    if (cfg->n_layers <= 0) return bail(MG_ERR_ARG, "no layers");
+    for (int i = 0; i < cfg->n_layers; i++) {
+        LayerWeights l;
+        l.c = layers[i];
+        m.layers.push_back(l);
+    }
+    mg_config& c = e->cfg;
+    c.dim = cfg->width; c.vocab = cfg->vocab; c.n_layers = cfg->n_layers; c.max_seq = cfg->max_seq; c.rms_eps = cfg->norm_eps;
+    c.layer_fmt = c.head_fmt = MG_FMT_BF16; c.device = cfg->device; c.max_batch = 1;
+    int rc = create_common(e);
+    if (rc) return bail(rc, "no usable device");
+    std::string why;
+    if ((rc = layered_shapes(m, e->num_sms, &why))) return bail(rc, why.c_str());
+    size_t want = 0;
+    layered_buffers(m, [&](void**, size_t bytes) { want += (bytes + 511) & ~(size_t)255; return 0; });
+    want += (size_t)c.vocab * 4 + (size_t)c.dim * 8 + (size_t)e->out_cap * 4 + (4u << 20);
+    if (const char* mb = getenv("MG_ARENA_MB")) want = (size_t)atoll(mb) << 20;
+    if (!e->arena.init(want)) fprintf(stderr, "[mongoose-b200] arena of %zu MB not available: falling back to one allocation per buffer\n", want >> 20);
+    rc = layered_buffers(m, [&](void** p, size_t bytes) {
+        uint8_t* b = nullptr;
+        const int r = dev_alloc(e, &b, bytes);
+        *p = b;
+        // zeros everywhere: the padding columns of weights and activations stay zero
+        return r ? r : cudaMemset(b, 0, bytes) == cudaSuccess ? MG_OK : MG_ERR_CUDA;
+    });
+    if (rc) return bail(rc, e->err.c_str());
+    if ((rc = dev_alloc(e, &e->h, (size_t)c.dim)) || (rc = dev_alloc(e, &e->h2, (size_t)c.dim)) || (rc = dev_alloc(e, &e->logits, (size_t)c.vocab)))
+        return bail(rc, e->err.c_str());
+    if ((rc = create_cursor(e))) return bail(rc, "cursor");
+    layered_slots(m);
+    for (LayerWeights& l : m.layers) {
+        std::vector<float> sl(l.at.heads);
+        for (int h = 0; h < l.at.heads; h++) sl[h] = (float)pow(2.0, -8.0 * (h + 1) / l.at.heads);
+        if (cudaMemcpy(l.slopes, sl.data(), sl.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) return bail(MG_ERR_CUDA, "upload");
+    }
+    {   // position vectors in float64 on the host, narrowed to fp32, like the RoPE tables of mg_create
+        const int W = c.dim;
+        std::vector<double> f((W + 1) / 2);
+        for (size_t i = 0; i < f.size(); i++) f[i] = pow(10000.0, -2.0 * (double)i / W);
+        std::vector<float> tab((size_t)c.max_seq * W);
+        for (int p = 0; p < c.max_seq; p++)
+            for (int i = 0; i < W; i++) tab[(size_t)p * W + i] = (float)(i & 1 ? cos(p * f[i / 2]) : sin(p * f[i / 2]));
+        if (cudaMemcpy(m.pos_tab, tab.data(), tab.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) return bail(MG_ERR_CUDA, "upload");
+    }
+    read_env(e);
+    e->use_mega = false;
     *out = e;
     return MG_OK;
 }
@@ -1403,14 +1509,16 @@ void mg_destroy(mg_engine* e) {
     if (e->stream1) { cudaStreamSynchronize(e->stream1); cudaStreamDestroy(e->stream1); }
     if (e->stream) cudaStreamDestroy(e->stream);
     e->arena.destroy();
+    delete e->lm;
     delete e;
 }
 
-int mg_num_weights(const mg_engine* e) { return e ? e->cfg.n_layers * 12 + 2 : 0; }
+int mg_num_weights(const mg_engine* e) { return !e ? 0 : e->lm ? (int)e->lm->slots.size() : e->cfg.n_layers * 12 + 2; }
 
 int mg_set_weight(mg_engine* e, int idx, const float* data, size_t count) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return layered_set(e, idx, data, count, false);
     bool is_matrix; int rows, cols, fmt;
     if (!data || !slot_info(e->cfg, idx, &is_matrix, &rows, &cols, &fmt))
         return fail(e, MG_ERR_ARG, "mg_set_weight: bad slot %d", idx);
@@ -1435,6 +1543,8 @@ int mg_set_weight(mg_engine* e, int idx, const float* data, size_t count) {
 int mg_set_weight_raw(mg_engine* e, int idx, const void* blocks, size_t bytes, int fmt) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return fmt == MG_FMT_BF16 ? layered_set(e, idx, blocks, bytes / 2, true)
+                                         : fail(e, MG_ERR_ARG, "layer-described models take raw weights as bf16");
     bool is_matrix; int rows, cols, slot_fmt;
     if (!blocks || !slot_info(e->cfg, idx, &is_matrix, &rows, &cols, &slot_fmt) || !is_matrix)
         return fail(e, MG_ERR_ARG, "mg_set_weight_raw: slot %d is not a matrix slot", idx);
@@ -1458,6 +1568,7 @@ int mg_set_weight_raw(mg_engine* e, int idx, const void* blocks, size_t bytes, i
 int mg_build(mg_engine* e) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return layered_build(e);
     const mg_config& c = e->cfg;
     for (int idx = 0; idx < c.n_layers * 12 + 2; idx++) {
         bool is_matrix; int rows, cols, fmt;
@@ -1479,6 +1590,10 @@ int mg_build(mg_engine* e) {
 int mg_reset_kv(mg_engine* e) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) {        // a step at position 0 reads nothing of the old sequence: there is nothing to clear
+        layered_reset(e);
+        return MG_OK;
+    }
     const size_t kv_bytes = (size_t)e->cfg.n_layers * e->cfg.max_seq * e->cfg.kv_dim * 2;
     MG_CUDA(e, cudaMemsetAsync(e->kc, 0, kv_bytes, e->stream));
     MG_CUDA(e, cudaMemsetAsync(e->vc, 0, kv_bytes, e->stream));
@@ -1492,7 +1607,7 @@ int mg_set_cursor(mg_engine* e, int token, int pos) {
     if (pos < 0 || pos >= e->cfg.max_seq || token < 0 || token >= e->cfg.vocab)
         return fail(e, MG_ERR_ARG, "mg_set_cursor: token %d / pos %d out of range", token, pos);
     MG_CUDA(e, cudaStreamSynchronize(e->stream));
-    e->pin_i[0] = pos; e->pin_i[1] = token; e->pin_i[2] = 0;
+    e->pin_i[0] = e->cursor = pos; e->pin_i[1] = token; e->pin_i[2] = 0;
     MG_CUDA(e, cudaMemcpyAsync(e->st, e->pin_i, 12, cudaMemcpyHostToDevice, e->stream));
     return MG_OK;
 }
@@ -1525,7 +1640,7 @@ int mg_partial_step(mg_engine* e, const float* hidden_in, int pos, int layer_sta
         return fail(e, MG_ERR_ARG, "mg_partial_step: bad arguments (pos %d, layers [%d,%d))", pos, layer_start, layer_end);
     if (layer_end > c.n_layers) layer_end = c.n_layers;
     MG_CUDA(e, cudaStreamSynchronize(e->stream));   // pin_i is reused
-    e->pin_i[0] = pos; e->pin_i[1] = 0;
+    e->pin_i[0] = e->cursor = pos; e->pin_i[1] = 0;
     MG_CUDA(e, cudaMemcpyAsync(e->st, e->pin_i, 8, cudaMemcpyHostToDevice, e->stream));
     MG_CUDA(e, cudaMemcpyAsync(e->h, hidden_in, (size_t)c.dim * 4, cudaMemcpyHostToDevice, e->stream));
     const bool want_logits = layer_end >= c.n_layers && logits_out;
@@ -1554,6 +1669,7 @@ int mg_partial_step(mg_engine* e, const float* hidden_in, int pos, int layer_sta
 int mg_set_layer_range(mg_engine* e, int layer_start, int layer_end) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return fail(e, MG_ERR_UNSUPPORTED, "a layer-described model lives on one stage");
     if (layer_start < 0 || layer_end <= layer_start || layer_end > e->cfg.n_layers)
         return fail(e, MG_ERR_ARG, "mg_set_layer_range: bad range [%d,%d) of %d layers", layer_start, layer_end, e->cfg.n_layers);
     if (e->sh.size > 1) return fail(e, MG_ERR_UNSUPPORTED, "mg_set_layer_range: not combined with tensor parallelism");
@@ -1571,7 +1687,7 @@ int mg_partial_step_continue(mg_engine* e, int pos, int layer_start, int layer_e
         return fail(e, MG_ERR_ARG, "mg_partial_step_continue: bad arguments (pos %d, layers [%d,%d))", pos, layer_start, layer_end);
     if (layer_end > c.n_layers) layer_end = c.n_layers;
     MG_CUDA(e, cudaStreamSynchronize(e->stream));   // pin_i is reused; a queued hidden state has landed after this
-    e->pin_i[0] = pos; e->pin_i[1] = 0;
+    e->pin_i[0] = e->cursor = pos; e->pin_i[1] = 0;
     MG_CUDA(e, cudaMemcpyAsync(e->st, e->pin_i, 8, cudaMemcpyHostToDevice, e->stream));
     const bool want_logits = layer_end >= c.n_layers && logits_out;
     if ((rc = run_step(e, layer_start, layer_end, MODE_HIDDEN, want_logits ? HEAD_LOGITS : HEAD_NONE))) return rc;
@@ -1595,7 +1711,7 @@ int mg_step_layer_resident(mg_engine* e, int layer, int pos, const float* hidden
     if (layer < 0 || layer >= c.n_layers || pos < 0 || pos >= c.max_seq || (layer == 0 && !hidden_in))
         return fail(e, MG_ERR_ARG, "mg_step_layer_resident: bad arguments (layer %d, pos %d)", layer, pos);
     MG_CUDA(e, cudaStreamSynchronize(e->stream));
-    e->pin_i[0] = pos; e->pin_i[1] = 0;
+    e->pin_i[0] = e->cursor = pos; e->pin_i[1] = 0;
     MG_CUDA(e, cudaMemcpyAsync(e->st, e->pin_i, 8, cudaMemcpyHostToDevice, e->stream));
     if (layer == 0) MG_CUDA(e, cudaMemcpyAsync(e->h, hidden_in, (size_t)c.dim * 4, cudaMemcpyHostToDevice, e->stream));
     if (pre_out) MG_CUDA(e, cudaMemcpyAsync(pre_out, e->h, (size_t)c.dim * 4, cudaMemcpyDeviceToHost, e->stream));
@@ -1668,7 +1784,7 @@ int mg_partial_step_continue_on_stream1(mg_engine* e, int pos, int layer_start, 
     MG_CUDA(e, cudaStreamSynchronize(e->stream));   // pin_i is reused
     MG_CUDA(e, cudaEventRecord(e->s1_in, e->stream1));
     MG_CUDA(e, cudaStreamWaitEvent(e->stream, e->s1_in, 0));
-    e->pin_i[0] = pos; e->pin_i[1] = 0;
+    e->pin_i[0] = e->cursor = pos; e->pin_i[1] = 0;
     MG_CUDA(e, cudaMemcpyAsync(e->st, e->pin_i, 8, cudaMemcpyHostToDevice, e->stream));
     const bool want_logits = layer_end >= c.n_layers && logits_out;
     if ((rc = run_step(e, layer_start, layer_end, MODE_HIDDEN, want_logits ? HEAD_LOGITS : HEAD_NONE))) return rc;
@@ -1789,7 +1905,7 @@ int mg_graph_launch(mg_engine* e, int pos, int layer_start, int layer_end) {
         return fail(e, MG_ERR_ARG, "mg_graph_launch: bad arguments (pos %d, layers [%d,%d))", pos, layer_start, layer_end);
     if (layer_end > c.n_layers) layer_end = c.n_layers;
     MG_CUDA(e, cudaStreamSynchronize(e->stream));   // the pinned cursor words are reused
-    e->pin_i[0] = pos; e->pin_i[1] = 0;
+    e->pin_i[0] = e->cursor = pos; e->pin_i[1] = 0;
     MG_CUDA(e, cudaMemcpyAsync(e->st, e->pin_i, 8, cudaMemcpyHostToDevice, e->stream));
     return run_step(e, layer_start, layer_end, MODE_HIDDEN, HEAD_NONE);
 }
@@ -1841,7 +1957,7 @@ int mg_step_token(mg_engine* e, int token, int pos, int* next_token, float* logi
     if (token < 0 || token >= c.vocab || pos < 0 || pos >= c.max_seq)
         return fail(e, MG_ERR_ARG, "mg_step_token: token %d / pos %d out of range", token, pos);
     MG_CUDA(e, cudaStreamSynchronize(e->stream));
-    e->pin_i[0] = pos; e->pin_i[1] = token;
+    e->pin_i[0] = e->cursor = pos; e->pin_i[1] = token;
     MG_CUDA(e, cudaMemcpyAsync(e->st, e->pin_i, 8, cudaMemcpyHostToDevice, e->stream));
     if ((rc = run_step(e, 0, c.n_layers, MODE_EMBED, logits_out ? HEAD_LOGITS : HEAD_ARGMAX))) return rc;
     if (logits_out)
@@ -1865,6 +1981,31 @@ int mg_enqueue_greedy(mg_engine* e, int n_steps) {
     return MG_OK;
 }
 
+int mg_forward(mg_engine* e, const int* tokens, int n, int pos, const int* want, int n_want, float* logits_out) {
+    int rc = check_engine(e);
+    if (rc) return rc;
+    if ((rc = ensure_built(e))) return rc;
+    const mg_config& c = e->cfg;
+    if (!tokens || n < 1 || pos < 0 || pos + n > c.max_seq || n_want < 0 || (n_want > 0 && (!want || !logits_out)))
+        return fail(e, MG_ERR_ARG, "mg_forward: %d tokens from position %d do not fit max_seq %d", n, pos, c.max_seq);
+    for (int i = 0; i < n; i++)
+        if (tokens[i] < 0 || tokens[i] >= c.vocab) return fail(e, MG_ERR_ARG, "mg_forward: token id %d out of range", tokens[i]);
+    for (int i = 0; i < n_want; i++)
+        if (want[i] < 0 || want[i] >= n || (i > 0 && want[i] <= want[i - 1]))
+            return fail(e, MG_ERR_ARG, "mg_forward: the wanted places are not ascending places among the tokens");
+    if (e->lm && n > 1) {
+        if ((rc = layered_forward(e, tokens, n, pos, want, n_want, logits_out))) return rc;
+        return check_mega_status(e);
+    }
+    for (int i = 0, w = 0; i < n; i++) {
+        const bool out = w < n_want && want[w] == i;
+        int next;
+        if ((rc = mg_step_token(e, tokens[i], pos + i, &next, out ? logits_out + (size_t)w * c.vocab : nullptr))) return rc;
+        w += out;
+    }
+    return MG_OK;
+}
+
 int mg_generate(mg_engine* e, const int* prompt, int n_prompt, int n_new, int start_pos, int* out_tokens) {
     int rc = check_engine(e);
     if (rc) return rc;
@@ -1877,6 +2018,21 @@ int mg_generate(mg_engine* e, const int* prompt, int n_prompt, int n_new, int st
     for (int i = 0; i < n_prompt; i++)
         if (prompt[i] < 0 || prompt[i] >= c.vocab) return fail(e, MG_ERR_ARG, "mg_generate: prompt id out of range");
     if ((rc = check_range(e, 0, c.n_layers, true, true))) return rc;
+    if (e->lm) {
+        // the prompt but its last token as one portion; that token and the new ones through the decode path
+        const int rows = n_prompt - 1;
+        if (rows == 1) {
+            int skip;
+            if ((rc = mg_step_token(e, prompt[0], start_pos, &skip, nullptr))) return rc;
+        } else if (rows > 0 && (rc = layered_forward(e, prompt, rows, start_pos, nullptr, 0, nullptr))) {
+            return rc;
+        }
+        if ((rc = mg_set_cursor(e, prompt[rows], start_pos + rows))) return rc;
+        for (int i = 0; i < n_new; i++)
+            if ((rc = run_step(e, 0, c.n_layers, MODE_EMBED, HEAD_ARGMAX))) return rc;
+        MG_CUDA(e, cudaMemcpyAsync(out_tokens, e->out_tokens, (size_t)n_new * 4, cudaMemcpyDeviceToHost, e->stream));
+        return check_mega_status(e);
+    }
     MG_CUDA(e, cudaStreamSynchronize(e->stream));
     e->pin_i[0] = start_pos; e->pin_i[1] = prompt[0]; e->pin_i[2] = 0;
     for (int i = 0; i < n_prompt; i++) e->pin_i[8 + i] = prompt[i];
@@ -1904,6 +2060,7 @@ int mg_generate(mg_engine* e, const int* prompt, int n_prompt, int n_new, int st
 int mg_dequant_rows(mg_engine* e, int idx, int row0, int nrows, float* out) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return layered_dequant(e, idx, row0, nrows, out);
     if (!out || idx < 0 || idx >= (int)e->mats.size() || !e->mats[idx].set)
         return fail(e, MG_ERR_ARG, "mg_dequant_rows: slot %d is not a set matrix", idx);
     const DevMatrix& m = e->mats[idx];
@@ -1937,6 +2094,7 @@ int mg_dequant_rows(mg_engine* e, int idx, int row0, int nrows, float* out) {
 int mg_read_kv(mg_engine* e, int layer, int pos0, int npos, uint16_t* k_out, uint16_t* v_out) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return fail(e, MG_ERR_UNSUPPORTED, "mg_read_kv: a layer-described model caches raw keys only");
     const mg_config& c = e->cfg;
     if (layer < 0 || layer >= c.n_layers || pos0 < 0 || npos < 0 || pos0 + npos > c.max_seq)
         return fail(e, MG_ERR_ARG, "mg_read_kv: out of range");
@@ -2054,6 +2212,7 @@ int mg_tp_unique_id(void* id_out, size_t bytes) {
 int mg_tp_init(mg_engine* e, int rank, int size, const void* id, size_t bytes) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return fail(e, MG_ERR_UNSUPPORTED, "layer-described models run on one GPU");
     if (e->any_weight_set || e->comm) return fail(e, MG_ERR_STATE, "mg_tp_init: call once, before any weight is set");
     if (size == 1 && rank == 0) return MG_OK;
     if (!id || bytes < sizeof(ncclUniqueId)) return fail(e, MG_ERR_ARG, "mg_tp_init: need the %zu-byte id of mg_tp_unique_id", sizeof(ncclUniqueId));
@@ -2137,6 +2296,7 @@ int mg_tp_init(mg_engine* e, int rank, int size, const void* id, size_t bytes) {
 int mg_tp_init_absent_peers(mg_engine* e, int size) {
     int rc = check_engine(e);
     if (rc) return rc;
+    if (e->lm) return fail(e, MG_ERR_UNSUPPORTED, "layer-described models run on one GPU");
     if (e->any_weight_set || e->comm || e->xchg) return fail(e, MG_ERR_STATE, "mg_tp_init_absent_peers: call once, before any weight is set");
     if (size < 2 || size > kMaxRanks) return fail(e, MG_ERR_ARG, "mg_tp_init_absent_peers: 2..%d ranks", kMaxRanks);
     std::string why;

@@ -7,7 +7,6 @@
 
 namespace mg {
 
-typedef void (*phase_fn_t)(const PhaseArgs);
 typedef void (*attn_fn_t)(const float*, const __half*, const __half*, float*, const StepState*, int, int, int);
 
 struct DenseKernels {

@@ -1,0 +1,461 @@
+// Portions of a prompt of a layer-described model: row-wise kernels, the 32-bit matrix product, attention on
+// the CUDA cores (32-bit mode and head counts the tensor-core kernel does not take), and the matrix
+// memory in chunked form: every chunk's contribution in parallel, one pass over the chunks, then every
+// chunk's outputs in parallel.
+#include "layered_ops.cuh"
+
+namespace mg {
+
+namespace {
+
+template <typename AT>
+__global__ void __launch_bounds__(256) embed_rows_kernel(WeightView embed, int ld_embed, const float* pos_tab, const int* tokens,
+                                                         int pos0, int width, float* x, AT* act, int ld_act) {
+    const int r = blockIdx.x, token = tokens[r];
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = embed_value(embed, FMT_BF16, ld_embed, token, i) + pos_tab[(size_t)(pos0 + r) * width + i];
+        x[(size_t)r * width + i] = v;
+        from_f32(v, act + (size_t)r * ld_act + i);
+    }
+}
+
+// 64 x 64 tile, 16 columns of K per step, 4 x 4 outputs per thread.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W,
+                                                       int ldw, float* out, int ldc, int n, int rows, int K, int gelu) {
+    __shared__ __align__(16) float As[16][68], Ws[16][68];
+    const int r0 = blockIdx.y * 64, c0 = blockIdx.x * 64;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < K; k0 += 16) {
+        float4 av = make_float4(0.f, 0.f, 0.f, 0.f);
+        float2 w0 = make_float2(0.f, 0.f), w1 = w0;
+        if (r0 + lr < n) av = *reinterpret_cast<const float4*>(A + (size_t)(r0 + lr) * lda + k0 + lk);
+        if (c0 + lr < rows) {
+            const __nv_bfloat16* wp = W + (size_t)(c0 + lr) * ldw + k0 + lk;
+            w0 = pair_f32(wp);
+            w1 = pair_f32(wp + 2);
+        }
+        As[lk][lr] = av.x; As[lk + 1][lr] = av.y; As[lk + 2][lr] = av.z; As[lk + 3][lr] = av.w;
+        Ws[lk][lr] = w0.x; Ws[lk + 1][lr] = w0.y; Ws[lk + 2][lr] = w1.x; Ws[lk + 3][lr] = w1.y;
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 16; k++) {
+            const float4 a = *reinterpret_cast<const float4*>(&As[k][ty * 4]), w = *reinterpret_cast<const float4*>(&Ws[k][tx * 4]);
+            const float aa[4] = {a.x, a.y, a.z, a.w}, ww[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(aa[i], ww[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int r = r0 + ty * 4 + i, c = c0 + tx * 4 + j;
+            if (r < n && c < rows) out[(size_t)r * ldc + c] = gelu ? gelu_tanh(acc[i][j]) : acc[i][j];
+        }
+}
+
+// One warp per (token, query head or key head).
+template <typename AT>
+__global__ void __launch_bounds__(256) qk_rows_kernel(GateAttn A, const float* proj, int ldp, int q_col, int k_col, int pos0, int n,
+                                                      AT* qh) {
+    const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+    const int per = A.heads + A.kv_heads, t = w / per, h = w - t * per;
+    if (t >= n) return;
+    const float* row = proj + (size_t)t * ldp;
+    if (h < A.heads)
+        norm_query(A, row + q_col + h * A.dim, query_temp(A, pos0 + t), qh + ((size_t)t * A.heads + h) * A.dim_s, lane);
+    else
+        store_key<AT>(A, row + k_col + (h - A.heads) * A.dim, pos0 + t, h - A.heads, lane);
+}
+
+template <typename KT, int NQ, int EP>
+__global__ void __launch_bounds__(kAttnThreads) gate_attn_rows_kernel(GateAttn A, const KT* qh, int pos0, int n, int tile, KT* out,
+                                                                      int ld_out) {
+    extern __shared__ __align__(16) float smem[];
+    const AttnSmem<KT> sm(A, NQ, tile, smem);
+    const int t0 = (gridDim.x - 1 - blockIdx.x) * NQ;      // the longest rows first
+    const int row = A.heads * A.dim_s;
+    for (int i = threadIdx.x; i < NQ * row; i += kAttnThreads) sm.q[i] = t0 + i / row < n ? to_f32(qh[(size_t)t0 * row + i]) : 0.f;
+    sm.load_tables(A);
+    __syncthreads();
+    const int last = min(t0 + NQ, n) - 1;
+    float acc[NQ][EP][2] = {};
+    attend<KT, NQ, EP>(A, sm, pos0 + t0, 0, pos0 + last + 1, tile, acc);
+#pragma unroll
+    for (int e = 0; e < EP; e++) {
+        const int el = 2 * (threadIdx.x + e * kAttnThreads);
+        if (el >= row) continue;
+        const int h = el / A.dim_s, d = el - h * A.dim_s;
+#pragma unroll
+        for (int q = 0; q < NQ; q++) {
+            if (t0 + q > last) continue;
+            KT* o = out + (size_t)(t0 + q) * ld_out + h * A.dim + d;
+            if (d < A.dim) from_f32(acc[q][e][0], o);
+            if (d + 1 < A.dim) from_f32(acc[q][e][1], o + 1);
+        }
+    }
+}
+
+template <typename AT>
+__global__ void __launch_bounds__(256) post_rows_kernel(float* x, const float* z0, const float* z1, const float* w0, const float* w1,
+                                                        const float* post_w, float eps, int width, AT* act, int ld_act) {
+    extern __shared__ __align__(16) float y[];
+    __shared__ float red[40];
+    const size_t r = blockIdx.x;
+    const float inv = 1.0f / (float)width;
+    const float *a = z0 + r * width, *b = z1 ? z1 + r * width : nullptr;
+    float ra = 1.f, rb = 0.f, ss = 0.f;
+    if (b) {
+        float s0 = 0.f, s1 = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) { s0 = fmaf(a[i], a[i], s0); s1 = fmaf(b[i], b[i], s1); }
+        ra = 0.5f / sqrtf(block_sum(s0, red) * inv + eps);
+        rb = 0.5f / sqrtf(block_sum(s1, red) * inv + eps);
+    }
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = b ? a[i] * ra * w0[i] + b[i] * rb * w1[i] : a[i];
+        y[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    const float rr = 1.0f / sqrtf(block_sum(ss, red) * inv + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = x[r * width + i] + y[i] * rr * (1.0f + post_w[i]);
+        x[r * width + i] = v;
+        from_f32(v, act + r * ld_act + i);
+    }
+}
+
+template <typename AT>
+__global__ void __launch_bounds__(256) last_norm_rows_kernel(const float* x, const int* rows, const float* w, float eps, int width,
+                                                             AT* act, int ld_act) {
+    __shared__ float red[40];
+    const float* a = x + (size_t)rows[blockIdx.x] * width;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(a[i], a[i], ss);
+    const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) from_f32(a[i] * r * (1.0f + w[i]), act + (size_t)blockIdx.x * ld_act + i);
+}
+
+// ---------------------------------------------------------------------
+// Matrix memory in chunks of kMemChunk tokens.
+// ---------------------------------------------------------------------
+
+// One warp per head: gates, the log-forget sum inside each chunk, and the running maximum
+// m_t = max(f_t + m_{t-1}, i_t) as a scan of the maps m -> max(m + f, i).
+__global__ void __launch_bounds__(32) mem_gates_kernel(MatMem M, int i_col, int f_col, const float* proj, int ldp, int pos0, int n,
+                                                       MemRows w) {
+    const int h = blockIdx.x, lane = threadIdx.x;
+    float m = pos0 == 0 ? 0.f : M.m[(pos0 & 1) * M.heads + h];
+    if (lane == 0) w.m0[h] = m;
+    double base = 0.0;
+    for (int t0 = 0; t0 < n; t0 += 32) {
+        const int t = t0 + lane;
+        float ig = -INFINITY, fg = 0.f;
+        if (t < n) {
+            ig = soft_cap(proj[(size_t)t * ldp + i_col + h] + M.i_bias[h], M.cap);
+            fg = log_sigmoid(soft_cap(proj[(size_t)t * ldp + f_col + h] + M.f_bias[h], M.cap));
+        }
+        if (t0 % kMemChunk == 0) base = 0.0;
+        double b = (double)fg;
+        float mi = ig;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double pb = __shfl_up_sync(MG_FULL_MASK, b, o);
+            const float pm = __shfl_up_sync(MG_FULL_MASK, mi, o);
+            if (lane >= o) { mi = fmaxf((float)((double)pm + b), mi); b += pb; }
+        }
+        const float mt = fmaxf((float)((double)m + b), mi);
+        if (t < n) {
+            w.b[(size_t)h * n + t] = base + b;
+            w.ig[(size_t)h * n + t] = ig;
+            w.mm[(size_t)h * n + t] = mt;
+        }
+        base += __shfl_sync(MG_FULL_MASK, b, 31);
+        m = __shfl_sync(MG_FULL_MASK, mt, 31);       // tokens past n have f = 0 and i = -inf: m passes through
+    }
+    if (lane == 0) M.m[((pos0 + n) & 1) * M.heads + h] = m;
+}
+
+// Running maximum before token t0 of the portion (the state's own slot may be overwritten by now).
+__device__ __forceinline__ float mem_before(const MemRows& w, int h, int n, int t0) {
+    return t0 > 0 ? w.mm[(size_t)h * n + t0 - 1] : w.m0[h];
+}
+
+// U[chunk][head] = sum over the chunk of exp(b_T - b_s + i_s - m_T) k_s v_s^T, a 64 x 64 tile per CTA.
+__global__ void __launch_bounds__(256) mem_chunk_kernel(MatMem M, int k_col, int v_col, const float* proj, int ldp, int n, int vtiles,
+                                                        MemRows w) {
+    __shared__ __align__(16) float Ks[kMemChunk][68], Vs[kMemChunk][68];
+    const int ch = blockIdx.x, h = blockIdx.y, d0 = blockIdx.z / vtiles * 64, v0 = blockIdx.z % vtiles * 64;
+    const int t0 = ch * kMemChunk, T = min(kMemChunk, n - t0);
+    const double bT = w.b[(size_t)h * n + t0 + T - 1];
+    const float mT = w.mm[(size_t)h * n + t0 + T - 1];
+    for (int i = threadIdx.x; i < kMemChunk * 64; i += 256) {
+        const int s = i >> 6, c = i & 63;
+        float k = 0.f, v = 0.f;
+        if (s < T) {
+            const float* row = proj + (size_t)(t0 + s) * ldp;
+            if (d0 + c < M.dim)
+                k = row[k_col + h * M.dim + d0 + c] *
+                    expf((float)(bT - w.b[(size_t)h * n + t0 + s]) + w.ig[(size_t)h * n + t0 + s] - mT);
+            if (v0 + c < M.vdim) v = row[v_col + h * M.vdim + v0 + c];
+        }
+        Ks[s][c] = k;
+        Vs[s][c] = v;
+    }
+    __syncthreads();
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    float acc[4][4] = {}, nk[4] = {};
+#pragma unroll 8
+    for (int s = 0; s < kMemChunk; s++) {
+        const float4 a = *reinterpret_cast<const float4*>(&Ks[s][ty * 4]), b = *reinterpret_cast<const float4*>(&Vs[s][tx * 4]);
+        const float aa[4] = {a.x, a.y, a.z, a.w}, bb[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            nk[i] += aa[i];
+#pragma unroll
+            for (int j = 0; j < 4; j++) acc[i][j] = fmaf(aa[i], bb[j], acc[i][j]);
+        }
+    }
+    float* U = w.U + ((size_t)ch * M.heads + h) * M.dim * M.vdim;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int d = d0 + ty * 4 + i;
+        if (d >= M.dim) continue;
+        if (v0 == 0 && tx == 0) w.nU[((size_t)ch * M.heads + h) * M.dim + d] = nk[i];
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+            if (v0 + tx * 4 + j < M.vdim) U[(size_t)d * M.vdim + v0 + tx * 4 + j] = acc[i][j];
+    }
+}
+
+// Pass over the chunks: U becomes the state BEFORE each chunk, and the state after the last is stored.
+__global__ void __launch_bounds__(256) mem_scan_kernel(MatMem M, int pos0, int n, int chunks, MemRows w) {
+    const size_t per = (size_t)M.dim * M.vdim, all = M.heads * per, nall = (size_t)M.heads * M.dim;
+    const size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (e >= all + nall) return;
+    const bool is_n = e >= all;
+    const size_t i = is_n ? e - all : e;
+    const int h = (int)(i / (is_n ? (size_t)M.dim : per));
+    float* U = is_n ? w.nU + i : w.U + i;
+    const size_t stride = is_n ? nall : all;
+    float s = 0.f;
+    if (pos0 > 0) s = is_n ? M.nrm[(pos0 & 1) * nall + i] : M.S[i];
+    for (int c = 0; c < chunks; c++) {
+        const int t0 = c * kMemChunk, tl = min(t0 + kMemChunk, n) - 1;
+        const float g = expf((float)w.b[(size_t)h * n + tl] + mem_before(w, h, n, t0) - w.mm[(size_t)h * n + tl]);
+        const float u = U[c * stride];
+        U[c * stride] = s;
+        s = fmaf(g, s, u);
+    }
+    if (is_n) M.nrm[((pos0 + n) & 1) * nall + i] = s;
+    else M.S[i] = s;
+}
+
+// Outputs of one chunk and head, 64 value columns per CTA.
+__global__ void __launch_bounds__(256) mem_out_kernel(MatMem M, int q_col, int k_col, int v_col, const float* proj, int ldp,
+                                                      int n, MemRows w) {
+    __shared__ __align__(16) float Qs[32][68], Ks[32][68], Ss[32][68];
+    __shared__ __align__(16) float P[kMemChunk][68];            // [s][t]
+    __shared__ float nq_s[kMemChunk];
+    __shared__ double bs[kMemChunk];
+    __shared__ float is[kMemChunk], ms[kMemChunk];
+    float (*Vs)[68] = reinterpret_cast<float (*)[68]>(&Qs[0][0]);   // 64 rows over Qs and Ks once they are consumed
+    static_assert(sizeof(Qs) + sizeof(Ks) == 64 * 68 * 4, "the value tile reuses the query and key tiles");
+    const int ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * 64;
+    const int t0 = ch * kMemChunk, T = min(kMemChunk, n - t0);
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    if (threadIdx.x < kMemChunk) {
+        const int t = threadIdx.x;
+        bs[t] = t < T ? w.b[(size_t)h * n + t0 + t] : 0.0;
+        is[t] = t < T ? w.ig[(size_t)h * n + t0 + t] : -INFINITY;
+        ms[t] = t < T ? w.mm[(size_t)h * n + t0 + t] : 0.f;
+    }
+    const float mprev = mem_before(w, h, n, t0);
+    const float qscale = 1.0f / sqrtf((float)M.dim);
+    const float* U = w.U + ((size_t)ch * M.heads + h) * M.dim * M.vdim;
+    const float* nU = w.nU + ((size_t)ch * M.heads + h) * M.dim;
+    float pa[4][4] = {}, oa[4][4] = {};         // rows t = ty*4.., columns s or v = tx*4..
+    float nq = 0.f;                             // thread t < 64: n_prev . q_t
+    for (int k0 = 0; k0 < M.dim; k0 += 32) {
+        __syncthreads();
+        for (int i = threadIdx.x; i < 32 * 64; i += 256) {
+            const int t = i >> 5, d = i & 31;
+            float q = 0.f, k = 0.f;
+            if (t < T && k0 + d < M.dim) {
+                const float* row = proj + (size_t)(t0 + t) * ldp + h * M.dim + k0 + d;
+                q = row[q_col] * qscale;
+                k = row[k_col];
+            }
+            Qs[d][t] = q;
+            Ks[d][t] = k;
+            const int sd = i >> 6, sv = i & 63;
+            Ss[sd][sv] = k0 + sd < M.dim && v0 + sv < M.vdim ? U[(size_t)(k0 + sd) * M.vdim + v0 + sv] : 0.f;
+        }
+        __syncthreads();
+        if (threadIdx.x < kMemChunk)
+            for (int d = 0; d < 32 && k0 + d < M.dim; d++) nq = fmaf(nU[k0 + d], Qs[d][threadIdx.x], nq);
+#pragma unroll 8
+        for (int d = 0; d < 32; d++) {
+            const float4 a = *reinterpret_cast<const float4*>(&Qs[d][ty * 4]), b = *reinterpret_cast<const float4*>(&Ks[d][tx * 4]),
+                         c = *reinterpret_cast<const float4*>(&Ss[d][tx * 4]);
+            const float aa[4] = {a.x, a.y, a.z, a.w}, bb[4] = {b.x, b.y, b.z, b.w}, cc[4] = {c.x, c.y, c.z, c.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    pa[i][j] = fmaf(aa[i], bb[j], pa[i][j]);
+                    oa[i][j] = fmaf(aa[i], cc[j], oa[i][j]);
+                }
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int t = ty * 4 + i;
+        const float inter = t < T ? expf((float)bs[t] + mprev - ms[t]) : 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int s = tx * 4 + j;
+            P[s][t] = s <= t && t < T ? pa[i][j] * expf((float)(bs[t] - bs[s]) + is[s] - ms[t]) : 0.f;
+            oa[i][j] *= inter;
+        }
+    }
+    for (int i = threadIdx.x; i < kMemChunk * 64; i += 256) {
+        const int s = i >> 6, c = i & 63;
+        Vs[s][c] = s < T && v0 + c < M.vdim ? proj[(size_t)(t0 + s) * ldp + v_col + h * M.vdim + v0 + c] : 0.f;
+    }
+    __syncthreads();
+    if (threadIdx.x < kMemChunk) {
+        const int t = threadIdx.x;
+        float d = nq * (t < T ? expf((float)bs[t] + mprev - ms[t]) : 0.f);
+        for (int s = 0; s < kMemChunk; s++) d += P[s][t];
+        nq_s[t] = 1.0f / (fmaxf(fabsf(d), expf(-ms[t])) + 1e-6f);
+    }
+#pragma unroll 8
+    for (int s = 0; s < kMemChunk; s++) {
+        const float4 a = *reinterpret_cast<const float4*>(&P[s][ty * 4]), b = *reinterpret_cast<const float4*>(&Vs[s][tx * 4]);
+        const float aa[4] = {a.x, a.y, a.z, a.w}, bb[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) oa[i][j] = fmaf(aa[i], bb[j], oa[i][j]);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int t = ty * 4 + i;
+        if (t >= T) continue;
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int v = v0 + tx * 4 + j;
+            if (v < M.vdim) w.o[(size_t)(t0 + t) * M.heads * M.vdim + h * M.vdim + v] = oa[i][j] * nq_s[t];
+        }
+    }
+}
+
+// One warp per (token, head): unit rms, norm weight, output gate.
+template <typename AT>
+__global__ void __launch_bounds__(256) mem_norm_kernel(MatMem M, int g_col, const float* proj, int ldp, int n, const float* o, AT* act,
+                                                       int ld_act) {
+    const int wq = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+    const int t = wq / M.heads, h = wq - t * M.heads;
+    if (t >= n) return;
+    const float* p = o + ((size_t)t * M.heads + h) * M.vdim;
+    float ss = 0.f;
+    for (int v = lane; v < M.vdim; v += 32) ss = fmaf(p[v], p[v], ss);
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)M.vdim + M.eps);
+    for (int v = lane; v < M.vdim; v += 32) {
+        const int c = h * M.vdim + v;
+        from_f32(p[v] * r * M.norm[c] * sigmoid(proj[(size_t)t * ldp + g_col + c]), act + (size_t)t * ld_act + c);
+    }
+}
+
+template <typename KT, int NQ>
+cudaError_t attn_rows_for(const GateAttn& at, const void* qh, int pos0, int n, void* out, int ld_out, cudaStream_t s) {
+    int tile;
+    const size_t smem = attn_smem(at, NQ, sizeof(KT), &tile);
+    if (!smem) return cudaErrorInvalidValue;
+    auto run = [&](auto kern) {
+        cudaError_t c = cudaFuncSetAttribute((const void*)kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (c != cudaSuccess) return c;
+        kern<<<(n + NQ - 1) / NQ, kAttnThreads, smem, s>>>(at, (const KT*)qh, pos0, n, tile, (KT*)out, ld_out);
+        return cudaGetLastError();
+    };
+    switch (attn_pairs(at)) {
+        case 1: return run(gate_attn_rows_kernel<KT, NQ, 1>);
+        case 2: return run(gate_attn_rows_kernel<KT, NQ, 2>);
+        case 4: return run(gate_attn_rows_kernel<KT, NQ, 4>);
+        case 8: return run(gate_attn_rows_kernel<KT, NQ, 8>);
+        case 16: return run(gate_attn_rows_kernel<KT, NQ, 16>);
+    }
+    return cudaErrorInvalidValue;
+}
+
+}  // namespace
+
+cudaError_t launch_embed_rows(const WeightView& embed, int ld_embed, const float* pos_tab, const int* tokens, int pos0, int n,
+                              int width, float* x, void* act, int ld_act, bool f32, cudaStream_t s) {
+    if (f32) embed_rows_kernel<float><<<n, 256, 0, s>>>(embed, ld_embed, pos_tab, tokens, pos0, width, x, (float*)act, ld_act);
+    else embed_rows_kernel<__nv_bfloat16><<<n, 256, 0, s>>>(embed, ld_embed, pos_tab, tokens, pos0, width, x, (__nv_bfloat16*)act, ld_act);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_gemm_f32(const float* A, int lda, const uint8_t* W, int ldw, float* out, int ldc, int n, int rows, int K, bool gelu,
+                            cudaStream_t s) {
+    const dim3 grid((rows + 63) / 64, (n + 63) / 64);
+    gemm_f32_kernel<<<grid, 256, 0, s>>>(A, lda, (const __nv_bfloat16*)W, ldw, out, ldc, n, rows, K, gelu ? 1 : 0);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_qk_rows(const GateAttn& at, const float* proj, int ldp, int q_col, int k_col, int pos0, int n, void* qh, bool f32,
+                           cudaStream_t s) {
+    const int grid = (n * (at.heads + at.kv_heads) + 7) / 8;
+    if (f32) qk_rows_kernel<float><<<grid, 256, 0, s>>>(at, proj, ldp, q_col, k_col, pos0, n, (float*)qh);
+    else qk_rows_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(at, proj, ldp, q_col, k_col, pos0, n, (__nv_bfloat16*)qh);
+    return cudaGetLastError();
+}
+
+size_t gate_attn_rows_smem(const GateAttn& at, bool f32, int* tile) { return attn_smem(at, 1, f32 ? 4 : 2, tile); }
+
+cudaError_t launch_gate_attn_rows(const GateAttn& at, const void* qh, int pos0, int n, void* out, int ld_out, bool f32, cudaStream_t s) {
+    int tile;
+    const bool four = attn_pairs(at) <= 8 && attn_smem(at, 4, f32 ? 4 : 2, &tile) > 0;
+    if (f32) return four ? attn_rows_for<float, 4>(at, qh, pos0, n, out, ld_out, s) : attn_rows_for<float, 1>(at, qh, pos0, n, out, ld_out, s);
+    return four ? attn_rows_for<__nv_bfloat16, 4>(at, qh, pos0, n, out, ld_out, s)
+                : attn_rows_for<__nv_bfloat16, 1>(at, qh, pos0, n, out, ld_out, s);
+}
+
+cudaError_t launch_post_rows(float* x, const float* z0, const float* z1, const float* w0, const float* w1, const float* post_w, float eps,
+                             int n, int width, void* act, int ld_act, bool f32, cudaStream_t s) {
+    const size_t smem = (size_t)width * sizeof(float);
+    if (f32) post_rows_kernel<float><<<n, 256, smem, s>>>(x, z0, z1, w0, w1, post_w, eps, width, (float*)act, ld_act);
+    else post_rows_kernel<__nv_bfloat16><<<n, 256, smem, s>>>(x, z0, z1, w0, w1, post_w, eps, width, (__nv_bfloat16*)act, ld_act);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_last_norm_rows(const float* x, const int* rows, const float* w, float eps, int n, int width, void* act, int ld_act,
+                                  bool f32, cudaStream_t s) {
+    if (f32) last_norm_rows_kernel<float><<<n, 256, 0, s>>>(x, rows, w, eps, width, (float*)act, ld_act);
+    else last_norm_rows_kernel<__nv_bfloat16><<<n, 256, 0, s>>>(x, rows, w, eps, width, (__nv_bfloat16*)act, ld_act);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_mem_rows(const MatMem& mem, const ProjCols& c, const float* proj, int ldp, int pos0, int n, const MemRows& w, void* act,
+                            int ld_act, bool f32, cudaStream_t s) {
+    const int chunks = (n + kMemChunk - 1) / kMemChunk, dt = (mem.dim + 63) / 64, vt = (mem.vdim + 63) / 64;
+    mem_gates_kernel<<<mem.heads, 32, 0, s>>>(mem, c.mi, c.mf, proj, ldp, pos0, n, w);
+    mem_chunk_kernel<<<dim3(chunks, mem.heads, dt * vt), 256, 0, s>>>(mem, c.mk, c.mv, proj, ldp, n, vt, w);
+    const size_t elems = (size_t)mem.heads * mem.dim * (mem.vdim + 1);
+    mem_scan_kernel<<<(unsigned)((elems + 255) / 256), 256, 0, s>>>(mem, pos0, n, chunks, w);
+    mem_out_kernel<<<dim3(chunks, mem.heads, vt), 256, 0, s>>>(mem, c.mq, c.mk, c.mv, proj, ldp, n, w);
+    const int grid = (n * mem.heads + 7) / 8;
+    if (f32) mem_norm_kernel<float><<<grid, 256, 0, s>>>(mem, c.mg, proj, ldp, n, w.o, (float*)act, ld_act);
+    else mem_norm_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(mem, c.mg, proj, ldp, n, w.o, (__nv_bfloat16*)act, ld_act);
+    return cudaGetLastError();
+}
+
+}  // namespace mg

@@ -9,7 +9,7 @@
 #define MG_FULL_MASK 0xffffffffu
 
 // Weight storage formats (values match MG_FMT_* in mongoose_kernels.h).
-enum : int { FMT_Q8_0 = 0, FMT_Q4_0 = 1, FMT_F16 = 2 };
+enum : int { FMT_Q8_0 = 0, FMT_Q4_0 = 1, FMT_F16 = 2, FMT_BF16 = 3 };
 
 namespace mg {
 
@@ -169,6 +169,26 @@ struct Chunk<FMT_F16> {
         a = fmaf(a2.y, x[1].y, a);
         a = fmaf(a3.x, x[1].z, a);
         a = fmaf(a3.y, x[1].w, a);
+        return a;
+    }
+};
+
+// bf16 weights: the upper half of an fp32, so a shift or a mask converts exactly.
+template <>
+struct Chunk<FMT_BF16> {
+    static constexpr int kWeights = 8;
+    static constexpr bool kScaled = false;
+    __device__ static __forceinline__ int scale_index(int c) { return c; }
+    __device__ static __forceinline__ float dot(uint4 w, const float4* x) {
+        float a = 0.f;
+        a = fmaf(__uint_as_float(w.x << 16), x[0].x, a);
+        a = fmaf(__uint_as_float(w.x & 0xffff0000u), x[0].y, a);
+        a = fmaf(__uint_as_float(w.y << 16), x[0].z, a);
+        a = fmaf(__uint_as_float(w.y & 0xffff0000u), x[0].w, a);
+        a = fmaf(__uint_as_float(w.z << 16), x[1].x, a);
+        a = fmaf(__uint_as_float(w.z & 0xffff0000u), x[1].y, a);
+        a = fmaf(__uint_as_float(w.w << 16), x[1].z, a);
+        a = fmaf(__uint_as_float(w.w & 0xffff0000u), x[1].w, a);
         return a;
     }
 };

@@ -326,6 +326,16 @@ class CUDAFusedInference:
         self._check(rc, "Generate")
         return out
 
+    def Forward(self, tokens, pos: int, want=()) -> np.ndarray:
+        """Tokens at positions pos.. of the sequence, continuing the cache and state; returns the
+        logits [len(want), vocab] after the tokens at the ascending places `want`.  Layer-described
+        models take several tokens as one prompt portion, the dense block one by one."""
+        t = np.ascontiguousarray(tokens, dtype=np.int32)
+        w = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.empty((w.size, self.cfg.vocab), np.float32)
+        self._check(self._lib.mg_forward(self._h, _np_ptr(t), t.size, int(pos), _np_ptr(w), w.size, _np_ptr(out)), "Forward")
+        return out
+
     def SetCursor(self, token: int, pos: int) -> None:
         self._check(self._lib.mg_set_cursor(self._h, int(token), pos), "SetCursor")
 

@@ -11,6 +11,8 @@ from __future__ import annotations
 import numpy as np
 
 from . import configs as mc
+from .layered import GateAttention, LayeredConfig, MatrixMemory, ParallelLayer, slot_shapes
+from .safetensors import to_bf16_bits
 
 
 def single_matvec_case(seed: int = 0, N: int = 4864, K: int = 896):
@@ -79,3 +81,48 @@ def load_engine(engine, cfg: mc.ModelConfig, seed: int = 0, jitter: float = 0.0,
         if on_matrix is not None:
             on_matrix(idx, w, fmt)
         del w
+
+
+# ---- layer-described models -----------------------------------------------------------------------
+
+def mitotar_like(name: str, width: int, n_layers: int, ffn: int, vocab: int, heads: int, kv_heads: int, dim: int, mem_heads: int,
+                 mem_dim: int, max_seq: int) -> LayeredConfig:
+    layer = ParallelLayer(GateAttention(heads, kv_heads, dim, dim ** -0.5, 0.25, 512), MatrixMemory(mem_heads, mem_dim, mem_dim, 15.0), ffn)
+    return LayeredConfig(name=name, width=width, vocab=vocab, layers=(layer,) * n_layers, norm_eps=1e-6, max_seq=max_seq)
+
+
+# layer widths of the dense configurations of the same name
+LAYERED = {c.name: c for c in (
+    mitotar_like("mitotar-tiny", 96, 2, 160, 300, 4, 2, 24, 3, 20, 256),
+    mitotar_like("mitotar-0.5b", 896, 24, 4864, 151936, 14, 2, 64, 4, 128, 4096),
+    mitotar_like("mitotar-1.1b", 2048, 22, 5632, 32000, 32, 4, 64, 8, 128, 4096),
+    mitotar_like("mitotar-7b-width-4l", 3584, 4, 18944, 16000, 28, 4, 128, 8, 256, 4096),
+)}
+
+
+def layered_tensors(cfg: LayeredConfig, seed: int = 0):
+    """Yield (slot, name, layer, fp32 tensor) of a random-init model: matrices N(0, 1 / fan-in), head mixing
+    near the identity, norm weights and biases jittered around their neutral value."""
+    around_zero = {"norm1", "norm2", "final_norm", "at.bias", "mem.i_bias"}
+    for idx, name, layer, rows, cols in slot_shapes(cfg):
+        rng = np.random.default_rng([seed, idx])
+        if rows:
+            w = rng.standard_normal((rows, cols), dtype=np.float32)
+            w *= np.float32(1.0 if name == "embed" else cols ** -0.5)
+        elif name == "at.talk":
+            n = cfg.layers[layer].attn.heads
+            w = (np.eye(n) + 0.3 * n ** -0.5 * rng.standard_normal((n, n))).astype(np.float32).reshape(-1)
+        else:
+            neutral = 0.0 if name in around_zero else 3.0 if name == "mem.f_bias" else 1.0
+            w = (neutral + 0.2 * rng.standard_normal(cols)).astype(np.float32)
+        yield idx, name, layer, w
+
+
+def load_layered(engine, seed: int = 0, on_tensor=None) -> None:
+    """Random-init weights for every slot of a layer-described model."""
+    for idx, name, layer, w in layered_tensors(engine.cfg, seed):
+        bits = to_bf16_bits(w)
+        engine.SetWeightBF16(idx, bits)
+        if on_tensor is not None:
+            on_tensor(name, layer, bits)
+    engine.BuildFusedDispatch()
