@@ -93,6 +93,12 @@ cudaError_t launch_qk_rows(const GateAttn& at, const float* proj, int ldp, int q
 cudaError_t launch_gate_attn_rows(const GateAttn& at, const void* qh, int pos0, int n, void* out, int ld_out, bool f32,
                                   cudaStream_t s);
 size_t gate_attn_rows_smem(const GateAttn& at, bool f32, int* tile);
+// The same on the tensor cores (bf16 only, gate_attn_tc.cu): `weights` holds block_rows rows of every head
+// (gate_attn_tc_rows of them fit `budget`), `vt` the keys transposed; qh has max_rows rows.
+bool gate_attn_tc_fits(const GateAttn& at);
+int gate_attn_tc_rows(const GateAttn& at, int max_seq, int max_rows, size_t budget);
+cudaError_t launch_gate_attn_tc(const GateAttn& at, const void* qh, int pos0, int n, int max_rows, void* weights, int block_rows, void* vt,
+                                void* out, int ld_out, int* status, int* launches, cudaStream_t s);
 // x += norm(z) or x += norm(half the sum of two normed branches); act = x
 cudaError_t launch_post_rows(float* x, const float* z0, const float* z1, const float* w0, const float* w1, const float* post_w,
                              float eps, int n, int width, void* act, int ld_act, bool f32, cudaStream_t s);

@@ -7,6 +7,7 @@ struct LayerWeights {
     mg_layer_config c{};
     ProjCols cols{};
     int splits = 1, tile = 16;
+    int block_rows = 0;                 // queries per block of the tensor-core attention; 0: CUDA-core kernel
     uint8_t *proj = nullptr, *at_o = nullptr, *mem_o = nullptr, *up = nullptr, *down = nullptr;
     float *norm1 = nullptr, *norm2 = nullptr, *at_out = nullptr, *mem_out = nullptr;
     float *q_norm = nullptr, *k_norm = nullptr, *talk = nullptr, *bias = nullptr, *slopes = nullptr;
@@ -40,6 +41,7 @@ struct Layered {
     int *tokens = nullptr, *want = nullptr;
     float *x = nullptr, *P = nullptr, *yr[2] = {}, *zr = nullptr, *logits = nullptr;
     uint8_t *act = nullptr, *qh = nullptr, *ao = nullptr, *my = nullptr, *midr = nullptr, *fin = nullptr;
+    uint8_t *aw = nullptr, *vt = nullptr;   // tensor-core attention: mixed weights of a query block, transposed keys
     MemRows mw{};
     int np = 0;                         // widest projection row
     int* status = nullptr;              // set by a wait inside a tensor-core kernel that ran out
@@ -59,7 +61,7 @@ int layered_buffers(Layered& m, F take) {
         if (!rc) rc = take((void**)p, count * elem);
     };
     int hd = 1, kat = 1, kmem = 1, ff = 1, mh = 1;
-    size_t u = 1, nu = 1, part = 1;
+    size_t u = 1, nu = 1, part = 1, aw = 1, vt = 1;
     for (LayerWeights& l : m.layers) {
         const mg_gate_attn_config& a = l.c.attn;
         const mg_mat_mem_config& r = l.c.mem;
@@ -85,6 +87,10 @@ int layered_buffers(Layered& m, F take) {
         ff = std::max(ff, pad_to(l.c.ffn_dim, 64)); mh = std::max(mh, r.heads);
         const size_t chunks = (T + kMemChunk - 1) / kMemChunk;
         u = std::max(u, chunks * r.heads * r.dim * r.vdim); nu = std::max(nu, chunks * r.heads * r.dim);
+        if (l.block_rows) {
+            aw = std::max(aw, (size_t)a.heads * l.block_rows * pad_to(c.max_seq, 64));
+            vt = std::max(vt, (size_t)a.kv_heads * a.dim * pad_to(c.max_seq, 64));
+        }
         part = std::max(part, (size_t)l.splits * a.heads * l.at.dim_s);
     }
     get(&m.embed, (size_t)c.vocab * kw, 2); get(&m.head, (size_t)c.vocab * kw, 2);
@@ -97,6 +103,7 @@ int layered_buffers(Layered& m, F take) {
     get(&m.logits, (size_t)m.logit_rows * c.vocab, 4);
     get(&m.act, (size_t)T * kw, as); get(&m.qh, (size_t)T * hd, as); get(&m.ao, (size_t)T * kat, as);
     get(&m.my, (size_t)T * kmem, as); get(&m.midr, (size_t)T * ff, as); get(&m.fin, (size_t)m.logit_rows * kw, as);
+    get(&m.aw, aw, 2); get(&m.vt, vt, 2);
     get(&m.mw.b, (size_t)mh * T, 8); get(&m.mw.ig, (size_t)mh * T, 4); get(&m.mw.mm, (size_t)mh * T, 4); get(&m.mw.m0, mh, 4);
     get(&m.mw.U, u, 4); get(&m.mw.nU, nu, 4); get(&m.mw.o, (size_t)T * kmem, 4);
     return rc;
@@ -124,6 +131,7 @@ int layered_shapes(Layered& m, int sms, std::string* why) {
         const int n_mem = r.heads * ((r.vdim + 31) / 32);
         l.splits = std::max(32, sms - n_mem);
         if (!mixer_step_smem(g, q, m.f32, &l.tile)) { *why = "attention heads do not fit one CTA's registers or shared memory"; return MG_ERR_UNSUPPORTED; }
+        if (!m.f32 && gate_attn_tc_fits(g)) l.block_rows = gate_attn_tc_rows(g, c.max_seq, m.max_rows, (size_t)256 << 20);
         ProjCols& p = l.cols;
         int o = 0;
         auto col = [&](int n) { const int at = o; o += n; return at; };
@@ -379,7 +387,13 @@ int layered_rows(mg_engine* e, int pos, int n) {
         const int kat = pad_to(l.kat(), 64), kmem = pad_to(l.kmem(), 64), kff = pad_to(l.c.ffn_dim, 64), np = pad_to(l.cols.total, 4);
         if ((rc = layered_matmul(e, m.act, m.max_rows, kw, l.proj, m.P, np, n, l.cols.total, false))) return rc;
         MG_CUDA(e, launch_qk_rows(l.at, m.P, np, l.cols.q, l.cols.k, pos, n, m.qh, m.f32, s));
-        MG_CUDA(e, launch_gate_attn_rows(l.at, m.qh, pos, n, m.ao, kat, m.f32, s));
+        if (l.block_rows) {
+            int k = 0;
+            MG_CUDA(e, launch_gate_attn_tc(l.at, m.qh, pos, n, m.max_rows, m.aw, l.block_rows, m.vt, m.ao, kat, m.status, &k, s));
+            e->launches += k - 1;
+        } else {
+            MG_CUDA(e, launch_gate_attn_rows(l.at, m.qh, pos, n, m.ao, kat, m.f32, s));
+        }
         MG_CUDA(e, launch_mem_rows(l.mem, l.cols, m.P, np, pos, n, m.mw, m.my, kmem, m.f32, s));
         e->launches += 7;
         if ((rc = layered_matmul(e, m.ao, m.max_rows, kat, l.at_o, m.yr[0], W, n, W, false))) return rc;

@@ -18,7 +18,7 @@ static const char* kNames[] = {
     "mongoose_copy", "mongoose_zero", "mongoose_sync", "mongoose_fp32_to_fp16", "mongoose_fp16_to_fp32",
     "mongoose_partial_step_q4_fused_graph", "mongoose_q4_0_matvec_dp4a_static", "mongoose_static_scratch_error",
     "mongoose_embed_gather",
-    "mg_create", "mg_destroy", "mg_num_weights", "mg_set_weight", "mg_set_weight_raw", "mg_build",
+    "mg_create", "mg_create_layered", "mg_forward", "mg_destroy", "mg_num_weights", "mg_set_weight", "mg_set_weight_raw", "mg_build",
     "mg_reset_kv", "mg_partial_step", "mg_partial_step_continue", "mg_export_hidden", "mg_step_token",
     "mg_generate", "mg_enqueue_greedy", "mg_set_cursor", "mg_get_cursor", "mg_sync", "mg_dequant_rows",
     "mg_read_kv", "mg_trace_step", "mg_set_wait_limit_ms", "mg_decode_path", "mg_tp_init_absent_peers", "mg_device_alloc", "mg_device_free", "mg_device_upload",
