@@ -62,6 +62,11 @@ WORKLOADS = {
     # sequence i on GPU i mod G, each decoded with batch-1 semantics as the reference would (one
     # engine pass per token); select sizes with --sequences / --prompt-len / --steps
     "tinyllama-1.1b-q8_0-seqs": mc.TINYLLAMA_11B,
+    # models described layer by layer (random-init Mitotar at the layer widths of the dense configurations):
+    # prefill and decode, beside the dense model of equal width
+    "mitotar-0.5b": synthetic.LAYERED["mitotar-0.5b"],
+    "mitotar-1.1b": synthetic.LAYERED["mitotar-1.1b"],
+    "mitotar-7b-width-4l": synthetic.LAYERED["mitotar-7b-width-4l"],
     # the single-op configuration: one Q8_0 dequant-matvec, W 4864 x 896 in raw 34-byte blocks
     "q8_0-matvec-4864x896": None,
 }
@@ -77,6 +82,9 @@ def parse_args():
     ap.add_argument("--workload", default="qwen2.5-0.5b-q8_0-b1", choices=sorted(WORKLOADS))
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN)
     ap.add_argument("--sequences", type=int, default=8, help="sequences of the *-seqs workload (full config: 64)")
+    ap.add_argument("--contexts", default="512,4000", help="positions before the timed decode steps of the mitotar-* workloads")
+    ap.add_argument("--prefill", type=int, default=2048, help="tokens of the timed prompt portion of the mitotar-* workloads")
+    ap.add_argument("--no-closest", action="store_true", help="skip the dense model beside a mitotar-* workload")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-e2e", action="store_true", help="skip the host-buffer leg (profiling runs)")
     ap.add_argument("--cpu-steps", type=int, default=0, help="steps of the CPU baseline sample (0 = auto)")
@@ -718,6 +726,134 @@ def run_matvec_workload(args):
     print(json.dumps(line), flush=True)
 
 
+# ---------------------------------------------------------------------------
+# Models described layer by layer
+# ---------------------------------------------------------------------------
+def measured_peak_tflops():
+    try:
+        return float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"]), "measured"
+    except Exception:
+        return 1590.0, "fallback"
+
+
+def timed_decode(torch, eng, context, tok, steps, warm, local_rank):
+    """Device-resident greedy steps after `context` positions; returns ms per step."""
+    stream = torch.cuda.ExternalStream(eng.stream, device=local_rank)
+    eng.SetCursor(tok, context)
+    eng.EnqueueGreedy(warm)
+    eng.Sync()
+    ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    ev0.record(stream)
+    eng.EnqueueGreedy(steps)
+    ev1.record(stream)
+    eng.Sync()
+    return ev0.elapsed_time(ev1) / steps
+
+
+def run_layered_workload(args, cfg, local_rank):
+    """Prefill of one portion and greedy decode at several contexts, random-init weights.  A step is one
+    decode token at the first context; `closest` is the dense model of the same widths (Q8_0 on its
+    default path, prompts fed token by token as it does)."""
+    import torch
+    from mongoose_b200 import layered
+    from mongoose_b200.fused_infer import CUDAFusedInference
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: there is no CPU fallback for this path")
+    torch.cuda.set_device(local_rank)
+    K, W, P = args.steps, max(args.warmup, 3), args.prefill
+    contexts = [int(c) for c in args.contexts.split(",")]
+    cfg = cfg.with_(max_seq=max(max(contexts) + W + K, P))
+    eng = layered.LayeredInference(cfg, device=local_rank)
+    synthetic.load_layered(eng, seed=0)
+    toks = synthetic.prompt_ids(0, max(max(contexts), P), cfg.vocab)
+    peak, peak_src = measured_peak_gbs()
+    tf_peak, _ = measured_peak_tflops()
+    stream = torch.cuda.ExternalStream(eng.stream, device=local_rank)
+    sampler = ClockSampler(local_rank)
+    sampler.start()
+
+    # ---- prefill: the portion from position 0, through the public call (token ids in, no logits out) ----
+    for _ in range(3):
+        eng.Forward(toks[:P], 0)
+    reps = 10
+    ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    launches0 = eng.LaunchCount()
+    sampler.begin()
+    t0 = time.perf_counter()
+    ev0.record(stream)
+    for _ in range(reps):
+        eng.Forward(toks[:P], 0)
+    ev1.record(stream)
+    torch.cuda.synchronize()
+    wall = (time.perf_counter() - t0) / reps
+    sampler.end()
+    ms_prefill = ev0.elapsed_time(ev1) / reps
+    flops = layered.prefill_flops(cfg, P)
+    prefill = {"tokens": P, "value": P / (ms_prefill / 1e3), "unit": "tok/s", "ms": ms_prefill, "wall_ms": wall * 1e3,
+               "tflops": flops / ms_prefill / 1e9, "frac_of_bf16_peak": flops / ms_prefill / 1e9 / tf_peak, "peak_tflops": tf_peak,
+               "launches": (eng.LaunchCount() - launches0) // reps}
+
+    # ---- decode ----
+    decode = []
+    for c in contexts:
+        eng.Forward(toks[:c], 0)
+        sampler.begin()
+        ms = timed_decode(torch, eng, c, int(toks[0]), K, W, local_rank)
+        sampler.end()
+        b = (layered.weight_bytes_per_token(cfg) + 2 * layered.state_bytes(cfg) +
+             layered.cache_bytes_per_position(cfg) * (c + W + (K + 1) / 2.0))
+        decode.append({"context": c, "value": 1e3 / ms, "unit": "tok/s", "ms_per_step": ms, "bytes_per_token": b,
+                       "GB/s": b / ms / 1e6, "frac_of_hbm": b / ms / 1e6 / peak})
+
+    # ---- end to end: token id in, logits out to the host, every step ----
+    eng.Forward(toks[:contexts[0]], 0)
+    logits = torch.empty(cfg.vocab, dtype=torch.float32).pin_memory()
+    for i in range(W):
+        eng.StepToken(int(toks[i]), contexts[0] + i, logits)
+    t0 = time.perf_counter()
+    for i in range(W, W + K):
+        eng.StepToken(int(toks[i % len(toks)]), contexts[0] + i, logits)
+    e2e = (time.perf_counter() - t0) / K
+    clocks = sampler.stop()
+    eng.close()
+
+    closest = None
+    if not args.no_closest:
+        d = {"mitotar-0.5b": mc.QWEN25_05B, "mitotar-1.1b": mc.TINYLLAMA_11B, "mitotar-7b-width-4l": TP_LEG_CFG}[args.workload]
+        d = d.with_(max_seq=contexts[0] + W + K)
+        eng = CUDAFusedInference(d, device=local_rank)
+        synthetic.load_engine(eng, d, seed=0)
+        eng.BuildFusedDispatch()
+        prompt = synthetic.prompt_ids(0, contexts[0], d.vocab)
+        eng.Generate(prompt[:8], 4)
+        stream = torch.cuda.ExternalStream(eng.stream, device=local_rank)
+        ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        ev0.record(stream)
+        tok = int(eng.Generate(prompt, 1)[0])
+        ev1.record(stream)
+        torch.cuda.synchronize()
+        ms_prompt = ev0.elapsed_time(ev1)
+        ms = timed_decode(torch, eng, contexts[0], tok, K, W, local_rank)
+        b = mc.weight_bytes_per_token(d) + mc.kv_bytes_per_position(d) * (contexts[0] + W + (K + 1) / 2.0)
+        closest = {"model": d.name, "format": FMT_NAME[d.layer_fmt], "prefill_tok_s": contexts[0] / (ms_prompt / 1e3), "context": contexts[0],
+                   "decode_tok_s": 1e3 / ms, "GB/s": b / ms / 1e6, "frac_of_hbm": b / ms / 1e6 / peak}
+        eng.close()
+    print(json.dumps({
+        "metric": "decode_tokens_per_s", "value": decode[0]["value"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
+        "ms_per_step": decode[0]["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic",
+        "config": {"workload": args.workload, "width": cfg.width, "layers": cfg.n_layers, "vocab": cfg.vocab, "batch": 1,
+                   "context": contexts[0], "l2": "inputs larger than L2 (weights streamed per token: %d MB)" % (layered.weight_bytes_per_token(cfg) // 2 ** 20),
+                   "timing": "CUDA events on the engine stream"},
+        "prefill": prefill, "decode": decode, "closest": closest,
+        "e2e": {"value": 1.0 / e2e, "unit": "tok/s", "h2d_bytes_per_step": 8, "d2h_bytes_per_step": cfg.vocab * 4 + 4,
+                "api": "StepToken(token, pos, logitsOut) with a pinned host buffer"},
+        "peak_source": peak_src, "clocks": clocks}), flush=True)
+
+
 def main():
     global PROMPT_LEN
     args = parse_args()
@@ -729,6 +865,12 @@ def main():
             run_matvec_workload(args)
         elif rank == 0:
             print(json.dumps({"impl": "reference", "unavailable": "the single-op workload times its CPU side inside the main arm (cpu_baseline)"}))
+        return
+    if args.workload in synthetic.LAYERED:
+        if rank == 0 and args.impl != "reference":
+            run_layered_workload(args, cfg, local_rank)
+        elif rank == 0:
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no layer-described models"}))
         return
     if args.impl == "reference":
         run_reference_arm(args, cfg, rank)

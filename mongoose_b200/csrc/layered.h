@@ -54,6 +54,9 @@ phase_fn_t layered_phase(int epi, int R);
 typedef void (*phase_pair_fn_t)(const PhaseArgs, const PhaseArgs, int);
 phase_pair_fn_t layered_phase_pair(int R);
 
+// Largest dynamic shared memory the phase kernels may be launched with.
+cudaError_t layered_phase_smem(size_t bytes);
+
 struct MixerStep {
     GateAttn at;
     MatMem mem;

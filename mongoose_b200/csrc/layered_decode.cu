@@ -187,6 +187,18 @@ cudaError_t step_for(const MixerStep& a, size_t smem, bool pdl, cudaStream_t s) 
 
 }  // namespace
 
+cudaError_t layered_phase_smem(size_t bytes) {
+    for (int R = 1; R <= 4; R *= 2) {
+        for (int epi : {EPI_STORE, EPI_GELU, EPI_LOGITS}) {
+            cudaError_t c = cudaFuncSetAttribute((const void*)layered_phase(epi, R), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+            if (c != cudaSuccess) return c;
+        }
+        cudaError_t c = cudaFuncSetAttribute((const void*)layered_phase_pair(R), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+        if (c != cudaSuccess) return c;
+    }
+    return cudaSuccess;
+}
+
 size_t mixer_step_smem(const GateAttn& at, const MatMem& mem, bool f32_cache, int* tile) {
     const size_t need_mem = (40 + kAttnThreads + 2 * (size_t)mem.dim) * sizeof(float);
     const size_t need = attn_smem(at, 1, f32_cache ? 4 : 2, tile);

@@ -116,6 +116,7 @@ int layered_shapes(Layered& m, int sms, std::string* why) {
         (c.math != MG_MATH_BF16 && c.math != MG_MATH_F32)) { *why = "bad model sizes"; return MG_ERR_ARG; }
     m.f32 = c.math == MG_MATH_F32;
     m.kw = pad_to(c.width, 64);
+    int kmax = m.kw;
     m.max_rows = std::min(c.max_seq, 2048);
     m.logit_rows = std::max(1, std::min(std::min(128, m.max_rows), (int)((64u << 20) / ((size_t)c.vocab * 4))));
     for (LayerWeights& l : m.layers) {
@@ -140,7 +141,11 @@ int layered_shapes(Layered& m, int sms, std::string* why) {
         p.mi = col(r.heads); p.mf = col(r.heads);
         p.total = o;
         m.np = std::max(m.np, pad_to(o, 4));
+        kmax = std::max(std::max(kmax, pad_to(l.kat(), 64)), std::max(pad_to(l.kmem(), 64), pad_to(l.c.ffn_dim, 64)));
     }
+    // the phase kernels stage a whole input vector per CTA
+    if (kmax > 48 * 1024) { *why = "a matrix with rows of more than 49152 values"; return MG_ERR_UNSUPPORTED; }
+    if (layered_phase_smem(((size_t)kmax + 40) * sizeof(float)) != cudaSuccess) { *why = "kernel attributes"; return MG_ERR_CUDA; }
     return MG_OK;
 }
 

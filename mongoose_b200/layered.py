@@ -121,6 +121,18 @@ def state_bytes(cfg: LayeredConfig) -> int:
     return sum(4 * l.mem.heads * (l.mem.dim * (l.mem.vdim + 1) + 1) for l in cfg.layers)
 
 
+def prefill_flops(cfg: LayeredConfig, n: int) -> float:
+    """Multiply-adds x 2 of a prompt of n tokens from position 0: matrices, causal scores, head mixing and
+    values, and the recurrence of the memory."""
+    total = 0.0
+    for l in cfg.layers:
+        a, m, W = l.attn, l.mem, cfg.width
+        total += n * W * (2 * a.heads * a.dim + a.kv_heads * a.dim + m.heads * (2 * m.dim + 3 * m.vdim + 2) + 2 * l.ffn_dim)
+        total += n * (n + 1) / 2 * a.heads * (2 * a.dim + a.heads)
+        total += n * m.heads * 2 * m.dim * m.vdim
+    return 2.0 * total
+
+
 class LayeredInference(CUDAFusedInference):
     def __init__(self, cfg: LayeredConfig, device: int = 0):
         self.cfg = cfg
