@@ -194,55 +194,142 @@ __device__ __forceinline__ float gelu_tanh(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
-// Prologue of layer-described models.  xs gets K floats, zero from k_valid on; with `keep` the residual
-// sum goes to h_store (never the buffer x_src names: other CTAs still read that one).
-__device__ __forceinline__ void stage_layered(const PhaseArgs& a, float* xs, float* red, bool keep) {
-    const int K = a.K, n = a.k_valid, nt = blockDim.x;
-    const float inv_n = 1.0f / (float)n;
-    for (int i = n + threadIdx.x; i < K; i += nt) xs[i] = 0.f;
-    if (a.pro == PRO_X || a.pro == PRO_EMBED_POS) {
-        const int token = a.pro == PRO_EMBED_POS ? a.st->token : 0, pos = a.pro == PRO_EMBED_POS ? a.st->pos : 0;
-        for (int i = threadIdx.x; i < n; i += nt) {
-            const float v = a.pro == PRO_X ? a.x_src[i]
-                                           : embed_value(a.embed, a.embed_fmt, K, token, i) + a.pos_tab[(size_t)pos * n + i];
-            xs[i] = v;
-            if (keep) a.h_store[i] = v;
-        }
-    } else {
-        float ss = 0.f;
-        if (a.pro == PRO_POST) {
-            for (int i = threadIdx.x; i < n; i += nt) {
-                const float v = a.z[0][i];
-                xs[i] = v;
-                ss = fmaf(v, v, ss);
+// Eight values per thread, loaded before any is used: a vector of up to 8 * blockDim.x values costs one trip
+// to L2.  Rows that are not 16-byte aligned are read value by value.
+struct Values8 {
+    static constexpr int N = 8;
+    float v[N];
+    __device__ __forceinline__ static int index(int j) { return 4 * ((j >> 2) * (int)blockDim.x + (int)threadIdx.x) + (j & 3); }
+    __device__ __forceinline__ static bool aligned(const float* p, int n) { return ((reinterpret_cast<uintptr_t>(p) & 15) | (n & 3)) == 0; }
+    __device__ __forceinline__ void load(const float* p, int base, int n) {
+        const bool vec = aligned(p, n);
+#pragma unroll
+        for (int j = 0; j < N; j += 4) {
+            const int i = base + index(j);
+            if (vec) {
+                const float4 t = i < n ? *reinterpret_cast<const float4*>(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[j] = t.x; v[j + 1] = t.y; v[j + 2] = t.z; v[j + 3] = t.w;
+            } else {
+#pragma unroll
+                for (int k = 0; k < 4; k++) v[j + k] = i + k < n ? p[i + k] : 0.f;
             }
-        } else {
-            float s0 = 0.f, s1 = 0.f;
-            for (int i = threadIdx.x; i < n; i += nt) {
-                const float u = a.z[0][i], v = a.z[1][i];
-                s0 = fmaf(u, u, s0);
-                s1 = fmaf(v, v, s1);
-            }
-            const float r0 = 0.5f / sqrtf(block_sum(s0, red) * inv_n + a.eps);
-            const float r1 = 0.5f / sqrtf(block_sum(s1, red) * inv_n + a.eps);
-            for (int i = threadIdx.x; i < n; i += nt) {
-                const float v = a.z[0][i] * r0 * a.z_w[0][i] + a.z[1][i] * r1 * a.z_w[1][i];
-                xs[i] = v;
-                ss = fmaf(v, v, ss);
-            }
-        }
-        const float r = 1.0f / sqrtf(block_sum(ss, red) * inv_n + a.eps);
-        for (int i = threadIdx.x; i < n; i += nt) {
-            const float v = a.x_src[i] + xs[i] * r * (1.0f + a.post_w[i]);
-            xs[i] = v;
-            if (keep) a.h_store[i] = v;
         }
     }
+    __device__ __forceinline__ float squares() const {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < N; j++) s = fmaf(v[j], v[j], s);
+        return s;
+    }
+    __device__ __forceinline__ void store(float* p, int base, int n) const {
+        const bool vec = aligned(p, n);
+#pragma unroll
+        for (int j = 0; j < N; j += 4) {
+            const int i = base + index(j);
+            if (vec) {
+                if (i < n) *reinterpret_cast<float4*>(p + i) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+            } else {
+#pragma unroll
+                for (int k = 0; k < 4; k++)
+                    if (i + k < n) p[i + k] = v[j + k];
+            }
+        }
+    }
+};
+
+// Two sums over a CTA at once; every thread gets both.  `red` is >= 66 floats of shared memory.
+__device__ __forceinline__ float2 block_sum2(float u, float v, float* red) {
+    u = warp_sum(u);
+    v = warp_sum(v);
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+    __syncthreads();
+    if (lane == 0) { red[wid] = u; red[33 + wid] = v; }
+    __syncthreads();
+    u = lane < nw ? red[lane] : 0.f;
+    v = lane < nw ? red[33 + lane] : 0.f;
+    return make_float2(warp_sum(u), warp_sum(v));
+}
+
+// Prologue of layer-described models.  xs gets K floats, zero from k_valid on; with `keep` the residual
+// sum goes to h_store (never the buffer x_src names: other CTAs still read that one).  `red` is 72 floats.
+// A vector of up to 8 values per thread stays in registers from the first load to the last norm; a
+// longer one goes through xs in pieces, each thread on its own elements.
+__device__ __forceinline__ void stage_layered(const PhaseArgs& a, float* xs, float* red, bool keep) {
+    const int K = a.K, n = a.k_valid, step = Values8::N * blockDim.x;
+    const float inv_n = 1.0f / (float)n;
+    for (int i = n + threadIdx.x; i < K; i += blockDim.x) xs[i] = 0.f;
+    const bool one = n <= step;
+    const bool pair = a.pro == PRO_POST_PAIR, post = pair || a.pro == PRO_POST;
+    float r = 0.f;
+    Values8 x, y;
+    if (post) {
+        float r0 = 1.f, r1 = 0.f, ss = 0.f;
+        Values8 z;
+        if (pair) {
+            float s0 = 0.f, s1 = 0.f;
+            for (int b = 0; b < n; b += step) {
+                y.load(a.z[0], b, n);
+                z.load(a.z[1], b, n);
+                if (one) x.load(a.x_src, 0, n);
+                s0 += y.squares();
+                s1 += z.squares();
+            }
+            const float2 t = block_sum2(s0, s1, red);
+            r0 = 0.5f / sqrtf(t.x * inv_n + a.eps);
+            r1 = 0.5f / sqrtf(t.y * inv_n + a.eps);
+        }
+        for (int b = 0; b < n; b += step) {
+            if (!(one && pair)) {
+                y.load(a.z[0], b, n);
+                if (pair) z.load(a.z[1], b, n);
+                if (one) x.load(a.x_src, 0, n);
+            }
+            if (pair) {
+                Values8 w0, w1;
+                w0.load(a.z_w[0], b, n);
+                w1.load(a.z_w[1], b, n);
+#pragma unroll
+                for (int j = 0; j < Values8::N; j++) y.v[j] = y.v[j] * r0 * w0.v[j] + z.v[j] * r1 * w1.v[j];
+            }
+            ss += y.squares();
+            if (!one) y.store(xs, b, n);
+        }
+        r = 1.0f / sqrtf(block_sum2(ss, 0.f, red).x * inv_n + a.eps);
+    }
+    const int token = a.pro == PRO_EMBED_POS ? a.st->token : 0, pos = a.pro == PRO_EMBED_POS ? a.st->pos : 0;
+    float ss = 0.f;
+    for (int b = 0; b < n; b += step) {
+        if (a.pro == PRO_EMBED_POS) {
+            x.load(a.pos_tab + (size_t)pos * n, b, n);
+#pragma unroll
+            for (int j = 0; j < Values8::N; j++) {
+                const int i = b + Values8::index(j);
+                if (i < n) x.v[j] += embed_value(a.embed, a.embed_fmt, K, token, i);
+            }
+        } else {
+            if (!(one && post)) x.load(a.x_src, b, n);
+            if (post) {
+                Values8 w;
+                w.load(a.post_w, b, n);
+                if (!one) y.load(xs, b, n);
+#pragma unroll
+                for (int j = 0; j < Values8::N; j++) x.v[j] += y.v[j] * r * (1.0f + w.v[j]);
+            }
+        }
+        if (a.last_w) ss += x.squares();
+        if (keep) x.store(a.h_store, b, n);
+        if (!(one && a.last_w)) x.store(xs, b, n);
+    }
     if (a.last_w) {
-        float ss = 0.f;
-        for (int i = threadIdx.x; i < n; i += nt) ss = fmaf(xs[i], xs[i], ss);
-        const float r = 1.0f / sqrtf(block_sum(ss, red) * inv_n + a.eps);
-        for (int i = threadIdx.x; i < n; i += nt) xs[i] = xs[i] * r * (1.0f + a.last_w[i]);
+        const float rl = 1.0f / sqrtf(block_sum2(ss, 0.f, red).x * inv_n + a.eps);
+        for (int b = 0; b < n; b += step) {
+            Values8 w;
+            w.load(a.last_w, b, n);
+            if (!one) x.load(xs, b, n);
+#pragma unroll
+            for (int j = 0; j < Values8::N; j++) x.v[j] *= rl * (1.0f + w.v[j]);
+            x.store(xs, b, n);
+        }
     }
     __syncthreads();
 }

@@ -21,6 +21,8 @@ phase_pair_fn_t layered_phase_pair(int R) {
 
 namespace {
 
+constexpr int kStateRows = 16;      // rows of the state a warp holds at a time
+
 // One token of the matrix memory: CTA (head, slice of 32 value columns); lanes over columns, warps over
 // the rows of the state.  Every slice forms the head's normaliser; slice 0 stores it into the other
 // parity slot, so no slice reads what another writes.
@@ -35,6 +37,19 @@ __device__ __forceinline__ void mem_step(const MixerStep& a, int cta, float* sme
     const int pos = a.st->pos;
     const bool fresh = pos == 0;
     const float* row = a.proj;
+    const int v = slice * 32 + lane;
+    float* S = M.S + (size_t)head * M.dim * M.vdim + v;
+    // the state's rows come first: nothing they wait for is computed here
+    float s0[kStateRows];
+    auto load_rows = [&](int d0) {
+#pragma unroll
+        for (int i = 0; i < kStateRows; i++) {
+            const int d = d0 + wid + i * nw;
+            s0[i] = !fresh && v < M.vdim && d < M.dim ? S[(size_t)d * M.vdim] : 0.f;
+        }
+    };
+    load_rows(0);
+    const float vv = v < M.vdim ? row[a.c.mv + head * M.vdim + v] : 0.f;
     const float ig = soft_cap(row[a.c.mi + head] + M.i_bias[head], M.cap);
     const float fg = log_sigmoid(soft_cap(row[a.c.mf + head] + M.f_bias[head], M.cap));
     const int cur = pos & 1;
@@ -54,17 +69,17 @@ __device__ __forceinline__ void mem_step(const MixerStep& a, int cta, float* sme
     }
     nq = block_sum(nq, red);                // its barriers publish ks and qs
     if (slice == 0 && threadIdx.x == 0) M.m[(cur ^ 1) * M.heads + head] = m1;
-    const int v = slice * 32 + lane;
     float acc = 0.f;
-    if (v < M.vdim) {
-        const float vv = row[a.c.mv + head * M.vdim + v];
-        float* S = M.S + (size_t)head * M.dim * M.vdim + v;
-#pragma unroll 4
-        for (int d = wid; d < M.dim; d += nw) {
-            const float s0 = fresh ? 0.f : S[(size_t)d * M.vdim];
-            const float s1 = fmaf(ks[d], vv, keep * s0);
-            S[(size_t)d * M.vdim] = s1;
-            acc = fmaf(s1, qs[d], acc);
+    for (int d0 = 0; d0 < M.dim; d0 += kStateRows * nw) {
+        if (d0 > 0) load_rows(d0);
+#pragma unroll
+        for (int i = 0; i < kStateRows; i++) {
+            const int d = d0 + wid + i * nw;
+            if (v < M.vdim && d < M.dim) {
+                const float s1 = fmaf(ks[d], vv, keep * s0[i]);
+                S[(size_t)d * M.vdim] = s1;
+                acc = fmaf(s1, qs[d], acc);
+            }
         }
     }
     part[wid * 32 + lane] = acc;
@@ -96,7 +111,7 @@ __global__ void __launch_bounds__(kAttnThreads) mixer_step_kernel(const MixerSte
     // this token's query, and its key where this CTA's range ends with it
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
     const float temp = query_temp(A, pos);
-    for (int h = wid; h < A.heads; h += nw) norm_query(A, a.proj + a.c.q + h * A.dim, temp, sm.q + h * A.dim_s, lane);
+    norm_queries(A, a.proj + a.c.q, temp, sm.q);
     if (j1 == len)
         for (int c = wid; c < A.kv_heads; c += nw) store_key<KT>(A, a.proj + a.c.k + c * A.dim, pos, c, lane);
     sm.load_tables(A);
@@ -111,8 +126,10 @@ __global__ void __launch_bounds__(kAttnThreads) mixer_step_kernel(const MixerSte
     }
 }
 
+constexpr int kJoinCols = 32, kJoinParts = 8;      // outputs per CTA, threads that share one output's splits
+
 // Joins the key splits, and norms and gates the memory's outputs (one CTA per memory head).
-__global__ void __launch_bounds__(128) mixer_join_kernel(const MixerStep a) {
+__global__ void __launch_bounds__(kJoinCols * kJoinParts) mixer_join_kernel(const MixerStep a) {
     __shared__ float red[40];
     pdl_launch_dependents();
     pdl_wait();
@@ -131,17 +148,26 @@ __global__ void __launch_bounds__(128) mixer_join_kernel(const MixerStep a) {
         return;
     }
     const GateAttn& A = a.at;
-    const int e = (blockIdx.x - nm) * blockDim.x + threadIdx.x;
-    if (e >= A.heads * A.dim) return;
-    const int pos = a.st->pos;
+    const int col = threadIdx.x % kJoinCols, grp = threadIdx.x / kJoinCols;
+    const int e = (blockIdx.x - nm) * kJoinCols + col;
+    const bool ok = e < A.heads * A.dim;
     int j0, j1;
-    const int active = key_split(pos + 1, a.splits, a.tile, 0, &j0, &j1);
-    const int src = e / A.dim * A.dim_s + e % A.dim;
+    const int active = key_split(a.st->pos + 1, a.splits, a.tile, 0, &j0, &j1);
+    const int src = ok ? e / A.dim * A.dim_s + e % A.dim : 0;
     const size_t stride = (size_t)A.heads * A.dim_s;
     float v = 0.f;
+    if (ok) {
 #pragma unroll 8
-    for (int s = 0; s < active; s++) v += a.part[s * stride + src];
-    a.attn_out[e] = v;
+        for (int s = grp; s < active; s += kJoinParts) v += a.part[s * stride + src];
+    }
+    __shared__ float sum[kJoinParts][kJoinCols];
+    sum[grp][col] = v;
+    __syncthreads();
+    if (grp == 0 && ok) {
+#pragma unroll
+        for (int g = 1; g < kJoinParts; g++) v += sum[g][col];
+        a.attn_out[e] = v;
+    }
 }
 
 __global__ void __launch_bounds__(256) resolve_kernel(const ResolveArgs a) {
@@ -201,7 +227,7 @@ cudaError_t layered_phase_smem(size_t bytes) {
 
 size_t mixer_step_smem(const GateAttn& at, const MatMem& mem, bool f32_cache, int* tile) {
     const size_t need_mem = (40 + kAttnThreads + 2 * (size_t)mem.dim) * sizeof(float);
-    const size_t need = attn_smem(at, 1, f32_cache ? 4 : 2, tile);
+    const size_t need = attn_smem(at, 1, f32_cache ? 4 : 2, 8, tile);
     return need == 0 ? 0 : need > need_mem ? need : need_mem;
 }
 
@@ -213,11 +239,11 @@ cudaError_t launch_mixer_step(const MixerStep& a, bool f32_cache, bool pdl, cuda
 
 cudaError_t launch_mixer_join(const MixerStep& a, bool pdl, cudaStream_t s) {
     const int nm = a.n_mem ? a.mem.heads : 0;
-    return go(mixer_join_kernel, nm + (a.at.heads * a.at.dim + 127) / 128, 128, 0, pdl, s, a);
+    return go(mixer_join_kernel, nm + (a.at.heads * a.at.dim + kJoinCols - 1) / kJoinCols, kJoinCols * kJoinParts, 0, pdl, s, a);
 }
 
 cudaError_t launch_resolve(const ResolveArgs& a, bool pdl, cudaStream_t s) {
-    const size_t smem = ((size_t)a.p.K + 40) * sizeof(float);
+    const size_t smem = ((size_t)a.p.K + 72) * sizeof(float);
     cudaError_t c = cudaFuncSetAttribute((const void*)resolve_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return c != cudaSuccess ? c : go(resolve_kernel, 1, 256, smem, pdl, s, a);
 }

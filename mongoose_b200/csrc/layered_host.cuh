@@ -145,7 +145,7 @@ int layered_shapes(Layered& m, int sms, std::string* why) {
     }
     // the phase kernels stage a whole input vector per CTA
     if (kmax > 48 * 1024) { *why = "a matrix with rows of more than 49152 values"; return MG_ERR_UNSUPPORTED; }
-    if (layered_phase_smem(((size_t)kmax + 40) * sizeof(float)) != cudaSuccess) { *why = "kernel attributes"; return MG_ERR_CUDA; }
+    if (layered_phase_smem(((size_t)kmax + 72) * sizeof(float)) != cudaSuccess) { *why = "kernel attributes"; return MG_ERR_CUDA; }
     return MG_OK;
 }
 
@@ -297,7 +297,7 @@ int enqueue_layered_step(mg_engine* e, cudaStream_t s, int ls, int le, int mode,
         a.nitems = (a.rows[0] + R - 1) / R;
         int grid;
         layered_phase_shape(e, a.nitems, &grid);
-        MG_CUDA(e, launch(e, s, layered_phase(epi, R), grid, 256, ((size_t)a.K + 40) * sizeof(float), a));
+        MG_CUDA(e, launch(e, s, layered_phase(epi, R), grid, 256, ((size_t)a.K + 72) * sizeof(float), a));
         return MG_OK;
     };
     int rc;
@@ -327,7 +327,7 @@ int enqueue_layered_step(mg_engine* e, cudaStream_t s, int ls, int le, int mode,
             int ga;
             layered_phase_shape(e, a.nitems, &ga);
             const int gb = ga;
-            MG_CUDA(e, launch(e, s, layered_phase_pair(R), ga + gb, 256, ((size_t)std::max(a.K, b.K) + 40) * sizeof(float), a, b, ga));
+            MG_CUDA(e, launch(e, s, layered_phase_pair(R), ga + gb, 256, ((size_t)std::max(a.K, b.K) + 72) * sizeof(float), a, b, ga));
         }
         pending = PRO_POST_PAIR; z0 = m.y[0]; z1 = m.y[1]; w0 = l.at_out; w1 = l.mem_out; pw = l.norm1;
         if (l.c.ffn_dim) {

@@ -59,6 +59,33 @@ __device__ __forceinline__ void norm_query(const GateAttn& A, const float* q, fl
     for (int d = lane; d < A.dim_s; d += 32) from_f32(d < A.dim ? q[d] * r * A.q_norm[d] * A.k_norm[d] : 0.f, out + d);
 }
 
+// The same for every head of one token by the whole CTA, eight lanes per head.
+__device__ __forceinline__ void norm_queries(const GateAttn& A, const float* q, float temp, float* out) {
+    const int sub = threadIdx.x & 7;
+    const unsigned mask = 0xffu << (threadIdx.x & 24);
+    for (int h = threadIdx.x >> 3; h < A.heads; h += kAttnThreads / 8) {
+        const float* p = q + h * A.dim;
+        float v[16], ss = 0.f;              // the first 128 values are loaded at once
+#pragma unroll
+        for (int i = 0; i < 16; i++) {
+            const int d = sub + 8 * i;
+            v[i] = d < A.dim ? p[d] : 0.f;
+            ss = fmaf(v[i], v[i], ss);
+        }
+        for (int d = sub + 128; d < A.dim; d += 8) ss = fmaf(p[d], p[d], ss);
+        ss += __shfl_xor_sync(mask, ss, 1);
+        ss += __shfl_xor_sync(mask, ss, 2);
+        ss += __shfl_xor_sync(mask, ss, 4);
+        const float r = temp * A.scale / sqrtf(ss / (float)A.dim + A.eps);
+#pragma unroll
+        for (int i = 0; i < 16; i++) {
+            const int d = sub + 8 * i;
+            if (d < A.dim_s) out[h * A.dim_s + d] = d < A.dim ? v[i] * r * A.q_norm[d] * A.k_norm[d] : 0.f;
+        }
+        for (int d = sub + 128; d < A.dim_s; d += 8) out[h * A.dim_s + d] = d < A.dim ? p[d] * r * A.q_norm[d] * A.k_norm[d] : 0.f;
+    }
+}
+
 // One warp: key head c of position pos into the cache, with the 1 / rms of the row as stored.
 template <typename KT>
 __device__ __forceinline__ void store_key(const GateAttn& A, const float* k, int pos, int c, int lane) {
@@ -116,10 +143,10 @@ struct AttnSmem {
     }
 };
 
-// Bytes of AttnSmem with the largest tile of 32, 16 or 8 keys that fits; 0 when none does.
-inline size_t attn_smem(const GateAttn& at, int nq, int kt_bytes, int* tile) {
+// Bytes of AttnSmem with the largest tile of at most `most` (32, 16 or 8) keys that fits; 0 when none does.
+inline size_t attn_smem(const GateAttn& at, int nq, int kt_bytes, int most, int* tile) {
     if (!attn_pairs(at)) return 0;
-    for (int t = 32; t >= 8; t /= 2) {
+    for (int t = most; t >= 8; t /= 2) {
         const size_t b = 2 * (size_t)t * at.kv_heads * at.dim_s * kt_bytes +
                          ((size_t)pad_to(2 * t * at.kv_heads, 4) + (size_t)nq * at.heads * (at.dim_s + 2 * t) +
                           (size_t)at.heads * at.heads + 2 * at.heads) * sizeof(float);
@@ -160,6 +187,15 @@ __device__ __forceinline__ void attend(const GateAttn& A, const AttnSmem<KT>& sm
     const int H = A.heads, DS = A.dim_s, row = A.kv_heads * DS, group = H / A.kv_heads;
     const int sub = threadIdx.x & 7, gid = threadIdx.x >> 3;
     const int chunks = DS / CN;
+    const int ts = 31 - __clz(tile);                // tiles are powers of two
+    int head_of[EP], key_of[EP];                    // this thread's output elements
+#pragma unroll
+    for (int e = 0; e < EP; e++) {
+        const int el = 2 * (threadIdx.x + e * kAttnThreads);
+        const int h = el / DS;
+        head_of[e] = el < H * DS ? h : -1;
+        key_of[e] = h / group * DS + el - h * DS;
+    }
     load_keys<KT>(A, sm, 0, j0, j1, tile);
     cp_async_commit();
     int buf = 0;
@@ -171,7 +207,7 @@ __device__ __forceinline__ void attend(const GateAttn& A, const AttnSmem<KT>& sm
         const KT* K = sm.k + (size_t)buf * tile * row;
         const float* R = sm.r + buf * tile * A.kv_heads;
         for (int u = gid; u < H * tile; u += kAttnThreads / 8) {
-            const int h = u / tile, p = u - h * tile, c = h / group;
+            const int h = u >> ts, p = u & (tile - 1), c = h / group;
             const KT* kp = K + (size_t)p * row + c * DS;
             float dot[NQ] = {};
             for (int ch = sub; ch < chunks; ch += 8) {
@@ -204,19 +240,25 @@ __device__ __forceinline__ void attend(const GateAttn& A, const AttnSmem<KT>& sm
         }
         __syncthreads();
         for (int u = threadIdx.x; u < NQ * H * tile; u += kAttnThreads) {
-            const int p = u % tile, qh = u / tile, h = qh % H;
+            const int p = u & (tile - 1), qh = u >> ts, h = NQ == 1 ? qh : qh % H;
             const float* wq = sm.w + (qh - h) * tile + p;
             const float* t = sm.talk + h * H;
-            float v = 0.f;
-            for (int g = 0; g < H; g++) v = fmaf(t[g], wq[g * tile], v);
-            sm.mix[u] = v;
+            float v0 = 0.f, v1 = 0.f;
+            int g = 0;
+#pragma unroll 4
+            for (; g + 1 < H; g += 2) {
+                v0 = fmaf(t[g], wq[g * tile], v0);
+                v1 = fmaf(t[g + 1], wq[(g + 1) * tile], v1);
+            }
+            if (g < H) v0 = fmaf(t[g], wq[g * tile], v0);
+            sm.mix[u] = v0 + v1;
         }
         __syncthreads();
 #pragma unroll
         for (int e = 0; e < EP; e++) {
-            const int el = 2 * (threadIdx.x + e * kAttnThreads);
-            if (el < H * DS) {
-                const int h = el / DS, off = h / group * DS + el - h * DS;
+            const int h = head_of[e], off = key_of[e];
+            if (h >= 0) {
+#pragma unroll 8
                 for (int p = 0; p < tile; p++) {
                     const float2 kv = pair_f32(K + (size_t)p * row + off);
 #pragma unroll

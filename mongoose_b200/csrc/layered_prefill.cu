@@ -377,7 +377,7 @@ __global__ void __launch_bounds__(256) mem_norm_kernel(MatMem M, int g_col, cons
 template <typename KT, int NQ>
 cudaError_t attn_rows_for(const GateAttn& at, const void* qh, int pos0, int n, void* out, int ld_out, cudaStream_t s) {
     int tile;
-    const size_t smem = attn_smem(at, NQ, sizeof(KT), &tile);
+    const size_t smem = attn_smem(at, NQ, sizeof(KT), 32, &tile);
     if (!smem) return cudaErrorInvalidValue;
     auto run = [&](auto kern) {
         cudaError_t c = cudaFuncSetAttribute((const void*)kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -419,11 +419,11 @@ cudaError_t launch_qk_rows(const GateAttn& at, const float* proj, int ldp, int q
     return cudaGetLastError();
 }
 
-size_t gate_attn_rows_smem(const GateAttn& at, bool f32, int* tile) { return attn_smem(at, 1, f32 ? 4 : 2, tile); }
+size_t gate_attn_rows_smem(const GateAttn& at, bool f32, int* tile) { return attn_smem(at, 1, f32 ? 4 : 2, 32, tile); }
 
 cudaError_t launch_gate_attn_rows(const GateAttn& at, const void* qh, int pos0, int n, void* out, int ld_out, bool f32, cudaStream_t s) {
     int tile;
-    const bool four = attn_pairs(at) <= 8 && attn_smem(at, 4, f32 ? 4 : 2, &tile) > 0;
+    const bool four = attn_pairs(at) <= 8 && attn_smem(at, 4, f32 ? 4 : 2, 32, &tile) > 0;
     if (f32) return four ? attn_rows_for<float, 4>(at, qh, pos0, n, out, ld_out, s) : attn_rows_for<float, 1>(at, qh, pos0, n, out, ld_out, s);
     return four ? attn_rows_for<__nv_bfloat16, 4>(at, qh, pos0, n, out, ld_out, s)
                 : attn_rows_for<__nv_bfloat16, 1>(at, qh, pos0, n, out, ld_out, s);
