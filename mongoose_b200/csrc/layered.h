@@ -113,6 +113,7 @@ struct MemRows {                // workspace of the chunked memory for up to n t
     double* b;                  // [heads][n] log-forget sum inside the chunk
     float* ig;                  // [heads][n] log input gate
     float* mm;                  // [heads][n] running maximum
+    float* g;                   // [heads][chunks] decay of the state over a chunk
     float* m0;                  // [heads] the maximum before the portion
     float* U;                   // [chunks][heads][dim][vdim]
     float* nU;                  // [chunks][heads][dim]

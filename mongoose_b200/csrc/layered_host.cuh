@@ -105,6 +105,7 @@ int layered_buffers(Layered& m, F take) {
     get(&m.my, (size_t)T * kmem, as); get(&m.midr, (size_t)T * ff, as); get(&m.fin, (size_t)m.logit_rows * kw, as);
     get(&m.aw, aw, 2); get(&m.vt, vt, 2);
     get(&m.mw.b, (size_t)mh * T, 8); get(&m.mw.ig, (size_t)mh * T, 4); get(&m.mw.mm, (size_t)mh * T, 4); get(&m.mw.m0, mh, 4);
+    get(&m.mw.g, (size_t)mh * ((T + kMemChunk - 1) / kMemChunk), 4);
     get(&m.mw.U, u, 4); get(&m.mw.nU, nu, 4); get(&m.mw.o, (size_t)T * kmem, 4);
     return rc;
 }

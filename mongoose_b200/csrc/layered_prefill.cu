@@ -144,40 +144,69 @@ __global__ void __launch_bounds__(256) last_norm_rows_kernel(const float* x, con
 // Matrix memory in chunks of kMemChunk tokens.
 // ---------------------------------------------------------------------
 
-// One warp per head: gates, the log-forget sum inside each chunk, and the running maximum
-// m_t = max(f_t + m_{t-1}, i_t) as a scan of the maps m -> max(m + f, i).
-__global__ void __launch_bounds__(32) mem_gates_kernel(MatMem M, int i_col, int f_col, const float* proj, int ldp, int pos0, int n,
-                                                       MemRows w) {
-    const int h = blockIdx.x, lane = threadIdx.x;
-    float m = pos0 == 0 ? 0.f : M.m[(pos0 & 1) * M.heads + h];
-    if (lane == 0) w.m0[h] = m;
-    double base = 0.0;
-    for (int t0 = 0; t0 < n; t0 += 32) {
-        const int t = t0 + lane;
-        float ig = -INFINITY, fg = 0.f;
-        if (t < n) {
-            ig = soft_cap(proj[(size_t)t * ldp + i_col + h] + M.i_bias[h], M.cap);
-            fg = log_sigmoid(soft_cap(proj[(size_t)t * ldp + f_col + h] + M.f_bias[h], M.cap));
-        }
-        if (t0 % kMemChunk == 0) base = 0.0;
-        double b = (double)fg;
-        float mi = ig;
+// One CTA per head, one warp per chunk: gates, the log-forget sum inside each chunk, and the running maximum
+// m_t = max(f_t + m_{t-1}, i_t) as a scan of the maps m -> max(m + f, i): within halves of a chunk by
+// shuffles, across the chunks through shared memory.
+constexpr int kGateWarps = 32;
+
+__global__ void __launch_bounds__(kGateWarps * 32) mem_gates_kernel(MatMem M, int i_col, int f_col, const float* proj, int ldp, int pos0,
+                                                                    int n, MemRows w) {
+    static_assert(kMemChunk == 64, "a warp holds a chunk as two tokens per lane");
+    __shared__ double sum_f[kGateWarps];
+    __shared__ float top_i[kGateWarps], m_end;
+    const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    float m = pos0 == 0 ? 0.f : M.m[(pos0 & 1) * M.heads + h];      // before the chunks of this pass
+    if (threadIdx.x == 0) w.m0[h] = m;
+    const float ib = M.i_bias[h], fb = M.f_bias[h];
+    for (int c0 = 0; c0 * kMemChunk < n; c0 += kGateWarps) {
+        const int t0 = (c0 + warp) * kMemChunk;
+        float ig[2], mi[2];
+        double b[2];
 #pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const double pb = __shfl_up_sync(MG_FULL_MASK, b, o);
-            const float pm = __shfl_up_sync(MG_FULL_MASK, mi, o);
-            if (lane >= o) { mi = fmaxf((float)((double)pm + b), mi); b += pb; }
+        for (int k = 0; k < 2; k++) {
+            const int t = t0 + 32 * k + lane;
+            ig[k] = -INFINITY;                      // tokens past n change nothing: f = 0, i = -inf
+            float fg = 0.f;
+            if (t < n) {
+                ig[k] = soft_cap(proj[(size_t)t * ldp + i_col + h] + ib, M.cap);
+                fg = log_sigmoid(soft_cap(proj[(size_t)t * ldp + f_col + h] + fb, M.cap));
+            }
+            b[k] = (double)fg;
+            mi[k] = ig[k];
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const double pb = __shfl_up_sync(MG_FULL_MASK, b[k], o);
+                const float pm = __shfl_up_sync(MG_FULL_MASK, mi[k], o);
+                if (lane >= o) { mi[k] = fmaxf((float)((double)pm + b[k]), mi[k]); b[k] += pb; }
+            }
         }
-        const float mt = fmaxf((float)((double)m + b), mi);
-        if (t < n) {
-            w.b[(size_t)h * n + t] = base + b;
-            w.ig[(size_t)h * n + t] = ig;
-            w.mm[(size_t)h * n + t] = mt;
+        const double b0 = __shfl_sync(MG_FULL_MASK, b[0], 31);
+        const float i0 = __shfl_sync(MG_FULL_MASK, mi[0], 31);
+        mi[1] = fmaxf((float)((double)i0 + b[1]), mi[1]);
+        b[1] += b0;
+        __syncthreads();                            // the last pass's sums have been read
+        if (lane == 31) { sum_f[warp] = b[1]; top_i[warp] = mi[1]; }
+        __syncthreads();
+        float before = m;
+        for (int c = 0; c < warp; c++) before = fmaxf((float)((double)before + sum_f[c]), top_i[c]);
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+            const int t = t0 + 32 * k + lane;
+            const float mt = fmaxf((float)((double)before + b[k]), mi[k]);
+            if (t < n) {
+                w.b[(size_t)h * n + t] = b[k];
+                w.ig[(size_t)h * n + t] = ig[k];
+                w.mm[(size_t)h * n + t] = mt;
+            }
+            if (k == 1 && lane == 31) {
+                if (t0 < n) w.g[(size_t)h * ((n + kMemChunk - 1) / kMemChunk) + c0 + warp] = expf((float)b[1] + before - mt);
+                if (warp == kGateWarps - 1) m_end = mt;
+            }
         }
-        base += __shfl_sync(MG_FULL_MASK, b, 31);
-        m = __shfl_sync(MG_FULL_MASK, mt, 31);       // tokens past n have f = 0 and i = -inf: m passes through
+        __syncthreads();
+        m = m_end;
     }
-    if (lane == 0) M.m[((pos0 + n) & 1) * M.heads + h] = m;
+    if (threadIdx.x == 0) M.m[((pos0 + n) & 1) * M.heads + h] = m;
 }
 
 // Running maximum before token t0 of the portion (the state's own slot may be overwritten by now).
@@ -244,12 +273,19 @@ __global__ void __launch_bounds__(256) mem_scan_kernel(MatMem M, int pos0, int n
     const size_t stride = is_n ? nall : all;
     float s = 0.f;
     if (pos0 > 0) s = is_n ? M.nrm[(pos0 & 1) * nall + i] : M.S[i];
-    for (int c = 0; c < chunks; c++) {
-        const int t0 = c * kMemChunk, tl = min(t0 + kMemChunk, n) - 1;
-        const float g = expf((float)w.b[(size_t)h * n + tl] + mem_before(w, h, n, t0) - w.mm[(size_t)h * n + tl]);
-        const float u = U[c * stride];
-        U[c * stride] = s;
-        s = fmaf(g, s, u);
+    const float* g = w.g + (size_t)h * chunks;
+    for (int c0 = 0; c0 < chunks; c0 += 8) {        // eight chunks' loads in flight
+        float u[8], gg[8];
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            u[i] = c0 + i < chunks ? U[(c0 + i) * stride] : 0.f;
+            gg[i] = c0 + i < chunks ? g[c0 + i] : 1.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            if (c0 + i < chunks) U[(c0 + i) * stride] = s;
+            s = fmaf(gg[i], s, u[i]);
+        }
     }
     if (is_n) M.nrm[((pos0 + n) & 1) * nall + i] = s;
     else M.S[i] = s;
@@ -260,7 +296,7 @@ __global__ void __launch_bounds__(256) mem_out_kernel(MatMem M, int q_col, int k
                                                       int n, MemRows w) {
     __shared__ __align__(16) float Qs[32][68], Ks[32][68], Ss[32][68];
     __shared__ __align__(16) float P[kMemChunk][68];            // [s][t]
-    __shared__ float nq_s[kMemChunk];
+    __shared__ float nq_s[kMemChunk], ns[32];
     __shared__ double bs[kMemChunk];
     __shared__ float is[kMemChunk], ms[kMemChunk];
     float (*Vs)[68] = reinterpret_cast<float (*)[68]>(&Qs[0][0]);   // 64 rows over Qs and Ks once they are consumed
@@ -282,6 +318,7 @@ __global__ void __launch_bounds__(256) mem_out_kernel(MatMem M, int q_col, int k
     float nq = 0.f;                             // thread t < 64: n_prev . q_t
     for (int k0 = 0; k0 < M.dim; k0 += 32) {
         __syncthreads();
+#pragma unroll
         for (int i = threadIdx.x; i < 32 * 64; i += 256) {
             const int t = i >> 5, d = i & 31;
             float q = 0.f, k = 0.f;
@@ -295,9 +332,12 @@ __global__ void __launch_bounds__(256) mem_out_kernel(MatMem M, int q_col, int k
             const int sd = i >> 6, sv = i & 63;
             Ss[sd][sv] = k0 + sd < M.dim && v0 + sv < M.vdim ? U[(size_t)(k0 + sd) * M.vdim + v0 + sv] : 0.f;
         }
+        if (threadIdx.x < 32) ns[threadIdx.x] = k0 + threadIdx.x < M.dim ? nU[k0 + threadIdx.x] : 0.f;
         __syncthreads();
-        if (threadIdx.x < kMemChunk)
-            for (int d = 0; d < 32 && k0 + d < M.dim; d++) nq = fmaf(nU[k0 + d], Qs[d][threadIdx.x], nq);
+        if (threadIdx.x < kMemChunk) {
+#pragma unroll 8
+            for (int d = 0; d < 32; d++) nq = fmaf(ns[d], Qs[d][threadIdx.x], nq);
+        }
 #pragma unroll 8
         for (int d = 0; d < 32; d++) {
             const float4 a = *reinterpret_cast<const float4*>(&Qs[d][ty * 4]), b = *reinterpret_cast<const float4*>(&Ks[d][tx * 4]),
@@ -447,7 +487,7 @@ cudaError_t launch_last_norm_rows(const float* x, const int* rows, const float* 
 cudaError_t launch_mem_rows(const MatMem& mem, const ProjCols& c, const float* proj, int ldp, int pos0, int n, const MemRows& w, void* act,
                             int ld_act, bool f32, cudaStream_t s) {
     const int chunks = (n + kMemChunk - 1) / kMemChunk, dt = (mem.dim + 63) / 64, vt = (mem.vdim + 63) / 64;
-    mem_gates_kernel<<<mem.heads, 32, 0, s>>>(mem, c.mi, c.mf, proj, ldp, pos0, n, w);
+    mem_gates_kernel<<<mem.heads, kGateWarps * 32, 0, s>>>(mem, c.mi, c.mf, proj, ldp, pos0, n, w);
     mem_chunk_kernel<<<dim3(chunks, mem.heads, dt * vt), 256, 0, s>>>(mem, c.mk, c.mv, proj, ldp, n, vt, w);
     const size_t elems = (size_t)mem.heads * mem.dim * (mem.vdim + 1);
     mem_scan_kernel<<<(unsigned)((elems + 255) / 256), 256, 0, s>>>(mem, pos0, n, chunks, w);
