@@ -2,8 +2,12 @@
 //
 // Mixing couples every head at every (query, key) pair, so a CTA owns a tile of 128 queries x BN keys for
 // ALL heads: each head's scores land in their own TMEM columns (heads x BN <= 512), then a thread reads
-// one query row's scores of all heads for four keys at a time, forms the sigmoids and the mixed weights
-// in fp32 registers (packed fma.rn.f32x2), and writes them as bf16.  The product with the raw keys is a
+// one query row's scores of all heads for four keys at a time, forms the sigmoids in fp32, and the mixed
+// weights are written as bf16.  Up to 8 heads are mixed in registers (packed fma.rn.f32x2).  With more
+// heads the mixing is a small product per key, mix[h][query] = sum_g T[h][g] w[g][query]: T is bf16 as
+// stored, and the fp32 weights go in as two bf16 parts, high and low (16 bits of mantissa together), in
+// two rounds of mma.sync over the same accumulator; their operand layout is what the TMEM rows give
+// after one pass through shared memory.  The product with the raw keys is a
 // batched gemm_tc over heads (its causal bound skips the zero part), against keys transposed once per
 // call.  Queries go in blocks, so that the weights of a block stay within the workspace.
 #include <algorithm>
@@ -16,7 +20,6 @@ namespace mg {
 
 namespace {
 
-constexpr int kStages = 4;
 constexpr int kThreads = 320;       // TMA warp, MMA warp, 8 epilogue warps
 
 struct ScoreArgs {
@@ -31,12 +34,20 @@ struct ScoreArgs {
 
 template <int HP>
 struct Geo {
+    static constexpr bool tensor_mix = HP >= 16;
     static constexpr int bn = HP <= 8 ? 32 : 16;
     static constexpr int cols = HP * bn < 32 ? 32 : HP * bn;
     static constexpr int per_sm = cols <= 256 ? 2 : 1;
+    static constexpr int stages = HP == 32 ? 8 : HP == 16 ? 5 : 4;
     static constexpr int stage = 128 * 128 + bn * 128;
-    static constexpr int table_floats = 2 * HP * HP + 2 * HP + bn * HP;    // mixing pairs, bias, slope, 1 / rms of the keys
-    static constexpr int bytes = kStages * stage + 1024 + 128 + table_floats * 4;
+    static constexpr int ring = stages * stage;
+    // the epilogue's operand rows take the ring's place: per warp 4 keys x 32 queries x {high, low}
+    static constexpr int point = HP * 2 + 16;               // bytes of a row of bf16 weights, padded against conflicts
+    static constexpr int part = 4 * 32 * point;
+    static constexpr int mix_bytes = tensor_mix ? 8 * 2 * part : 0;
+    static constexpr int body = ring > mix_bytes ? ring : mix_bytes;
+    static constexpr int talk_bytes = tensor_mix ? 0 : 8 * HP * HP;    // mixing pairs {t, t}
+    static constexpr int bytes = body + 1024 + 256 + talk_bytes + (2 * HP + bn * HP) * 4;
 };
 
 __device__ __forceinline__ unsigned long long pack2(float a, float b) {
@@ -50,10 +61,29 @@ __device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigne
 __device__ __forceinline__ float lo(unsigned long long v) { return __uint_as_float((unsigned)v); }
 __device__ __forceinline__ float hi(unsigned long long v) { return __uint_as_float((unsigned)(v >> 32)); }
 
+// 1 / (1 + 2^t)
+__device__ __forceinline__ float sigmoid_of_exp2(float t) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(t));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return r;
+}
+__device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t bf16_pair(float a, float b) {
+    const __nv_bfloat162 p = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&p);
+}
+
 template <int HP>
 __global__ void __launch_bounds__(kThreads, Geo<HP>::per_sm) gate_scores_kernel(const __grid_constant__ ScoreArgs a) {
     using G = Geo<HP>;
-    constexpr int BN = G::bn;
+    constexpr int BN = G::bn, kStages = G::stages;
     const GateAttn& A = a.at;
     const int tile_row = blockIdx.y * 128, j0 = blockIdx.x * BN;
     const int tile_rows = min(128, a.rows - tile_row);
@@ -62,14 +92,14 @@ __global__ void __launch_bounds__(kThreads, Geo<HP>::per_sm) gate_scores_kernel(
 
     extern __shared__ uint8_t raw[];
     uint8_t* base = reinterpret_cast<uint8_t*>(((uintptr_t)raw + 1023) & ~(uintptr_t)1023);
-    uint64_t* full = reinterpret_cast<uint64_t*>(base + kStages * G::stage);
+    uint64_t* full = reinterpret_cast<uint64_t*>(base + G::body);
     uint64_t* empty = full + kStages;
     uint64_t* done = empty + kStages;
     uint32_t* tmem_base = reinterpret_cast<uint32_t*>(done + 1);
-    ulonglong2* talk = reinterpret_cast<ulonglong2*>(base + kStages * G::stage + 128);   // [h][g / 2]: {t, t} of two g
-    float* bias = reinterpret_cast<float*>(talk + HP * HP / 2);
-    float* slope = bias + HP;
-    float* kr = slope + HP;         // [key][head]
+    ulonglong2* talk = reinterpret_cast<ulonglong2*>(base + G::body + 256);     // [h][g / 2]: {t, t} of two g
+    float2* line = reinterpret_cast<float2*>(base + G::body + 256 + G::talk_bytes);  // per head: slope, -bias, in units of log2 e
+    float* kr = reinterpret_cast<float*>(line + HP);                            // [head][key]: -1 / rms of the key, likewise
+    static_assert((2 * kStages + 1) * 8 + 4 <= 256, "barriers fit their place");
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int H = A.heads, group = H / A.kv_heads;
@@ -83,19 +113,20 @@ __global__ void __launch_bounds__(kThreads, Geo<HP>::per_sm) gate_scores_kernel(
         tma_prefetch_map(&a.k);
     }
     if (warp == 1) tmem_alloc(tmem_base, G::cols);
-    for (int i = threadIdx.x; i < HP * HP / 2; i += kThreads) {
-        const int h = i / (HP / 2), g = 2 * (i % (HP / 2));
-        const float t0 = h < H && g < H ? A.talk[h * H + g] : 0.f, t1 = h < H && g + 1 < H ? A.talk[h * H + g + 1] : 0.f;
-        talk[i] = make_ulonglong2(pack2(t0, t0), pack2(t1, t1));
+    constexpr float kLog2e = 1.4426950408889634f;
+    if constexpr (!G::tensor_mix) {
+        for (int i = threadIdx.x; i < HP * HP / 2; i += kThreads) {
+            const int h = i / (HP / 2), g = 2 * (i % (HP / 2));
+            const float t0 = h < H && g < H ? A.talk[h * H + g] : 0.f, t1 = h < H && g + 1 < H ? A.talk[h * H + g + 1] : 0.f;
+            talk[i] = make_ulonglong2(pack2(t0, t0), pack2(t1, t1));
+        }
     }
-    for (int i = threadIdx.x; i < HP; i += kThreads) {
-        bias[i] = i < H ? A.head_bias[i] : 0.f;
-        slope[i] = i < H ? A.slopes[i] : 0.f;
-    }
+    for (int i = threadIdx.x; i < HP; i += kThreads)
+        line[i] = i < H ? make_float2(A.slopes[i] * kLog2e, -A.head_bias[i] * kLog2e) : make_float2(0.f, 0.f);
     const int len = a.pos0 + a.row0 + a.rows;       // keys the block's queries can see
     for (int i = threadIdx.x; i < BN * HP; i += kThreads) {
-        const int p = i / HP, h = i % HP;
-        kr[i] = h < H && j0 + p < len ? A.cache_r[(size_t)(j0 + p) * A.kv_heads + h / group] : 0.f;
+        const int p = i % BN, h = i / BN;
+        kr[i] = h < H && j0 + p < len ? -kLog2e * A.cache_r[(size_t)(j0 + p) * A.kv_heads + h / group] : 0.f;
     }
     tc_fence_before();
     __syncthreads();
@@ -137,51 +168,121 @@ __global__ void __launch_bounds__(kThreads, Geo<HP>::per_sm) gate_scores_kernel(
         const int quarter = warp & 3, half = (warp - 2) >> 2;
         const int row = tile_row + quarter * 32 + lane;
         const int pos = a.pos0 + a.row0 + row;
+        // mixing matrix as MMA operands: rows h, columns g
+        constexpr int MT = HP >= 16 ? HP / 16 : 1;
+        uint32_t ta[MT][MT][4];
+        if constexpr (G::tensor_mix) {
+#pragma unroll
+            for (int m = 0; m < MT; m++)
+#pragma unroll
+                for (int k = 0; k < MT; k++)
+#pragma unroll
+                    for (int r = 0; r < 4; r++) {
+                        const int h = m * 16 + (lane >> 2) + (r & 1) * 8, g = k * 16 + (lane & 3) * 2 + (r >> 1) * 8;
+                        ta[m][k][r] = bf16_pair(h < H && g < H ? A.talk[h * H + g] : 0.f, h < H && g + 1 < H ? A.talk[h * H + g + 1] : 0.f);
+                    }
+        }
+        uint8_t* mine = base + (warp - 2) * 2 * G::part;
         if (ok) {
 #pragma unroll 1
             for (int c = half * (BN / 2); c < (half + 1) * (BN / 2); c += 4) {
-                unsigned long long w[HP][2];
                 constexpr int GB = HP < 8 ? HP : 8;         // heads per round of loads
+                unsigned long long w[G::tensor_mix ? 1 : HP][2];
+                const float dist = (float)(pos - (j0 + c));
 #pragma unroll
                 for (int g0 = 0; g0 < HP; g0 += GB) {
                     uint32_t s[GB][4];
+                    float v[GB][4];
 #pragma unroll
                     for (int g = 0; g < GB; g++)
                         if (g0 + g < H) tmem_load4_async(acc + ((uint32_t)(quarter * 32) << 16) + (g0 + g) * BN + c, s[g]);
                     tmem_wait_load();
 #pragma unroll
                     for (int g = 0; g < GB; g++) {
-                        float v[4] = {0.f, 0.f, 0.f, 0.f};
-                        if (g0 + g < H) {
+                        const float2 ln = line[g0 + g];
+                        const float4 k4 = *reinterpret_cast<const float4*>(kr + (g0 + g) * BN + c);
+                        const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
 #pragma unroll
-                            for (int i = 0; i < 4; i++) {
-                                const int dist = pos - (j0 + c + i);
-                                const float x = __uint_as_float(s[g][i]) * kr[(c + i) * HP + g0 + g] - slope[g0 + g] * (float)dist + bias[g0 + g];
-                                v[i] = dist >= 0 ? __fdividef(1.0f, 1.0f + __expf(-x)) : 0.f;
-                            }
+                        for (int i = 0; i < 4; i++) {
+                            const float t = fmaf(__uint_as_float(s[g][i]), kk[i], fmaf(ln.x, dist - (float)i, ln.y));
+                            v[g][i] = g0 + g < H && dist >= (float)i ? sigmoid_of_exp2(t) : 0.f;
                         }
-                        w[g0 + g][0] = pack2(v[0], v[1]);
-                        w[g0 + g][1] = pack2(v[2], v[3]);
+                    }
+                    if constexpr (G::tensor_mix) {
+                        // eight heads are 16 bytes of a point's row, as bf16 and what bf16 leaves over
+#pragma unroll
+                        for (int i = 0; i < 4; i++) {
+                            uint32_t hi4[4], lo4[4];
+#pragma unroll
+                            for (int g = 0; g < GB; g += 2) {
+                                const uint32_t p = bf16_pair(v[g][i], v[g + 1][i]);
+                                hi4[g / 2] = p;
+                                lo4[g / 2] = bf16_pair(v[g][i] - __uint_as_float(p << 16), v[g + 1][i] - __uint_as_float(p & 0xffff0000u));
+                            }
+                            uint8_t* row_at = mine + (i * 32 + lane) * G::point + g0 * 2;
+                            *reinterpret_cast<uint4*>(row_at) = make_uint4(hi4[0], hi4[1], hi4[2], hi4[3]);
+                            *reinterpret_cast<uint4*>(row_at + G::part) = make_uint4(lo4[0], lo4[1], lo4[2], lo4[3]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int g = 0; g < GB; g++) {
+                            w[g0 + g][0] = pack2(v[g][0], v[g][1]);
+                            w[g0 + g][1] = pack2(v[g][2], v[g][3]);
+                        }
                     }
                 }
-                __nv_bfloat16* out = a.w + (long long)row * a.ldp + j0 + c;
-#pragma unroll 2
-                for (int h = 0; h < H; h++) {
-                    unsigned long long m0 = 0ull, m1 = 0ull;
+                if constexpr (G::tensor_mix) {
+                    __syncwarp();
+#pragma unroll 1
+                    for (int nt = 0; nt < 4; nt++) {            // eight queries at a time
+                        float o[MT][4][4] = {};                 // [h tile][key][accumulator]
 #pragma unroll
-                    for (int g = 0; g < HP; g += 2) {
-                        const ulonglong2 t = talk[h * (HP / 2) + g / 2];
-                        m0 = fma2(t.x, w[g][0], m0);
-                        m1 = fma2(t.x, w[g][1], m1);
-                        m0 = fma2(t.y, w[g + 1][0], m0);
-                        m1 = fma2(t.y, w[g + 1][1], m1);
+                        for (int i = 0; i < 4; i++) {
+                            uint32_t bh[4], bl[4];
+                            if constexpr (MT == 2) {
+                                const uint32_t at = smem_addr(mine) + (i * 32 + nt * 8 + (lane & 7)) * G::point + (lane >> 3) * 16;
+                                ldmatrix4(bh, at);
+                                ldmatrix4(bl, at + G::part);
+                            } else {                            // high columns 0-7, 8-15, then low
+                                uint32_t b4[4];
+                                ldmatrix4(b4, smem_addr(mine) + (i * 32 + nt * 8 + (lane & 7)) * G::point + ((lane >> 3) & 1) * 16 + (lane >> 4) * G::part);
+                                bh[0] = b4[0]; bh[1] = b4[1]; bl[0] = b4[2]; bl[1] = b4[3];
+                            }
+#pragma unroll
+                            for (int m = 0; m < MT; m++)
+#pragma unroll
+                                for (int k = 0; k < MT; k++) {
+                                    mma_16816(o[m][i], ta[m][k], bh[2 * k], bh[2 * k + 1]);
+                                    mma_16816(o[m][i], ta[m][k], bl[2 * k], bl[2 * k + 1]);
+                                }
+                        }
+#pragma unroll
+                        for (int m = 0; m < MT; m++)
+#pragma unroll
+                            for (int r = 0; r < 4; r++) {
+                                const int h = m * 16 + (lane >> 2) + (r >> 1) * 8;
+                                const int q = tile_row + quarter * 32 + nt * 8 + (lane & 3) * 2 + (r & 1);
+                                if (h < H && q < a.rows)
+                                    *reinterpret_cast<uint2*>(a.w + h * a.head_stride + (long long)q * a.ldp + j0 + c) =
+                                        make_uint2(bf16_pair(o[m][0][r], o[m][1][r]), bf16_pair(o[m][2][r], o[m][3][r]));
+                            }
                     }
-                    if (row < a.rows) {
-                        __nv_bfloat162 p0 = __floats2bfloat162_rn(lo(m0), hi(m0)), p1 = __floats2bfloat162_rn(lo(m1), hi(m1));
-                        uint2 v;
-                        v.x = *reinterpret_cast<uint32_t*>(&p0);
-                        v.y = *reinterpret_cast<uint32_t*>(&p1);
-                        *reinterpret_cast<uint2*>(out + h * a.head_stride) = v;
+                    __syncwarp();                               // the rows are free again
+                } else {
+                    __nv_bfloat16* out = a.w + (long long)row * a.ldp + j0 + c;
+#pragma unroll 2
+                    for (int h = 0; h < H; h++) {
+                        unsigned long long m0 = 0ull, m1 = 0ull;
+#pragma unroll
+                        for (int g = 0; g < HP; g += 2) {
+                            const ulonglong2 t = talk[h * (HP / 2) + g / 2];
+                            m0 = fma2(t.x, w[g][0], m0);
+                            m1 = fma2(t.x, w[g][1], m1);
+                            m0 = fma2(t.y, w[g + 1][0], m0);
+                            m1 = fma2(t.y, w[g + 1][1], m1);
+                        }
+                        if (row < a.rows)
+                            *reinterpret_cast<uint2*>(out + h * a.head_stride) = make_uint2(bf16_pair(lo(m0), hi(m0)), bf16_pair(lo(m1), hi(m1)));
                     }
                 }
             }

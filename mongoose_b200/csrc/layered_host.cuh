@@ -23,6 +23,7 @@ struct LayerSlot {
     int rows = 0, cols = 0;             // 0: the slot does not exist
     uint8_t* mat = nullptr;             // bf16 rows padded to pad_to(cols, 64)
     float* vec = nullptr;
+    bool rounds = false;                // a small matrix among the vectors: held as fp32, rounded to bf16
     bool set = false;
 };
 
@@ -166,7 +167,7 @@ void layered_slots(Layered& m) {
         vec(MG_SLOT_NORM1, l.norm1, W);
         mat(MG_SLOT_AT_Q, l.proj, l.cols.q, a.heads * a.dim, W); mat(MG_SLOT_AT_K, l.proj, l.cols.k, a.kv_heads * a.dim, W);
         vec(MG_SLOT_AT_QNORM, l.q_norm, a.dim); vec(MG_SLOT_AT_KNORM, l.k_norm, a.dim);
-        vec(MG_SLOT_AT_TALK, l.talk, a.heads * a.heads); vec(MG_SLOT_AT_BIAS, l.bias, a.heads);
+        vec(MG_SLOT_AT_TALK, l.talk, a.heads * a.heads); s[MG_SLOT_AT_TALK].rounds = true; vec(MG_SLOT_AT_BIAS, l.bias, a.heads);
         mat(MG_SLOT_AT_O, l.at_o, 0, W, l.kat()); vec(MG_SLOT_AT_OUT, l.at_out, W);
         mat(MG_SLOT_MEM_Q, l.proj, l.cols.mq, r.heads * r.dim, W); mat(MG_SLOT_MEM_K, l.proj, l.cols.mk, r.heads * r.dim, W);
         mat(MG_SLOT_MEM_V, l.proj, l.cols.mv, r.heads * r.vdim, W); mat(MG_SLOT_MEM_G, l.proj, l.cols.mg, r.heads * r.vdim, W);
@@ -199,6 +200,8 @@ int layered_set(mg_engine* e, int idx, const void* data, size_t count, bool bf16
             if (bf16) { const uint32_t w = (uint32_t)h[i] << 16; memcpy(&v[i], &w, 4); }
             else v[i] = f[i];
         }
+        if (!bf16 && s.rounds)              // multiplied on the tensor cores: kept as bf16, like every matrix
+            for (float& x : v) x = __bfloat162float(__float2bfloat16_rn(x));
         MG_CUDA(e, cudaMemcpy(s.vec, v.data(), count * 4, cudaMemcpyHostToDevice));
     } else {
         const size_t ld = pad_to(s.cols, 64);
