@@ -111,7 +111,7 @@ __global__ void __launch_bounds__(kAttnThreads) mixer_step_kernel(const MixerSte
     // this token's query, and its key where this CTA's range ends with it
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
     const float temp = query_temp(A, pos);
-    norm_queries(A, a.proj + a.c.q, temp, sm.q);
+    norm_queries(A, a.proj + a.c.q, temp, sm.q, sm.qs);
     if (j1 == len)
         for (int c = wid; c < A.kv_heads; c += nw) store_key<KT>(A, a.proj + a.c.k + c * A.dim, pos, c, lane);
     sm.load_tables(A);

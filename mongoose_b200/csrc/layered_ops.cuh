@@ -60,7 +60,7 @@ __device__ __forceinline__ void norm_query(const GateAttn& A, const float* q, fl
 }
 
 // The same for every head of one token by the whole CTA, eight lanes per head.
-__device__ __forceinline__ void norm_queries(const GateAttn& A, const float* q, float temp, float* out) {
+__device__ __forceinline__ void norm_queries(const GateAttn& A, const float* q, float temp, float* out, int qs) {
     const int sub = threadIdx.x & 7;
     const unsigned mask = 0xffu << (threadIdx.x & 24);
     for (int h = threadIdx.x >> 3; h < A.heads; h += kAttnThreads / 8) {
@@ -80,9 +80,9 @@ __device__ __forceinline__ void norm_queries(const GateAttn& A, const float* q, 
 #pragma unroll
         for (int i = 0; i < 16; i++) {
             const int d = sub + 8 * i;
-            if (d < A.dim_s) out[h * A.dim_s + d] = d < A.dim ? v[i] * r * A.q_norm[d] * A.k_norm[d] : 0.f;
+            if (d < A.dim_s) out[h * qs + d] = d < A.dim ? v[i] * r * A.q_norm[d] * A.k_norm[d] : 0.f;
         }
-        for (int d = sub + 128; d < A.dim_s; d += 8) out[h * A.dim_s + d] = d < A.dim ? p[d] * r * A.q_norm[d] * A.k_norm[d] : 0.f;
+        for (int d = sub + 128; d < A.dim_s; d += 8) out[h * qs + d] = d < A.dim ? p[d] * r * A.q_norm[d] * A.k_norm[d] : 0.f;
     }
 }
 
@@ -113,32 +113,41 @@ __host__ __device__ inline int key_split(int len, int splits, int tile, int spli
 
 // Accumulator pairs per thread (rounded up to an instance), 0 when the heads do not fit.
 inline int attn_pairs(const GateAttn& at) {
+    if (at.dim_s > 1024) return 0;          // KeyCopy: a key row is at most one piece per thread
     const int pairs = (at.heads * at.dim_s / 2 + kAttnThreads - 1) / kAttnThreads;
     for (int p = 1; p <= 16; p *= 2)
         if (pairs <= p) return p;
     return 0;
 }
 
+// Rows in shared memory are 16 bytes longer than their data (mixed-head rows one float), so that lanes that
+// walk different rows meet different banks.
 template <typename KT>
 struct AttnSmem {
-    KT* k;          // [2][tile][kv_heads * dim_s]
+    KT* k;          // [2][tile][kv_heads][ks]
     float* r;       // [2][tile][kv_heads]
-    float* q;       // [nq][heads][dim_s]
-    float* w;       // [nq][heads][tile] sigmoid weights
-    float* mix;     // [nq][heads][tile] mixed over heads
+    float* q;       // [nq][heads][qs]
+    float* w;       // [nq][heads][ws] sigmoid weights
+    float* mix;     // [nq][heads][ws] mixed over heads
     float *talk, *bias, *slope;
+    int ks, qs, ws, ts;
     __device__ __forceinline__ AttnSmem(const GateAttn& A, int nq, int tile, float* base) {
+        ks = A.dim_s + 16 / (int)sizeof(KT);
+        qs = A.dim_s + 4;
+        ws = tile + 1;
+        ts = A.heads + 1;
         k = reinterpret_cast<KT*>(base);
-        r = reinterpret_cast<float*>(k + 2 * (size_t)tile * A.kv_heads * A.dim_s);
+        r = reinterpret_cast<float*>(k + 2 * (size_t)tile * A.kv_heads * ks);
         q = r + pad_to(2 * tile * A.kv_heads, 4);
-        w = q + nq * A.heads * A.dim_s;
-        mix = w + nq * A.heads * tile;
-        talk = mix + nq * A.heads * tile;
-        bias = talk + A.heads * A.heads;
+        w = q + nq * A.heads * qs;
+        mix = w + nq * A.heads * ws;
+        talk = mix + nq * A.heads * ws;
+        bias = talk + A.heads * ts;
         slope = bias + A.heads;
     }
     __device__ __forceinline__ void load_tables(const GateAttn& A) const {
-        for (int i = threadIdx.x; i < A.heads * A.heads; i += kAttnThreads) talk[i] = A.talk[i];
+        for (int h = threadIdx.x / 32; h < A.heads; h += kAttnThreads / 32)
+            for (int g = threadIdx.x % 32; g < A.heads; g += 32) talk[h * ts + g] = A.talk[h * A.heads + g];
         for (int i = threadIdx.x; i < A.heads; i += kAttnThreads) { bias[i] = A.head_bias[i]; slope[i] = A.slopes[i]; }
     }
 };
@@ -147,9 +156,9 @@ struct AttnSmem {
 inline size_t attn_smem(const GateAttn& at, int nq, int kt_bytes, int most, int* tile) {
     if (!attn_pairs(at)) return 0;
     for (int t = most; t >= 8; t /= 2) {
-        const size_t b = 2 * (size_t)t * at.kv_heads * at.dim_s * kt_bytes +
-                         ((size_t)pad_to(2 * t * at.kv_heads, 4) + (size_t)nq * at.heads * (at.dim_s + 2 * t) +
-                          (size_t)at.heads * at.heads + 2 * at.heads) * sizeof(float);
+        const size_t b = 2 * (size_t)t * at.kv_heads * (at.dim_s * kt_bytes + 16) +
+                         ((size_t)pad_to(2 * t * at.kv_heads, 4) + (size_t)nq * at.heads * (at.dim_s + 4 + 2 * (t + 1)) +
+                          (size_t)at.heads * (at.heads + 1) + 2 * at.heads) * sizeof(float);
         if (b <= 200 * 1024) { *tile = t; return b; }
     }
     return 0;
@@ -162,96 +171,106 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-template <typename KT>
-__device__ __forceinline__ void load_keys(const GateAttn& A, const AttnSmem<KT>& sm, int buf, int j, int j1, int tile) {
-    const int row = A.kv_heads * A.dim_s, per = row * (int)sizeof(KT) / 16;
-    KT* dst = sm.k + (size_t)buf * tile * row;
-    const KT* src = static_cast<const KT*>(A.cache) + (size_t)j * row;
-    const int valid = (j1 - j < tile ? j1 - j : tile) * per;
-    for (int i = threadIdx.x; i < tile * per; i += kAttnThreads) {
-        void* d = reinterpret_cast<uint4*>(dst) + i;
-        if (i < valid) cp_async16(d, reinterpret_cast<const uint4*>(src) + i);
-        else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+__device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+
+// Which 16-byte pieces of a tile this thread copies: piece `ch` of rows row0, row0 + step, ...
+struct KeyCopy {
+    int ch, row0, step;
+    __device__ __forceinline__ KeyCopy(int pieces) {
+        step = kAttnThreads / pieces;
+        row0 = threadIdx.x / pieces;
+        ch = threadIdx.x - row0 * pieces;
+        if (row0 >= step) row0 = 1 << 30;       // no whole row left for these threads
     }
-    for (int i = threadIdx.x; i < tile * A.kv_heads; i += kAttnThreads)
-        sm.r[buf * tile * A.kv_heads + i] = j + i / A.kv_heads < j1 ? A.cache_r[(size_t)j * A.kv_heads + i] : 0.f;
+};
+
+template <typename KT>
+__device__ __forceinline__ void load_keys(const GateAttn& A, const AttnSmem<KT>& sm, const KeyCopy& cp, int buf, int j, int j1, int tile) {
+    constexpr int CN = Chunk16<KT>::n;
+    const int rows = tile * A.kv_heads, valid = min(rows, (j1 - j) * A.kv_heads);
+    KT* dst = sm.k + (size_t)buf * rows * sm.ks + cp.ch * CN;
+    const KT* src = static_cast<const KT*>(A.cache) + (size_t)j * A.kv_heads * A.dim_s + cp.ch * CN;
+    for (int r = cp.row0; r < rows; r += cp.step) {
+        if (r < valid) cp_async16(dst + r * sm.ks, src + (size_t)r * A.dim_s);
+        else *reinterpret_cast<uint4*>(dst + r * sm.ks) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    for (int i = threadIdx.x; i < valid; i += kAttnThreads) cp_async4(sm.r + buf * rows + i, A.cache_r + (size_t)j * A.kv_heads + i);
 }
 
 // acc[q][pair] += sum over keys [j0, j1) of the mixed weights times the raw keys, for the NQ queries in
 // sm.q at positions pos0 .. pos0 + NQ - 1.  Thread t owns elements 2 * (t + p * kAttnThreads) and the next of the
-// [heads][dim_s] output.
+// [heads][dim_s] output.  A score belongs to one thread, lanes over heads.
 template <typename KT, int NQ, int EP>
 __device__ __forceinline__ void attend(const GateAttn& A, const AttnSmem<KT>& sm, int pos0, int j0, int j1, int tile,
                                        float (&acc)[NQ][EP][2]) {
     constexpr int CN = Chunk16<KT>::n;
-    const int H = A.heads, DS = A.dim_s, row = A.kv_heads * DS, group = H / A.kv_heads;
-    const int sub = threadIdx.x & 7, gid = threadIdx.x >> 3;
+    const int H = A.heads, DS = A.dim_s, KV = A.kv_heads, group = H / KV, row = KV * sm.ks;
     const int chunks = DS / CN;
-    const int ts = 31 - __clz(tile);                // tiles are powers of two
+    const int tsh = 31 - __clz(tile);               // tiles are powers of two
+    const KeyCopy cp(chunks);
     int head_of[EP], key_of[EP];                    // this thread's output elements
 #pragma unroll
     for (int e = 0; e < EP; e++) {
         const int el = 2 * (threadIdx.x + e * kAttnThreads);
         const int h = el / DS;
         head_of[e] = el < H * DS ? h : -1;
-        key_of[e] = h / group * DS + el - h * DS;
+        key_of[e] = h / group * sm.ks + el - h * DS;
     }
-    load_keys<KT>(A, sm, 0, j0, j1, tile);
+    load_keys<KT>(A, sm, cp, 0, j0, j1, tile);
     cp_async_commit();
     int buf = 0;
     for (int j = j0; j < j1; j += tile, buf ^= 1) {
-        if (j + tile < j1) load_keys<KT>(A, sm, buf ^ 1, j + tile, j1, tile);
+        if (j + tile < j1) load_keys<KT>(A, sm, cp, buf ^ 1, j + tile, j1, tile);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
         const KT* K = sm.k + (size_t)buf * tile * row;
-        const float* R = sm.r + buf * tile * A.kv_heads;
-        for (int u = gid; u < H * tile; u += kAttnThreads / 8) {
-            const int h = u >> ts, p = u & (tile - 1), c = h / group;
-            const KT* kp = K + (size_t)p * row + c * DS;
-            float dot[NQ] = {};
-            for (int ch = sub; ch < chunks; ch += 8) {
+        const float* R = sm.r + buf * tile * KV;
+        const int keys = min(tile, j1 - j);
+        for (int u = threadIdx.x; u < H * tile; u += kAttnThreads) {
+            const int p = u / H, h = u - p * H, c = h / group;
+            const KT* kp = K + p * row + c * sm.ks;
+            const float* qp = sm.q + h * sm.qs;
+            float dot[NQ][2] = {};
+#pragma unroll 2
+            for (int ch = 0; ch < chunks; ch++) {
                 float kk[CN];
                 Chunk16<KT>::load(kp + ch * CN, kk);
 #pragma unroll
-                for (int q = 0; q < NQ; q++) {
-                    const float* qp = sm.q + (q * H + h) * DS + ch * CN;
+                for (int q = 0; q < NQ; q++)
 #pragma unroll
                     for (int i = 0; i < CN; i += 4) {
-                        const float4 v = *reinterpret_cast<const float4*>(qp + i);
-                        dot[q] = fmaf(kk[i], v.x, fmaf(kk[i + 1], v.y, fmaf(kk[i + 2], v.z, fmaf(kk[i + 3], v.w, dot[q]))));
+                        const float4 v = *reinterpret_cast<const float4*>(qp + q * H * sm.qs + ch * CN + i);
+                        dot[q][0] = fmaf(kk[i], v.x, dot[q][0]);
+                        dot[q][1] = fmaf(kk[i + 1], v.y, dot[q][1]);
+                        dot[q][0] = fmaf(kk[i + 2], v.z, dot[q][0]);
+                        dot[q][1] = fmaf(kk[i + 3], v.w, dot[q][1]);
                     }
-                }
             }
-            float mine = 0.f;
+            const float r = p < keys ? R[p * KV + c] : 0.f;
 #pragma unroll
             for (int q = 0; q < NQ; q++) {
-                float d = dot[q];
-                d += __shfl_xor_sync(0xffu << (threadIdx.x & 24), d, 1);
-                d += __shfl_xor_sync(0xffu << (threadIdx.x & 24), d, 2);
-                d += __shfl_xor_sync(0xffu << (threadIdx.x & 24), d, 4);
-                if (sub == q) mine = d;
-            }
-            if (sub < NQ) {
-                const int dist = pos0 + sub - (j + p);
-                const float s = mine * R[p * A.kv_heads + c] - sm.slope[h] * (float)dist + sm.bias[h];
-                sm.w[(sub * H + h) * tile + p] = dist >= 0 && j + p < j1 ? sigmoid(s) : 0.f;
+                const int dist = pos0 + q - (j + p);
+                const float s = (dot[q][0] + dot[q][1]) * r - sm.slope[h] * (float)dist + sm.bias[h];
+                sm.w[(q * H + h) * sm.ws + p] = dist >= 0 && p < keys ? sigmoid(s) : 0.f;
             }
         }
         __syncthreads();
         for (int u = threadIdx.x; u < NQ * H * tile; u += kAttnThreads) {
-            const int p = u & (tile - 1), qh = u >> ts, h = NQ == 1 ? qh : qh % H;
-            const float* wq = sm.w + (qh - h) * tile + p;
-            const float* t = sm.talk + h * H;
+            const int p = u & (tile - 1), qh = u >> tsh, h = NQ == 1 ? qh : qh % H;
+            const float* wq = sm.w + (qh - h) * sm.ws + p;
+            const float* t = sm.talk + h * sm.ts;
             float v0 = 0.f, v1 = 0.f;
             int g = 0;
-#pragma unroll 4
+#pragma unroll 8
             for (; g + 1 < H; g += 2) {
-                v0 = fmaf(t[g], wq[g * tile], v0);
-                v1 = fmaf(t[g + 1], wq[(g + 1) * tile], v1);
+                v0 = fmaf(t[g], wq[g * sm.ws], v0);
+                v1 = fmaf(t[g + 1], wq[(g + 1) * sm.ws], v1);
             }
-            if (g < H) v0 = fmaf(t[g], wq[g * tile], v0);
-            sm.mix[u] = v0 + v1;
+            if (g < H) v0 = fmaf(t[g], wq[g * sm.ws], v0);
+            sm.mix[qh * sm.ws + p] = v0 + v1;
         }
         __syncthreads();
 #pragma unroll
@@ -260,10 +279,10 @@ __device__ __forceinline__ void attend(const GateAttn& A, const AttnSmem<KT>& sm
             if (h >= 0) {
 #pragma unroll 8
                 for (int p = 0; p < tile; p++) {
-                    const float2 kv = pair_f32(K + (size_t)p * row + off);
+                    const float2 kv = pair_f32(K + p * row + off);
 #pragma unroll
                     for (int q = 0; q < NQ; q++) {
-                        const float m = sm.mix[(q * H + h) * tile + p];
+                        const float m = sm.mix[(q * H + h) * sm.ws + p];
                         acc[q][e][0] = fmaf(m, kv.x, acc[q][e][0]);
                         acc[q][e][1] = fmaf(m, kv.y, acc[q][e][1]);
                     }

@@ -80,7 +80,8 @@ __global__ void __launch_bounds__(kAttnThreads) gate_attn_rows_kernel(GateAttn A
     const AttnSmem<KT> sm(A, NQ, tile, smem);
     const int t0 = (gridDim.x - 1 - blockIdx.x) * NQ;      // the longest rows first
     const int row = A.heads * A.dim_s;
-    for (int i = threadIdx.x; i < NQ * row; i += kAttnThreads) sm.q[i] = t0 + i / row < n ? to_f32(qh[(size_t)t0 * row + i]) : 0.f;
+    for (int i = threadIdx.x; i < NQ * row; i += kAttnThreads)
+        sm.q[i / A.dim_s * sm.qs + i % A.dim_s] = t0 + i / row < n ? to_f32(qh[(size_t)t0 * row + i]) : 0.f;
     sm.load_tables(A);
     __syncthreads();
     const int last = min(t0 + NQ, n) - 1;
