@@ -163,11 +163,6 @@ __global__ void __launch_bounds__(kThreads, Geo<HP>::per_sm) gate_scores_kernel(
         }
         __syncwarp();
     } else {
-        const bool ok = __all_sync(0xffffffffu, bar_wait(done, 0, a.status));
-        tc_fence_after();
-        const int quarter = warp & 3, half = (warp - 2) >> 2;
-        const int row = tile_row + quarter * 32 + lane;
-        const int pos = a.pos0 + a.row0 + row;
         // mixing matrix as MMA operands: rows h, columns g
         constexpr int MT = HP >= 16 ? HP / 16 : 1;
         uint32_t ta[MT][MT][4];
@@ -182,6 +177,11 @@ __global__ void __launch_bounds__(kThreads, Geo<HP>::per_sm) gate_scores_kernel(
                         ta[m][k][r] = bf16_pair(h < H && g < H ? A.talk[h * H + g] : 0.f, h < H && g + 1 < H ? A.talk[h * H + g + 1] : 0.f);
                     }
         }
+        const bool ok = __all_sync(0xffffffffu, bar_wait(done, 0, a.status));
+        tc_fence_after();
+        const int quarter = warp & 3, half = (warp - 2) >> 2;
+        const int row = tile_row + quarter * 32 + lane;
+        const int pos = a.pos0 + a.row0 + row;
         uint8_t* mine = base + (warp - 2) * 2 * G::part;
         if (ok) {
 #pragma unroll 1
