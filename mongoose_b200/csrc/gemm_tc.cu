@@ -97,16 +97,30 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
 #pragma unroll
                 for (int i = 0; i < 32; i++) tile[lane * 33 + i] = v[i];
                 __syncwarp();
-                const int col = col0 + c + lane;
+                if (g.mode == GEMM_F32) {
+                    const int col = col0 + c + lane;
+                    float* out = static_cast<float*>(g.out) + z * g.batch_c + col;
+#pragma unroll 8
+                    for (int r = 0; r < 32; r++) {
+                        const int row = row0 + quarter * 32 + r;
+                        if (row < g.m && col < g.n) out[row * g.ldc] = tile[r * 33 + lane];
+                    }
+                } else {                            // two columns per lane, two rows at a time
+                    const int col = col0 + c + 2 * (lane & 15);
+                    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(g.out) + z * g.batch_c + col;
+                    const bool pair = (reinterpret_cast<uintptr_t>(out) & 3) == 0 && (g.ldc & 1) == 0 && col + 1 < g.n;
 #pragma unroll 4
-                for (int r = 0; r < 32; r++) {
-                    const int row = row0 + quarter * 32 + r;
-                    if (row >= g.m) break;
-                    if (col < g.n) {
-                        const float x = tile[r * 33 + lane];
-                        const long long o = z * g.batch_c + row * g.ldc + col;
-                        if (g.mode == GEMM_F32) static_cast<float*>(g.out)[o] = x;
-                        else static_cast<__nv_bfloat16*>(g.out)[o] = __float2bfloat16_rn(g.mode == GEMM_GELU_BF16 ? gelu_tanh_fast(x) : x);
+                    for (int r = lane >> 4; r < 32; r += 2) {
+                        const int row = row0 + quarter * 32 + r;
+                        float x = tile[r * 33 + 2 * (lane & 15)], y = tile[r * 33 + 2 * (lane & 15) + 1];
+                        if (g.mode == GEMM_GELU_BF16) { x = gelu_tanh_fast(x); y = gelu_tanh_fast(y); }
+                        if (row >= g.m) break;
+                        if (pair) {
+                            *reinterpret_cast<__nv_bfloat162*>(out + row * g.ldc) = __floats2bfloat162_rn(x, y);
+                        } else {
+                            if (col < g.n) out[row * g.ldc] = __float2bfloat16_rn(x);
+                            if (col + 1 < g.n) out[row * g.ldc + 1] = __float2bfloat16_rn(y);
+                        }
                     }
                 }
                 __syncwarp();

@@ -199,6 +199,24 @@ def test_sequences_that_reuse_the_cache(load, dtype):
         agree(portions(e, toks, [1, 5]), ref, dtype)
 
 
+def test_prompts_longer_than_a_block_of_rows(load):
+    """One call that the engine cuts into blocks of rows, and attention into blocks of queries, equals
+    portions that need no cutting, in 32-bit and (within its rounding) in bf16."""
+    cfg = U.config(64, 90, 1e-5, [U.layer(32, 8, 8, 0.35, 0.3, 300, 2, 16, 24, 8.0, 48)])
+    w = U.weights(cfg, seed=41)
+    n = 2175
+    toks = U.tokens(cfg, n)
+    places = [0, 700, 1919, 1920, 1921, 2046, 2047, 2048, 2049, 2100, n - 1]
+    e = load(cfg, w, max_seq=n)
+    parts = portions(e, toks, [640])[places]
+    assert U.rel(e.Forward(toks, 0, places), parts).max() < TOL["float32"]
+    b = load(cfg, w, "bfloat16", max_seq=n)
+    agree(b.Forward(toks, 0, places), parts, "bfloat16")
+    short = 300                                     # the oracle on what it can do quickly
+    assert U.rel(parts[:1], U.want(cfg, w, toks[:short])[places[:1]]).max() < TOL["float32"]
+    agree(portions(b, toks[:short], [short]), U.want(cfg, w, toks[:short]), "bfloat16")
+
+
 def test_long_decoding(load):
     cfg = U.CONFIGS["mixed"]
     w = U.weights(cfg, seed=19)
