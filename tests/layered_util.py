@@ -37,6 +37,7 @@ CONFIGS = {
     "many_heads": config(72, 70, 1e-3, [layer(20, 20, 12, 0.5, 0.4, 33, 2, 130, 70, 12.0, 65),
                                         layer(16, 4, 72, 0.1, 0.2, 5, 5, 16, 16, 12.0, 200)]),
     "beyond_tc": config(96, 83, 1e-5, [layer(40, 8, 8, 0.4, 0.5, 20, 2, 64, 64, 8.0, 96)]),
+    "odd": config(75, 53, 1e-5, [layer(3, 1, 15, 0.3, 0.7, 11, 3, 9, 33, 4.0, 101), layer(5, 5, 7, 0.6, 0.2, 3, 1, 65, 5, 4.0, 0)]),
     "pairs": config(64, 50, 1e-5, [layer(2, 2, 136, 0.08, 0.5, 9, 2, 40, 24, 6.0, 48)]),
 }
 
