@@ -152,10 +152,10 @@ struct AttnSmem {
     }
 };
 
-// Bytes of AttnSmem with the largest tile of at most `most` (32, 16 or 8) keys that fits; 0 when none does.
+// Bytes of AttnSmem with the largest tile of at most `most` keys (a power of two) that fits; 0 when none does.
 inline size_t attn_smem(const GateAttn& at, int nq, int kt_bytes, int most, int* tile) {
     if (!attn_pairs(at)) return 0;
-    for (int t = most; t >= 8; t /= 2) {
+    for (int t = most; t >= 2; t /= 2) {
         const size_t b = 2 * (size_t)t * at.kv_heads * (at.dim_s * kt_bytes + 16) +
                          ((size_t)pad_to(2 * t * at.kv_heads, 4) + (size_t)nq * at.heads * (at.dim_s + 4 + 2 * (t + 1)) +
                           (size_t)at.heads * (at.heads + 1) + 2 * at.heads) * sizeof(float);

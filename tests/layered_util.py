@@ -38,6 +38,7 @@ CONFIGS = {
                                         layer(16, 4, 72, 0.1, 0.2, 5, 5, 16, 16, 12.0, 200)]),
     "beyond_tc": config(96, 83, 1e-5, [layer(40, 8, 8, 0.4, 0.5, 20, 2, 64, 64, 8.0, 96)]),
     "odd": config(75, 53, 1e-5, [layer(3, 1, 15, 0.3, 0.7, 11, 3, 9, 33, 4.0, 101), layer(5, 5, 7, 0.6, 0.2, 3, 1, 65, 5, 4.0, 0)]),
+    "wide_keys": config(64, 40, 1e-5, [layer(16, 16, 256, 0.06, 0.4, 17, 1, 12, 12, 6.0, 32)]),
     "pairs": config(64, 50, 1e-5, [layer(2, 2, 136, 0.08, 0.5, 9, 2, 40, 24, 6.0, 48)]),
 }
 
