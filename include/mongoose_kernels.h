@@ -323,16 +323,37 @@ MG_API const float* mg_l3_hidden(mg_engine* e);
  * mg_partial_step, mg_graph_launch, ...) and keeps its sequence state - cached keys and recurrent state -
  * in the same arena.  Portions of a prompt go through mg_forward.  No counterpart in the reference.
  *
- * A layer: x += norm(mixer(x)); x += norm(ff(x)), norms with their weights stored around zero.  The mixer
+ * Two kinds of layers.  With MG_MIXER_PARALLEL: x += norm(mixer(x)); x += norm(ff(x)), root-mean-square norms
+ * with their weights stored around zero, a gelu feed-forward.  With the other mixers:
+ * x += mult * ls1 * mixer(norm1(x)); x += mult * ls2 * ff(norm2(x)), the norms of the kind mg_model_config names
+ * with plain weights, ls1 and ls2 vectors, ff a mixture of experts.
+ *
  * MG_MIXER_PARALLEL runs two branches on the same input and takes half the sum of their normed outputs:
  *   attention - grouped query heads, per-head query and key norms, query temperature
  *     1 + temp_coef * ln(floor((p + 1) / temp_every) + 1), score * scale minus slope_h * distance with
  *     slope_h = 2^(-8 (h + 1) / heads), weights sigmoid(score + bias_h) not normalised over keys and mixed
  *     over heads by a matrix, values = raw keys;
- *   matrix memory - per head a [dim][vdim] state with exponential gates (caps gate_cap), 32-bit. */
+ *   matrix memory - per head a [dim][vdim] state with exponential gates (caps gate_cap), 32-bit.
+ * MG_MIXER_LATENT is softmax attention whose queries, keys and values come out of low-rank latents (root-mean-
+ *   square norms with plain weights on both); each head's key is an unrotated part and a rotated part that
+ *   all heads share.  Only the key/value latent and the rotated part are cached.
+ * MG_MIXER_WKV is a linear recurrence: every projection reads its own mix of a token's vector and the one
+ *   before it; per head S <- diag(w) S + k v^T with a data-dependent decay w per key channel and a bonus for
+ *   the current token, 32-bit; unit rms per head, a weight, a silu gate.
+ * The mixture of experts sends every token through the `top` of `experts` gated feed-forwards with the largest
+ *   router logits (weights: their softmax) and, where shared_ff > 0, through a shared one times a sigmoid gate.
+ *
+ * Layers may loop: layers loop_start .. loop_stop - 1 run loop_times times in a row with the same weights, each
+ * pass with its own cache and state; before each pass x <- W_in [x; embedding].  Layer indices of the stepping
+ * calls (mg_partial_step and the like) count every run of a layer; weight slots count layers. */
 enum { MG_MATH_BF16 = 0,      /* matrix products and activations of prompts in bf16, fp32 accumulation */
        MG_MATH_F32 = 1 };     /* everything in 32-bit */
-enum { MG_MIXER_PARALLEL = 0 };
+enum { MG_MIXER_PARALLEL = 0, MG_MIXER_LATENT = 1, MG_MIXER_WKV = 2 };
+enum { MG_NORM_RMS_AROUND_ZERO = 0,   /* x / rms(x) * (1 + w) */
+       MG_NORM_LAYER = 1,             /* (x - mean) / sqrt(variance + eps) * w */
+       MG_NORM_RMS = 2 };             /* x / rms(x) * w */
+enum { MG_POS_SINUSOID = 0,           /* a sinusoidal vector is added to the embedding */
+       MG_POS_NONE = 1 };
 typedef struct mg_gate_attn_config {
     int heads, kv_heads, dim;
     float scale, temp_coef;
@@ -342,21 +363,42 @@ typedef struct mg_mat_mem_config {
     int heads, dim, vdim;
     float gate_cap;
 } mg_mat_mem_config;
+typedef struct mg_latent_attn_config {
+    int heads, dim, rot_dim, vdim;    /* per head: unrotated and rotated query/key dimensions, value size */
+    int q_rank, kv_rank;
+    float scale;
+    double rot_base;
+} mg_latent_attn_config;
+typedef struct mg_wkv_config {
+    int heads, dim, decay_rank;
+} mg_wkv_config;
+typedef struct mg_moe_config {
+    int experts, top, ff;             /* experts = 0: the layer has none */
+    int shared_ff;                    /* 0: no shared expert */
+} mg_moe_config;
 typedef struct mg_layer_config {
     int mixer;                /* MG_MIXER_* */
     mg_gate_attn_config attn;
     mg_mat_mem_config mem;
-    int ffn_dim;              /* inner width of the gelu feed-forward; 0 = the layer has none */
+    int ffn_dim;              /* inner width of the gelu feed-forward (MG_MIXER_PARALLEL); 0 = the layer has none */
+    mg_latent_attn_config latent;
+    mg_wkv_config wkv;
+    mg_moe_config moe;        /* feed-forward of the other mixers */
 } mg_layer_config;
 typedef struct mg_model_config {
     int width, vocab, n_layers, max_seq;
     float norm_eps;
     int math;                 /* MG_MATH_* */
     int device;
+    int norm;                 /* MG_NORM_* of the last norm and of pre-normed layers */
+    int positions;            /* MG_POS_* */
+    float residual_mult;
+    int loop_start, loop_stop, loop_times;    /* loop_times = 0: no loop */
 } mg_model_config;
 /* Weight slots of a layer-described model: index layer * MG_LAYER_SLOTS + slot; after the layers
- * n_layers * MG_LAYER_SLOTS + {0 embedding, 1 final norm (around zero), 2 output head}.  Matrices are
- * [out][in]; mg_set_weight takes fp32 (stored as bf16), mg_set_weight_raw takes bf16 for any slot. */
+ * n_layers * MG_LAYER_SLOTS + {0 embedding, 1 final norm, 2 output head, 3 loop input [width][2 width]}.
+ * Matrices are [out][in], those of the experts stacked one below the other; mg_set_weight takes fp32 (stored
+ * as bf16), mg_set_weight_raw takes bf16 for any slot. */
 enum {
     MG_SLOT_NORM1 = 0, MG_SLOT_NORM2 = 1,
     MG_SLOT_AT_Q = 2, MG_SLOT_AT_K = 3, MG_SLOT_AT_QNORM = 4, MG_SLOT_AT_KNORM = 5, MG_SLOT_AT_TALK = 6, MG_SLOT_AT_BIAS = 7,
@@ -364,7 +406,15 @@ enum {
     MG_SLOT_MEM_Q = 10, MG_SLOT_MEM_K = 11, MG_SLOT_MEM_V = 12, MG_SLOT_MEM_G = 13, MG_SLOT_MEM_O = 14, MG_SLOT_MEM_NORM = 15,
     MG_SLOT_MEM_I = 16, MG_SLOT_MEM_IB = 17, MG_SLOT_MEM_F = 18, MG_SLOT_MEM_FB = 19, MG_SLOT_MEM_OUT = 20,
     MG_SLOT_UP = 21, MG_SLOT_DOWN = 22,
-    MG_LAYER_SLOTS = 32
+    MG_SLOT_LS1 = 23, MG_SLOT_LS2 = 24,
+    MG_SLOT_LA_DQ = 25, MG_SLOT_LA_DQNORM = 26, MG_SLOT_LA_UQ = 27, MG_SLOT_LA_DKV = 28, MG_SLOT_LA_DKVNORM = 29, MG_SLOT_LA_UK = 30,
+    MG_SLOT_LA_UV = 31, MG_SLOT_LA_O = 32,
+    MG_SLOT_WKV_MU = 33,      /* 33..37: mixes of r, k, v, g, w */
+    MG_SLOT_WKV_R = 38, MG_SLOT_WKV_K = 39, MG_SLOT_WKV_V = 40, MG_SLOT_WKV_G = 41, MG_SLOT_WKV_W1 = 42, MG_SLOT_WKV_W2 = 43,
+    MG_SLOT_WKV_W0 = 44, MG_SLOT_WKV_U = 45, MG_SLOT_WKV_NORM = 46, MG_SLOT_WKV_O = 47,
+    MG_SLOT_MOE_ROUTER = 48, MG_SLOT_MOE_BIAS = 49, MG_SLOT_MOE_GATE = 50, MG_SLOT_MOE_UP = 51, MG_SLOT_MOE_DOWN = 52,
+    MG_SLOT_SHARED_GATE = 53, MG_SLOT_SHARED_UP = 54, MG_SLOT_SHARED_DOWN = 55, MG_SLOT_SHARED_SG = 56,
+    MG_LAYER_SLOTS = 64
 };
 MG_API int mg_create_layered(const mg_model_config* cfg, const mg_layer_config* layers, mg_engine** out);
 /* n tokens at positions pos .. pos + n - 1 of the engine's sequence, from the cache and state that

@@ -40,14 +40,31 @@ class MgMatMemConfig(C.Structure):
     _fields_ = [("heads", ci), ("dim", ci), ("vdim", ci), ("gate_cap", cf)]
 
 
+class MgLatentAttnConfig(C.Structure):
+    """struct mg_latent_attn_config of include/mongoose_kernels.h."""
+    _fields_ = [("heads", ci), ("dim", ci), ("rot_dim", ci), ("vdim", ci), ("q_rank", ci), ("kv_rank", ci), ("scale", cf), ("rot_base", cd)]
+
+
+class MgWkvConfig(C.Structure):
+    """struct mg_wkv_config of include/mongoose_kernels.h."""
+    _fields_ = [("heads", ci), ("dim", ci), ("decay_rank", ci)]
+
+
+class MgMoeConfig(C.Structure):
+    """struct mg_moe_config of include/mongoose_kernels.h."""
+    _fields_ = [("experts", ci), ("top", ci), ("ff", ci), ("shared_ff", ci)]
+
+
 class MgLayerConfig(C.Structure):
     """struct mg_layer_config of include/mongoose_kernels.h."""
-    _fields_ = [("mixer", ci), ("attn", MgGateAttnConfig), ("mem", MgMatMemConfig), ("ffn_dim", ci)]
+    _fields_ = [("mixer", ci), ("attn", MgGateAttnConfig), ("mem", MgMatMemConfig), ("ffn_dim", ci), ("latent", MgLatentAttnConfig),
+                ("wkv", MgWkvConfig), ("moe", MgMoeConfig)]
 
 
 class MgModelConfig(C.Structure):
     """struct mg_model_config of include/mongoose_kernels.h."""
-    _fields_ = [("width", ci), ("vocab", ci), ("n_layers", ci), ("max_seq", ci), ("norm_eps", cf), ("math", ci), ("device", ci)]
+    _fields_ = [("width", ci), ("vocab", ci), ("n_layers", ci), ("max_seq", ci), ("norm_eps", cf), ("math", ci), ("device", ci),
+                ("norm", ci), ("positions", ci), ("residual_mult", cf), ("loop_start", ci), ("loop_stop", ci), ("loop_times", ci)]
 
 
 # name -> (restype, argtypes): every symbol include/mongoose_kernels.h declares.

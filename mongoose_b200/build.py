@@ -27,6 +27,7 @@ UNITS = {
     "engine.cu": "core",
     "legacy_ops.cu": "abi", "block_ops.cu": "abi",
     "layered_decode.cu": "layered", "layered_prefill.cu": "layered", "gemm_tc.cu": "layered", "gate_attn_tc.cu": "layered",
+    "latent_attn.cu": "layered", "latent_attn_tc.cu": "layered", "wkv.cu": "layered", "moe.cu": "layered",
     "dense_phases.cu": "dense", "mega_single.cu": "dense", "mega_tp.cu": "dense",
 }
 # A family of models can be served by a library of its own, compiled from what that family needs (the

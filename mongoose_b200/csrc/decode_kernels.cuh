@@ -39,7 +39,10 @@ enum : int { PRO_PLAIN = 0, PRO_RMS = 1, PRO_RMS_EMBED = 2,
              PRO_X = 3,            // x as it is
              PRO_EMBED_POS = 4,    // embedding row + position vector
              PRO_POST = 5,         // x + norm(z)
-             PRO_POST_PAIR = 6 };  // x + norm(half the sum of two normed vectors)
+             PRO_POST_PAIR = 6,    // x + norm(half the sum of two normed vectors)
+             PRO_ADD = 7 };        // x + mult * scale vector * z
+// Kinds of norms of layer-described models (values match MG_NORM_* in mongoose_kernels.h).
+enum : int { NORM_RMS_AROUND_ZERO = 0, NORM_LAYER = 1, NORM_RMS = 2 };
 enum : int { EPI_QKV = 0, EPI_RESID = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_STORE = 4, EPI_GELU = 5 };
 
 // ---------------------------------------------------------------------
@@ -134,6 +137,7 @@ struct PhaseArgs {
     float eps;
     WeightView embed;     // RMS_EMBED: lm_head planes, row `token` is the input embedding
     int embed_fmt;
+    int embed_ld;         // EMBED_POS: padded row length of the embedding
     float* h_store;       // RMS_EMBED: CTA 0 stores the embedded hidden state here
     StepState* st;
     // epilogue
@@ -153,11 +157,17 @@ struct PhaseArgs {
     PushArgs push;        // RESID: send the output rows to every rank instead of (or besides) `out`
     // layer-described models: K is the padded row length of the matrix, k_valid the vector's own length
     int k_valid;
-    const float* pos_tab; // EMBED_POS: [max_seq][k_valid]
-    const float* z[2];    // POST: the sublayer's output; POST_PAIR: its two branches
-    const float* z_w[2];  // POST_PAIR: plain norm weights of the branches
+    const float* pos_tab; // EMBED_POS: [max_seq][k_valid], or NULL
+    const float* z[2];    // POST, ADD: the sublayer's output; POST_PAIR: its two branches
+    const float* z_w[2];  // POST_PAIR: plain norm weights of the branches; ADD: z_w[0] scales z
+    float z_mult;         // ADD
     const float* post_w;  // weight of the norm on the sublayer's output, stored around zero
-    const float* last_w;  // not NULL: a norm (weight around zero) of the sum follows (the model's last)
+    const float* last_w;  // not NULL: a norm of the sum follows (a layer's first step, the model's last)
+    int last_kind;        // NORM_*
+    float* n_store;       // the normed vector is kept here
+    const float* cat;     // appended to the vector: the matrix reads [x; cat], 2 * k_valid columns
+    const float* mix_mu;  // not NULL: the normed vector h becomes h + (h' - h) * mu, h' being the last token's
+    float* mix_prev;      // [2][k_valid]: the slot of parity p holds h' of position p; zeros before position 0
     GatherArgs gather;    // RMS prologue: the hidden state is the sum of the received rows; CTA 0 keeps it in h_store
 };
 
@@ -250,14 +260,15 @@ __device__ __forceinline__ float2 block_sum2(float u, float v, float* red) {
     return make_float2(warp_sum(u), warp_sum(v));
 }
 
-// Prologue of layer-described models.  xs gets K floats, zero from k_valid on; with `keep` the residual
-// sum goes to h_store (never the buffer x_src names: other CTAs still read that one).  `red` is 72 floats.
-// A vector of up to 8 values per thread stays in registers from the first load to the last norm; a
-// longer one goes through xs in pieces, each thread on its own elements.
+// Prologue of layer-described models.  xs gets K floats, zero behind the vector; with `keep` the residual sum
+// goes to h_store (never the buffer x_src names: other CTAs still read that one), the normed vector to
+// n_store and, for a mixed one, to the other slot of mix_prev.  `red` is 72 floats.  A vector of up to 8
+// values per thread stays in registers from the first load to the last norm; a longer one goes through xs
+// in pieces, each thread on its own elements.
 __device__ __forceinline__ void stage_layered(const PhaseArgs& a, float* xs, float* red, bool keep) {
     const int K = a.K, n = a.k_valid, step = Values8::N * blockDim.x;
     const float inv_n = 1.0f / (float)n;
-    for (int i = n + threadIdx.x; i < K; i += blockDim.x) xs[i] = 0.f;
+    for (int i = (a.cat ? 2 * n : n) + threadIdx.x; i < K; i += blockDim.x) xs[i] = 0.f;
     const bool one = n <= step;
     const bool pair = a.pro == PRO_POST_PAIR, post = pair || a.pro == PRO_POST;
     float r = 0.f;
@@ -296,15 +307,17 @@ __device__ __forceinline__ void stage_layered(const PhaseArgs& a, float* xs, flo
         }
         r = 1.0f / sqrtf(block_sum2(ss, 0.f, red).x * inv_n + a.eps);
     }
-    const int token = a.pro == PRO_EMBED_POS ? a.st->token : 0, pos = a.pro == PRO_EMBED_POS ? a.st->pos : 0;
-    float ss = 0.f;
+    const int token = a.pro == PRO_EMBED_POS ? a.st->token : 0;
+    const int pos = a.pro == PRO_EMBED_POS || a.mix_mu ? a.st->pos : 0;
+    float ss = 0.f, sum = 0.f;
     for (int b = 0; b < n; b += step) {
         if (a.pro == PRO_EMBED_POS) {
-            x.load(a.pos_tab + (size_t)pos * n, b, n);
+            if (a.pos_tab) x.load(a.pos_tab + (size_t)pos * n, b, n);
 #pragma unroll
             for (int j = 0; j < Values8::N; j++) {
                 const int i = b + Values8::index(j);
-                if (i < n) x.v[j] += embed_value(a.embed, a.embed_fmt, K, token, i);
+                const float p = a.pos_tab ? x.v[j] : 0.f;
+                x.v[j] = i < n ? p + embed_value(a.embed, a.embed_fmt, a.embed_ld, token, i) : 0.f;
             }
         } else {
             if (!(one && post)) x.load(a.x_src, b, n);
@@ -314,24 +327,68 @@ __device__ __forceinline__ void stage_layered(const PhaseArgs& a, float* xs, flo
                 if (!one) y.load(xs, b, n);
 #pragma unroll
                 for (int j = 0; j < Values8::N; j++) x.v[j] += y.v[j] * r * (1.0f + w.v[j]);
+            } else if (a.pro == PRO_ADD) {
+                Values8 w;
+                w.load(a.z_w[0], b, n);
+                y.load(a.z[0], b, n);
+#pragma unroll
+                for (int j = 0; j < Values8::N; j++) x.v[j] += a.z_mult * (w.v[j] * y.v[j]);
             }
         }
-        if (a.last_w) ss += x.squares();
-        if (keep) x.store(a.h_store, b, n);
+        if (a.last_w) {
+            ss += x.squares();
+#pragma unroll
+            for (int j = 0; j < Values8::N; j++) sum += x.v[j];
+        }
+        if (keep && a.h_store) x.store(a.h_store, b, n);
         if (!(one && a.last_w)) x.store(xs, b, n);
     }
     if (a.last_w) {
-        const float rl = 1.0f / sqrtf(block_sum2(ss, 0.f, red).x * inv_n + a.eps);
+        const float2 t = block_sum2(ss, sum, red);
+        float mean = 0.f, var = t.x * inv_n;
+        if (a.last_kind == NORM_LAYER) {            // the mean square of the deviations themselves
+            mean = t.y * inv_n;
+            float dd = 0.f;
+            for (int b = 0; b < n; b += step) {
+                if (!one) x.load(xs, b, n);
+#pragma unroll
+                for (int j = 0; j < Values8::N; j++) {
+                    const float d = b + Values8::index(j) < n ? x.v[j] - mean : 0.f;
+                    dd = fmaf(d, d, dd);
+                }
+            }
+            var = block_sum2(dd, 0.f, red).x * inv_n;
+        }
+        const float rl = 1.0f / sqrtf(var + a.eps);
+        const float one_more = a.last_kind == NORM_RMS_AROUND_ZERO ? 1.0f : 0.0f;
         for (int b = 0; b < n; b += step) {
             Values8 w;
             w.load(a.last_w, b, n);
             if (!one) x.load(xs, b, n);
 #pragma unroll
-            for (int j = 0; j < Values8::N; j++) x.v[j] *= rl * (1.0f + w.v[j]);
+            for (int j = 0; j < Values8::N; j++) x.v[j] = (x.v[j] - mean) * (rl * (one_more + w.v[j]));
+            if (keep && a.n_store) x.store(a.n_store, b, n);
+            if (a.mix_mu) {
+                if (keep) x.store(a.mix_prev + (size_t)((pos + 1) & 1) * n, b, n);
+                w.load(a.mix_mu, b, n);
+                if (pos > 0) {
+                    y.load(a.mix_prev + (size_t)(pos & 1) * n, b, n);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < Values8::N; j++) y.v[j] = 0.f;
+                }
+#pragma unroll
+                for (int j = 0; j < Values8::N; j++) x.v[j] = fmaf(y.v[j] - x.v[j], w.v[j], x.v[j]);
+            }
             x.store(xs, b, n);
         }
     }
     __syncthreads();
+    if (a.cat) {
+        const bool own = a.cat == a.h_store;        // this kernel stores it: the others have it in xs as well
+        for (int i = threadIdx.x; i < n; i += blockDim.x) xs[n + i] = own ? xs[i] : a.cat[i];
+        __syncthreads();
+    }
 }
 
 __device__ __forceinline__ void stage_x(const PhaseArgs& a, float* xs, float* red) {
@@ -545,7 +602,7 @@ __device__ __forceinline__ void load_stage(const Tile<EPI, R>& t, int c, bool va
 // Dynamic shared memory: K floats (x) + 40 floats (reductions).
 // ---------------------------------------------------------------------
 template <int FMT, int EPI, int R, int D>
-__device__ __forceinline__ void phase_body(const PhaseArgs& a, const int bid, const int nblocks) {
+__device__ __forceinline__ void phase_body(const PhaseArgs& a, const int bid, const int nblocks, const bool keep) {
     using C = Chunk<FMT>;
     extern __shared__ __align__(16) float smem[];
     float* xs = smem;
@@ -584,7 +641,7 @@ __device__ __forceinline__ void phase_body(const PhaseArgs& a, const int bid, co
     constexpr bool kInt = (FMT != FMT_F16 && FMT != FMT_BF16);          // int8 / 4-bit weights: integer dot products
     float rms = 1.0f;
     if (kInt) rms = stage_xq(a, reinterpret_cast<uint8_t*>(smem), red, FMT == FMT_Q4_0);
-    else if (FMT == FMT_BF16) stage_layered(a, xs, red, bid == 0 && a.h_store != nullptr);
+    else if (FMT == FMT_BF16) stage_layered(a, xs, red, keep);
     else stage_x(a, xs, red);
     const uint8_t* P0 = reinterpret_cast<const uint8_t*>(smem);
     const uint8_t* P1 = P0 + a.K;
@@ -789,14 +846,36 @@ __device__ __forceinline__ void phase_body(const PhaseArgs& a, const int bid, co
 
 template <int FMT, int EPI, int R, int D>
 __global__ void __launch_bounds__(256) phase_kernel(const PhaseArgs a) {
-    phase_body<FMT, EPI, R, D>(a, blockIdx.x, gridDim.x);
+    phase_body<FMT, EPI, R, D>(a, blockIdx.x, gridDim.x, blockIdx.x == 0);
 }
 
 // Two independent matrices in one launch: the first `split` CTAs multiply a's, the others b's.
 template <int FMT, int EPI, int R, int D>
 __global__ void __launch_bounds__(256) phase_pair_kernel(const PhaseArgs a, const PhaseArgs b, int split) {
     const bool first = (int)blockIdx.x < split;
-    phase_body<FMT, EPI, R, D>(first ? a : b, first ? blockIdx.x : blockIdx.x - split, first ? split : gridDim.x - split);
+    phase_body<FMT, EPI, R, D>(first ? a : b, first ? blockIdx.x : blockIdx.x - split, first ? split : gridDim.x - split, first ? blockIdx.x == 0 : (int)blockIdx.x == split);
+}
+
+// Several matrices on mixes of one vector: part p's CTAs multiply its matrix by the mix with its own mu.
+constexpr int kMaxParts = 5;
+struct PhaseParts {
+    int n;
+    int first[kMaxParts + 1];   // CTAs [first[p], first[p + 1])
+    WeightView w[kMaxParts];
+    int rows[kMaxParts];
+    const float* mu[kMaxParts];
+    float* out[kMaxParts];
+};
+
+template <int FMT, int EPI, int R, int D>
+__global__ void __launch_bounds__(256) phase_parts_kernel(const PhaseArgs a, const PhaseParts parts) {
+    int p = 0;
+#pragma unroll
+    for (int i = 1; i < kMaxParts; i++)
+        if (i < parts.n && (int)blockIdx.x >= parts.first[i]) p = i;
+    PhaseArgs b = a;
+    b.w[0] = parts.w[p]; b.rows[0] = parts.rows[p]; b.nitems = (parts.rows[p] + R - 1) / R; b.mix_mu = parts.mu[p]; b.out = parts.out[p];
+    phase_body<FMT, EPI, R, D>(b, blockIdx.x - parts.first[p], parts.first[p + 1] - parts.first[p], blockIdx.x == 0);
 }
 
 // Sum of the received rows into a plain vector (the hidden state a layer range hands back to the

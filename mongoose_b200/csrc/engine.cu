@@ -1426,7 +1426,10 @@ int mg_create_layered(const mg_model_config* cfg, const mg_layer_config* layers,
         m.layers.push_back(l);
     }
     mg_config& c = e->cfg;
-    c.dim = cfg->width; c.vocab = cfg->vocab; c.n_layers = cfg->n_layers; c.max_seq = cfg->max_seq; c.rms_eps = cfg->norm_eps;
+    const bool loops = cfg->loop_times > 0 && cfg->loop_start >= 0 && cfg->loop_stop > cfg->loop_start && cfg->loop_stop <= cfg->n_layers;
+    // the stepping calls count the runs of layers
+    c.n_layers = cfg->n_layers + (loops ? (cfg->loop_stop - cfg->loop_start) * (cfg->loop_times - 1) : 0);
+    c.dim = cfg->width; c.vocab = cfg->vocab; c.max_seq = cfg->max_seq; c.rms_eps = cfg->norm_eps;
     c.layer_fmt = c.head_fmt = MG_FMT_BF16; c.device = cfg->device; c.max_batch = 1;
     int rc = create_common(e);
     if (rc) return bail(rc, "no usable device");
@@ -1449,20 +1452,7 @@ int mg_create_layered(const mg_model_config* cfg, const mg_layer_config* layers,
         return bail(rc, e->err.c_str());
     if ((rc = create_cursor(e))) return bail(rc, "cursor");
     layered_slots(m);
-    for (LayerWeights& l : m.layers) {
-        std::vector<float> sl(l.at.heads);
-        for (int h = 0; h < l.at.heads; h++) sl[h] = (float)pow(2.0, -8.0 * (h + 1) / l.at.heads);
-        if (cudaMemcpy(l.slopes, sl.data(), sl.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) return bail(MG_ERR_CUDA, "upload");
-    }
-    {   // position vectors in float64 on the host, narrowed to fp32, like the RoPE tables of mg_create
-        const int W = c.dim;
-        std::vector<double> f((W + 1) / 2);
-        for (size_t i = 0; i < f.size(); i++) f[i] = pow(10000.0, -2.0 * (double)i / W);
-        std::vector<float> tab((size_t)c.max_seq * W);
-        for (int p = 0; p < c.max_seq; p++)
-            for (int i = 0; i < W; i++) tab[(size_t)p * W + i] = (float)(i & 1 ? cos(p * f[i / 2]) : sin(p * f[i / 2]));
-        if (cudaMemcpy(m.pos_tab, tab.data(), tab.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) return bail(MG_ERR_CUDA, "upload");
-    }
+    if ((rc = layered_tables(e))) return bail(rc, e->err.c_str());
     read_env(e);
     e->use_mega = false;
     *out = e;

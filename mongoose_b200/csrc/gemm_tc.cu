@@ -19,6 +19,8 @@ __device__ __forceinline__ float gelu_tanh_fast(float z) {
     return z - z * __fdividef(1.0f, 1.0f + __expf(2.0f * u));
 }
 
+__device__ __forceinline__ float silu_fast(float z) { return z * __fdividef(1.0f, 1.0f + __expf(-z)); }
+
 template <int BN>
 struct Smem {
     static constexpr int a_bytes = 128 * 128, b_bytes = BN * 128, stage = a_bytes + b_bytes;
@@ -35,7 +37,13 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
     uint32_t* tmem_base = reinterpret_cast<uint32_t*>(done + 1);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int col0 = blockIdx.x * BN, row0 = blockIdx.y * 128, z = blockIdx.z;
+    const bool dual = BN == 128 && g.mode == GEMM_SILU_BF16;
+    const int col0 = blockIdx.x * (dual ? 64 : BN), row0 = blockIdx.y * 128, z = blockIdx.z;
+    int zb = z / g.b_group;
+    if (g.group) {
+        zb = g.group[blockIdx.y];
+        if (zb < 0) return;
+    }
     int kt = (g.k + 63) / 64;
     if (g.causal_pos0 >= 0) kt = min(kt, (g.causal_pos0 + min(row0 + 128, g.m) + 63) / 64);
 
@@ -45,6 +53,7 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
         bar_init_fence();
         tma_prefetch_map(&g.a);
         tma_prefetch_map(&g.b);
+        if (dual) tma_prefetch_map(&g.b2);
     }
     if (warp == 1) tmem_alloc(tmem_base, BN);
     tc_fence_before();
@@ -61,7 +70,8 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
                 bar_expect(full + s, Smem<BN>::stage);
                 uint8_t* st = base + s * Smem<BN>::stage;
                 tma_load_3d(st, &g.a, i * 64, row0, z, full + s);
-                tma_load_3d(st + Smem<BN>::a_bytes, &g.b, i * 64, col0, z / g.b_group, full + s);
+                tma_load_3d(st + Smem<BN>::a_bytes, &g.b, i * 64, col0, zb, full + s);
+                if (dual) tma_load_3d(st + Smem<BN>::a_bytes + 64 * 128, &g.b2, i * 64, col0, zb, full + s);
                 issued = i + 1;
             }
             // no copy may be in flight when the CTA leaves
@@ -91,9 +101,15 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
         float* tile = reinterpret_cast<float*>(base) + quarter * 32 * 33;     // every stage has been consumed
         if (ok) {
 #pragma unroll 1
-            for (int c = 0; c < BN; c += 32) {
+            for (int c = 0; c < (dual ? 64 : BN); c += 32) {
                 float v[32];
                 tmem_load32(acc + ((uint32_t)(quarter * 32) << 16) + c, v);
+                if (dual) {
+                    float u[32];
+                    tmem_load32(acc + ((uint32_t)(quarter * 32) << 16) + 64 + c, u);
+#pragma unroll
+                    for (int i = 0; i < 32; i++) v[i] = silu_fast(v[i]) * u[i];
+                }
 #pragma unroll
                 for (int i = 0; i < 32; i++) tile[lane * 33 + i] = v[i];
                 __syncwarp();
@@ -159,7 +175,8 @@ template <int BN>
 cudaError_t run(const GemmTC& g, cudaStream_t s) {
     static cudaError_t attr = cudaFuncSetAttribute((const void*)gemm_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<BN>::bytes);
     if (attr != cudaSuccess) return attr;
-    gemm_tc_kernel<BN><<<dim3((g.n + BN - 1) / BN, (g.m + 127) / 128, g.batch), kThreads, Smem<BN>::bytes, s>>>(g);
+    const int cols = g.mode == GEMM_SILU_BF16 ? 64 : BN;
+    gemm_tc_kernel<BN><<<dim3((g.n + cols - 1) / cols, (g.m + 127) / 128, g.batch), kThreads, Smem<BN>::bytes, s>>>(g);
     return cudaGetLastError();
 }
 
@@ -180,7 +197,7 @@ bool make_head_map(CUtensorMap* map, const void* base, int k, int batch, int row
 }
 
 cudaError_t launch_gemm_tc(const GemmTC& g, cudaStream_t s) {
-    if (g.bn == 64) return run<64>(g, s);
+    if (g.bn == 64 && g.mode != GEMM_SILU_BF16) return run<64>(g, s);
     if (g.bn == 128) return run<128>(g, s);
     return cudaErrorInvalidValue;
 }

@@ -1,6 +1,7 @@
 // Launchers of the kernels that serve layer-described models (mg_create_layered).  One entry per
 // mechanism, every size and constant an argument; the kernels themselves are in layered_decode.cu (one
-// token), layered_prefill.cu (portions of a prompt), gate_attn_tc.cu and gemm_tc.cu (bf16 tensor cores).
+// token), layered_prefill.cu (portions of a prompt), latent_attn.cu, wkv.cu and moe.cu (both), gate_attn_tc.cu,
+// latent_attn_tc.cu and gemm_tc.cu (bf16 tensor cores).
 #pragma once
 
 #include <cuda.h>
@@ -49,10 +50,54 @@ struct ProjCols {
     int q, k, mq, mk, mv, mg, mi, mf, total;
 };
 
+// Softmax attention over a cached latent c (rank values) and a rotated key part shared by the heads.  A head's
+// unrotated key is U_k c and its value U_v c, so q . (U_k c) = (U_k^T q) . c: one token, and 32-bit mode, score
+// the cached rows themselves with U_k^T q and apply U_v to the weighted sum of rows; bf16 prompts form keys and
+// values.  Parts of a row are padded to multiples of 8 with zeros.
+struct LatentAttn {
+    int heads, dim, rot, vdim, rank, q_rank;
+    int dim_s, rot_s, rank_s;
+    float scale, eps;
+    const float *q_norm, *c_norm;       // [q_rank], [rank]
+    const float *cos_tab, *sin_tab;     // [max_seq][rot / 2]
+    const __nv_bfloat16 *uk, *uv;       // [heads * dim_s][ld], [heads * vdim][ld]
+    int ld;                             // rank padded to a multiple of 64
+    void* cache;                        // [max_seq][rank_s + rot_s] bf16 or fp32
+    int max_seq;
+    __host__ __device__ int row() const { return rank_s + rot_s; }      // a cached row
+    __host__ __device__ int qrow() const { return dim_s + rot_s; }      // a head's query
+};
+
+// Linear recurrence with a decay per key channel.
+struct Wkv {
+    int heads, dim, rank;               // rank of the decay's projection
+    float eps;
+    const __nv_bfloat16* w2;            // [heads * dim][ld2]
+    int ld2;
+    const float *w0, *u, *norm;         // [heads * dim]
+    float* S;                           // [heads][dim key channels][dim value channels]
+};
+
+// Mixture of experts: `top` of `experts` gated feed-forwards of inner width ff, and a shared one.
+struct Moe {
+    int experts, top, ff, shared_ff, width;
+    int ffs, shared_ffs;                // padded to multiples of 64
+    const float* bias;                  // [experts]
+    const uint8_t *gate, *up, *down;    // bf16 [experts * ff][ldw], [experts * ff][ldw], [experts * width][ffs]
+    const uint8_t* shared_down;         // [width][shared_ffs]
+    int ldw;
+    // a router row: logits, the shared expert's gate, then (one token) its gate and up projections
+    __host__ __device__ int sg_col() const { return experts; }
+};
+constexpr int kMaxExperts = 1024, kMaxTop = 64;
+
 // ---- one token (layered_decode.cu) -------------------------------------------------------------
 phase_fn_t layered_phase(int epi, int R);
 typedef void (*phase_pair_fn_t)(const PhaseArgs, const PhaseArgs, int);
 phase_pair_fn_t layered_phase_pair(int R);
+
+typedef void (*phase_parts_fn_t)(const PhaseArgs, const PhaseParts);
+phase_parts_fn_t layered_phase_parts(int R);
 
 // Largest dynamic shared memory the phase kernels may be launched with.
 cudaError_t layered_phase_smem(size_t bytes);
@@ -83,13 +128,101 @@ struct ResolveArgs {            // the pending residual update of a step that en
 };
 cudaError_t launch_resolve(const ResolveArgs& a, bool pdl, cudaStream_t s);
 
+// ---- latent attention (latent_attn.cu) ----
+// Work on tokens one after the other in memory: one token at st->pos, or `tokens` of them from pos0 (st NULL).
+struct LatentStep {
+    LatentAttn at;
+    const StepState* st;
+    int pos0, tokens;
+    const float* q;             // [tokens][heads * qrow] queries, not yet rotated
+    const float* down;          // one token: [q_rank + rank + rot], its latent and rotated part go into the cache
+    float* qa;                  // [tokens][heads][row]: U_k^T q and the rotated part, times scale
+    int splits, tile, group;    // key ranges; keys per tile; heads per CTA
+    float* part;                // [tokens][splits][heads][rank_s]
+    float2* ml;                 // [tokens][splits][heads] maximum and sum of the range
+    void* out;                  // [tokens][ld_out]
+    int ld_out;
+};
+// Tile and heads per CTA of the attention over cached rows; 0: the sizes do not fit.
+size_t latent_attend_smem(const LatentAttn& at, bool f32_cache, int* tile, int* group);
+cudaError_t launch_latent_query(const LatentStep& a, bool f32_cache, bool pdl, cudaStream_t s);
+cudaError_t launch_latent_attend(const LatentStep& a, bool f32_cache, bool pdl, cudaStream_t s);
+cudaError_t launch_latent_value(const LatentStep& a, bool f32_out, bool pdl, cudaStream_t s);
+// rows of a portion: act = normed query latent; normed latent and rotated key part into the cache
+cudaError_t launch_latent_rows(const LatentAttn& at, const float* down, int ldd, int pos0, int n, void* act, int ld_act, bool f32, cudaStream_t s);
+// rows of a portion: qh = queries with their rotated part rotated, times scale * log2 e (bf16)
+cudaError_t launch_latent_q_rows(const LatentAttn& at, const float* q, int pos0, int n, void* qh, cudaStream_t s);
+// bf16 prompts on the tensor cores (latent_attn_tc.cu): keys [max_seq][heads * dim_s] and values, transposed,
+// [heads * vdim][ldv] of positions [0, pos0 + n) are formed from the cache, then attention in tiles of 128 queries.
+bool latent_attn_tc_fits(const LatentAttn& at);
+cudaError_t launch_latent_attn_tc(const LatentAttn& at, const void* qh, int pos0, int n, void* keys, void* vt, int ldv, void* out, int ld_out,
+                                  int* status, int* launches, cudaStream_t s);
+
+// ---- linear recurrence (wkv.cu) ----
+struct WkvStep {
+    Wkv wk;
+    const float* row;           // r, k, v, g [heads * dim] each, then the decay's inner projection [rank]
+    const StepState* st;
+    float* y;                   // [heads * dim]
+};
+cudaError_t launch_wkv_step(const WkvStep& a, bool pdl, cudaStream_t s);
+size_t wkv_step_smem(const Wkv& wk);
+// act[j][r] = the mix of row r and the one before it (prev before the first) with mu[j]
+cudaError_t launch_wkv_mix(const float* h, const float* prev, const float* const mu[5], int pos0, int n, int width, void* act, int ld_act,
+                           long long act_stride, bool f32, cudaStream_t s);
+bool wkv_rows_fits(const Wkv& wk);
+// proj rows as WkvStep's, decays [n][heads * dim]; out [n][heads * dim] raw outputs
+cudaError_t launch_wkv_rows(const Wkv& wk, const float* proj, int ldp, const float* decay, int pos0, int n, float* out, cudaStream_t s);
+
+// ---- mixture of experts (moe.cu) ----
+struct MoeStep {
+    Moe moe;
+    const float* router;        // one router row
+    const float* h;             // [width] normed
+    float* mid;                 // [top * ff] of the chosen experts
+    float* out;                 // [width]
+};
+size_t moe_step_smem(const Moe& m);
+cudaError_t moe_step_attrs(size_t bytes);
+cudaError_t launch_moe_up(const MoeStep& a, int sms, bool pdl, cudaStream_t s);
+cudaError_t launch_moe_down(const MoeStep& a, int sms, bool pdl, cudaStream_t s);
+struct MoeRows {                // workspace of a portion
+    int *sel, *slot;            // [n][top] chosen expert, its row among the grouped rows
+    float* weight;              // [n][top]
+    int* count;                 // [experts], zero between calls
+    int* first;                 // [experts + 1] first grouped row of an expert
+    int* group;                 // [tiles] expert of every 128 grouped rows, -1: none
+    int tiles;
+    void* x;                    // [tiles * 128][ldw] grouped inputs
+    float* y;                   // [tiles * 128][width]
+};
+inline int moe_tiles(const Moe& m, int n) { return (int)(((long long)n * m.top + 127) / 128) + m.experts; }
+// choice, grouping and the grouped inputs
+cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s);
+// z = weighted sum of the grouped rows (+ z times the shared expert's gate)
+cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, cudaStream_t s);
+
 // ---- portions of a prompt (layered_prefill.cu) -----------------------------------------------------
 // `act` buffers hold bf16 or fp32 (f32 = true) rows padded to a multiple of 64 with zeros.
 cudaError_t launch_embed_rows(const WeightView& embed, int ld_embed, const float* pos_tab, const int* tokens, int pos0, int n,
                               int width, float* x, void* act, int ld_act, bool f32, cudaStream_t s);
-// out[n][ldc] = A[n][K] W[rows][K]^T, fp32 accumulation on the CUDA cores (32-bit mode)
-cudaError_t launch_gemm_f32(const float* A, int lda, const uint8_t* W, int ldw, float* out, int ldc, int n, int rows, int K,
-                            bool gelu, cudaStream_t s);
+// out[n][ldc] = A[n][K] W[rows][K]^T, fp32 on the CUDA cores (32-bit mode, and what is 32-bit in every mode)
+enum : int { F32_STORE = 0, F32_GELU = 1,
+             F32_SILU_MUL = 2,      // silu(aux) * the product
+             F32_DECAY = 3 };       // exp(-exp(tanh(A) W^T + bias))
+struct GemmF32 {
+    const float* A;
+    int lda;
+    const uint8_t* W;
+    int ldw;
+    float* out;
+    int ldc, n, rows, K, epi;
+    const float* aux;               // [n][ldc]
+    const float* bias;              // [rows]
+    const int* group;               // per 128 rows of A: which of the stacked matrices (-1: none); NULL: one matrix
+    long long group_stride;         // elements between the stacked matrices
+};
+cudaError_t launch_gemm_f32(const GemmF32& g, cudaStream_t s);
 // queries: normed, times temperature, score scale and key-norm weight; keys: raw rows into the cache
 cudaError_t launch_qk_rows(const GateAttn& at, const float* proj, int ldp, int q_col, int k_col, int pos0, int n, void* qh,
                            bool f32, cudaStream_t s);
@@ -105,9 +238,29 @@ cudaError_t launch_gate_attn_tc(const GateAttn& at, const void* qh, int pos0, in
 // x += norm(z) or x += norm(half the sum of two normed branches); act = x
 cudaError_t launch_post_rows(float* x, const float* z0, const float* z1, const float* w0, const float* w1, const float* post_w,
                              float eps, int n, int width, void* act, int ld_act, bool f32, cudaStream_t s);
-// act[r] = norm(x[rows[r]]), weight around zero
-cudaError_t launch_last_norm_rows(const float* x, const int* rows, const float* w, float eps, int n, int width, void* act,
+// act[r] = norm(x[rows[r]]) of the kind NORM_*
+cudaError_t launch_last_norm_rows(const float* x, const int* rows, const float* w, int kind, float eps, int n, int width, void* act,
                                   int ld_act, bool f32, cudaStream_t s);
+// x += mult * ls * z (where z is given); then act (or h, 32-bit rows without padding) = norm(x), or, where cat is
+// given, act = [x, cat]
+struct PrenormRows {
+    float* x;
+    const float *z, *ls;
+    float mult;
+    const float* norm_w;            // NULL: no norm, act = x where given
+    int kind;
+    float eps;
+    int n, width;
+    void* act;
+    int ld_act;
+    float* h;
+    const float* cat;
+};
+cudaError_t launch_prenorm_rows(const PrenormRows& a, bool f32, cudaStream_t s);
+// act[t] = unit rms per head of o[t] (a norm weight over all heads) times a gate
+enum : int { GATE_SIGMOID = 0, GATE_SILU = 1 };
+cudaError_t launch_head_norm_rows(int heads, int vdim, float eps, const float* norm, const float* gate, int ldg, int gate_kind, int n,
+                                  const float* o, void* act, int ld_act, bool f32, cudaStream_t s);
 
 struct MemRows {                // workspace of the chunked memory for up to n tokens
     double* b;                  // [heads][n] log-forget sum inside the chunk

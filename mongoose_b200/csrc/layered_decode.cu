@@ -19,6 +19,10 @@ phase_pair_fn_t layered_phase_pair(int R) {
     return R == 4 ? phase_pair_kernel<FMT_BF16, EPI_STORE, 4, 2> : R == 2 ? phase_pair_kernel<FMT_BF16, EPI_STORE, 2, 4> : phase_pair_kernel<FMT_BF16, EPI_STORE, 1, 8>;
 }
 
+phase_parts_fn_t layered_phase_parts(int R) {
+    return R == 4 ? phase_parts_kernel<FMT_BF16, EPI_STORE, 4, 2> : R == 2 ? phase_parts_kernel<FMT_BF16, EPI_STORE, 2, 4> : phase_parts_kernel<FMT_BF16, EPI_STORE, 1, 8>;
+}
+
 namespace {
 
 constexpr int kStateRows = 16;      // rows of the state a warp holds at a time
@@ -178,28 +182,13 @@ __global__ void __launch_bounds__(256) resolve_kernel(const ResolveArgs a) {
     for (int i = threadIdx.x; i < a.p.k_valid; i += blockDim.x) a.out[i] = smem[i];
 }
 
-template <typename F, typename... Args>
-cudaError_t go(F kern, int grid, int threads, size_t smem, bool pdl, cudaStream_t s, Args... args) {
-    cudaLaunchConfig_t cfg{};
-    cfg.gridDim = dim3((unsigned)grid);
-    cfg.blockDim = dim3((unsigned)threads);
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = s;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = pdl ? 1 : 0;
-    return cudaLaunchKernelEx(&cfg, kern, args...);
-}
-
 template <typename KT>
 cudaError_t step_for(const MixerStep& a, size_t smem, bool pdl, cudaStream_t s) {
     const int ep = attn_pairs(a.at);
     const int grid = a.n_mem + a.splits;
     auto run = [&](auto kern) {
         cudaError_t c = cudaFuncSetAttribute((const void*)kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        return c != cudaSuccess ? c : go(kern, grid, kAttnThreads, smem, pdl, s, a);
+        return c != cudaSuccess ? c : launch_pdl(kern, grid, kAttnThreads, smem, pdl, s, a);
     };
     switch (ep) {
         case 1: return run(mixer_step_kernel<KT, 1>);
@@ -219,8 +208,10 @@ cudaError_t layered_phase_smem(size_t bytes) {
             cudaError_t c = cudaFuncSetAttribute((const void*)layered_phase(epi, R), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
             if (c != cudaSuccess) return c;
         }
-        cudaError_t c = cudaFuncSetAttribute((const void*)layered_phase_pair(R), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
-        if (c != cudaSuccess) return c;
+        for (const void* f : {(const void*)layered_phase_pair(R), (const void*)layered_phase_parts(R)}) {
+            cudaError_t c = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+            if (c != cudaSuccess) return c;
+        }
     }
     return cudaSuccess;
 }
@@ -239,13 +230,13 @@ cudaError_t launch_mixer_step(const MixerStep& a, bool f32_cache, bool pdl, cuda
 
 cudaError_t launch_mixer_join(const MixerStep& a, bool pdl, cudaStream_t s) {
     const int nm = a.n_mem ? a.mem.heads : 0;
-    return go(mixer_join_kernel, nm + (a.at.heads * a.at.dim + kJoinCols - 1) / kJoinCols, kJoinCols * kJoinParts, 0, pdl, s, a);
+    return launch_pdl(mixer_join_kernel, nm + (a.at.heads * a.at.dim + kJoinCols - 1) / kJoinCols, kJoinCols * kJoinParts, 0, pdl, s, a);
 }
 
 cudaError_t launch_resolve(const ResolveArgs& a, bool pdl, cudaStream_t s) {
     const size_t smem = ((size_t)a.p.K + 72) * sizeof(float);
     cudaError_t c = cudaFuncSetAttribute((const void*)resolve_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return c != cudaSuccess ? c : go(resolve_kernel, 1, 256, smem, pdl, s, a);
+    return c != cudaSuccess ? c : launch_pdl(resolve_kernel, 1, 256, smem, pdl, s, a);
 }
 
 }  // namespace mg

@@ -293,4 +293,22 @@ __device__ __forceinline__ void attend(const GateAttn& A, const AttnSmem<KT>& sm
     }
 }
 
+__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+
+// Launch with the programmatic attribute, so that the kernel may start under its predecessor's tail.
+template <typename F, typename... Args>
+inline cudaError_t launch_pdl(F kern, dim3 grid, int threads, size_t smem, bool pdl, cudaStream_t s, Args... args) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3((unsigned)threads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl ? 1 : 0;
+    return cudaLaunchKernelEx(&cfg, kern, args...);
+}
+
 }  // namespace mg

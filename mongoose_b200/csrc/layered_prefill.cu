@@ -13,30 +13,47 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(WeightView embed, int l
                                                          int pos0, int width, float* x, AT* act, int ld_act) {
     const int r = blockIdx.x, token = tokens[r];
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = embed_value(embed, FMT_BF16, ld_embed, token, i) + pos_tab[(size_t)(pos0 + r) * width + i];
+        const float v = embed_value(embed, FMT_BF16, ld_embed, token, i) + (pos_tab ? pos_tab[(size_t)(pos0 + r) * width + i] : 0.f);
         x[(size_t)r * width + i] = v;
         from_f32(v, act + (size_t)r * ld_act + i);
     }
 }
 
-// 64 x 64 tile, 16 columns of K per step, 4 x 4 outputs per thread.
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W,
-                                                       int ldw, float* out, int ldc, int n, int rows, int K, int gelu) {
+// 64 x 64 tile, 16 columns of K per step, 4 x 4 outputs per thread.  W's rows are padded with zeros to a multiple
+// of 16 at least; A's columns from K on are not read.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 g) {
     __shared__ __align__(16) float As[16][68], Ws[16][68];
     const int r0 = blockIdx.y * 64, c0 = blockIdx.x * 64;
+    const __nv_bfloat16* W = reinterpret_cast<const __nv_bfloat16*>(g.W);
+    if (g.group) {
+        const int e = g.group[r0 / 128];
+        if (e < 0) return;
+        W += e * g.group_stride;
+    }
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
     float acc[4][4] = {};
-    for (int k0 = 0; k0 < K; k0 += 16) {
-        float4 av = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int k0 = 0; k0 < g.K; k0 += 16) {
+        float a4[4] = {0.f, 0.f, 0.f, 0.f};
         float2 w0 = make_float2(0.f, 0.f), w1 = w0;
-        if (r0 + lr < n) av = *reinterpret_cast<const float4*>(A + (size_t)(r0 + lr) * lda + k0 + lk);
-        if (c0 + lr < rows) {
-            const __nv_bfloat16* wp = W + (size_t)(c0 + lr) * ldw + k0 + lk;
+        if (r0 + lr < g.n) {
+            const float* ap = g.A + (size_t)(r0 + lr) * g.lda + k0 + lk;
+            if (k0 + lk + 4 <= g.K) {
+                const float4 av = *reinterpret_cast<const float4*>(ap);
+                a4[0] = av.x; a4[1] = av.y; a4[2] = av.z; a4[3] = av.w;
+            } else {
+                for (int i = 0; i < 4; i++)
+                    if (k0 + lk + i < g.K) a4[i] = ap[i];
+            }
+            if (g.epi == F32_DECAY)
+                for (int i = 0; i < 4; i++) a4[i] = tanhf(a4[i]);
+        }
+        if (c0 + lr < g.rows) {
+            const __nv_bfloat16* wp = W + (size_t)(c0 + lr) * g.ldw + k0 + lk;
             w0 = pair_f32(wp);
             w1 = pair_f32(wp + 2);
         }
-        As[lk][lr] = av.x; As[lk + 1][lr] = av.y; As[lk + 2][lr] = av.z; As[lk + 3][lr] = av.w;
+        As[lk][lr] = a4[0]; As[lk + 1][lr] = a4[1]; As[lk + 2][lr] = a4[2]; As[lk + 3][lr] = a4[3];
         Ws[lk][lr] = w0.x; Ws[lk + 1][lr] = w0.y; Ws[lk + 2][lr] = w1.x; Ws[lk + 3][lr] = w1.y;
         __syncthreads();
 #pragma unroll
@@ -55,7 +72,12 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int r = r0 + ty * 4 + i, c = c0 + tx * 4 + j;
-            if (r < n && c < rows) out[(size_t)r * ldc + c] = gelu ? gelu_tanh(acc[i][j]) : acc[i][j];
+            if (r >= g.n || c >= g.rows) continue;
+            float v = acc[i][j];
+            if (g.epi == F32_GELU) v = gelu_tanh(v);
+            else if (g.epi == F32_SILU_MUL) v *= silu(g.aux[(size_t)r * g.ldc + c]);
+            else if (g.epi == F32_DECAY) v = expf(-expf(v + g.bias[c]));
+            g.out[(size_t)r * g.ldc + c] = v;
         }
 }
 
@@ -130,15 +152,70 @@ __global__ void __launch_bounds__(256) post_rows_kernel(float* x, const float* z
     }
 }
 
+// Mean and 1 / sqrt(spread + eps) of a row for a norm of the given kind; get(i) is the thread's own element i.
+template <typename F>
+__device__ __forceinline__ float2 row_norm(F get, int kind, float eps, int width, float* red) {
+    const float inv = 1.0f / (float)width;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = get(i);
+        s += kind == NORM_LAYER ? v : v * v;
+    }
+    s = block_sum(s, red) * inv;
+    if (kind != NORM_LAYER) return make_float2(0.f, 1.0f / sqrtf(s + eps));
+    float d = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = get(i) - s;
+        d = fmaf(v, v, d);
+    }
+    return make_float2(s, 1.0f / sqrtf(block_sum(d, red) * inv + eps));
+}
+
 template <typename AT>
-__global__ void __launch_bounds__(256) last_norm_rows_kernel(const float* x, const int* rows, const float* w, float eps, int width,
+__global__ void __launch_bounds__(256) last_norm_rows_kernel(const float* x, const int* rows, const float* w, int kind, float eps, int width,
                                                              AT* act, int ld_act) {
     __shared__ float red[40];
     const float* a = x + (size_t)rows[blockIdx.x] * width;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(a[i], a[i], ss);
-    const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) from_f32(a[i] * r * (1.0f + w[i]), act + (size_t)blockIdx.x * ld_act + i);
+    const float2 n = row_norm([&](int i) { return a[i]; }, kind, eps, width, red);
+    const float one = kind == NORM_RMS_AROUND_ZERO ? 1.0f : 0.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) from_f32((a[i] - n.x) * n.y * (one + w[i]), act + (size_t)blockIdx.x * ld_act + i);
+}
+
+template <typename AT>
+__global__ void __launch_bounds__(256) prenorm_rows_kernel(const PrenormRows a) {
+    extern __shared__ __align__(16) float y[];
+    __shared__ float red[40];
+    const int W = a.width;
+    const size_t r = blockIdx.x;
+    float* x = a.x + r * W;
+    AT* act = static_cast<AT*>(a.act) + r * a.ld_act;
+    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+        float v = x[i];
+        if (a.z) {
+            v += a.mult * (a.ls[i] * a.z[r * W + i]);
+            x[i] = v;
+        }
+        y[i] = v;
+    }
+    if (a.cat) {
+        for (int i = threadIdx.x; i < W; i += blockDim.x) {
+            from_f32(y[i], act + i);
+            from_f32(a.cat[r * W + i], act + W + i);
+        }
+        return;
+    }
+    if (!a.norm_w) {
+        if (a.act)
+            for (int i = threadIdx.x; i < W; i += blockDim.x) from_f32(y[i], act + i);
+        return;
+    }
+    const float2 n = row_norm([&](int i) { return y[i]; }, a.kind, a.eps, W, red);
+    const float one = a.kind == NORM_RMS_AROUND_ZERO ? 1.0f : 0.0f;
+    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+        const float v = (y[i] - n.x) * n.y * (one + a.norm_w[i]);
+        if (a.h) a.h[r * W + i] = v;
+        else from_f32(v, act + i);
+    }
 }
 
 // ---------------------------------------------------------------------
@@ -400,18 +477,19 @@ __global__ void __launch_bounds__(256) mem_out_kernel(MatMem M, int q_col, int k
 
 // One warp per (token, head): unit rms, norm weight, output gate.
 template <typename AT>
-__global__ void __launch_bounds__(256) mem_norm_kernel(MatMem M, int g_col, const float* proj, int ldp, int n, const float* o, AT* act,
-                                                       int ld_act) {
+__global__ void __launch_bounds__(256) head_norm_rows_kernel(int heads, int vdim, float eps, const float* norm, const float* gate, int ldg,
+                                                             int gate_kind, int n, const float* o, AT* act, int ld_act) {
     const int wq = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
-    const int t = wq / M.heads, h = wq - t * M.heads;
+    const int t = wq / heads, h = wq - t * heads;
     if (t >= n) return;
-    const float* p = o + ((size_t)t * M.heads + h) * M.vdim;
+    const float* p = o + ((size_t)t * heads + h) * vdim;
     float ss = 0.f;
-    for (int v = lane; v < M.vdim; v += 32) ss = fmaf(p[v], p[v], ss);
-    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)M.vdim + M.eps);
-    for (int v = lane; v < M.vdim; v += 32) {
-        const int c = h * M.vdim + v;
-        from_f32(p[v] * r * M.norm[c] * sigmoid(proj[(size_t)t * ldp + g_col + c]), act + (size_t)t * ld_act + c);
+    for (int v = lane; v < vdim; v += 32) ss = fmaf(p[v], p[v], ss);
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+    for (int v = lane; v < vdim; v += 32) {
+        const int c = h * vdim + v;
+        const float g = gate[(size_t)t * ldg + c];
+        from_f32(p[v] * r * norm[c] * (gate_kind == GATE_SILU ? silu(g) : sigmoid(g)), act + (size_t)t * ld_act + c);
     }
 }
 
@@ -445,10 +523,8 @@ cudaError_t launch_embed_rows(const WeightView& embed, int ld_embed, const float
     return cudaGetLastError();
 }
 
-cudaError_t launch_gemm_f32(const float* A, int lda, const uint8_t* W, int ldw, float* out, int ldc, int n, int rows, int K, bool gelu,
-                            cudaStream_t s) {
-    const dim3 grid((rows + 63) / 64, (n + 63) / 64);
-    gemm_f32_kernel<<<grid, 256, 0, s>>>(A, lda, (const __nv_bfloat16*)W, ldw, out, ldc, n, rows, K, gelu ? 1 : 0);
+cudaError_t launch_gemm_f32(const GemmF32& g, cudaStream_t s) {
+    gemm_f32_kernel<<<dim3((g.rows + 63) / 64, (g.n + 63) / 64), 256, 0, s>>>(g);
     return cudaGetLastError();
 }
 
@@ -478,10 +554,25 @@ cudaError_t launch_post_rows(float* x, const float* z0, const float* z1, const f
     return cudaGetLastError();
 }
 
-cudaError_t launch_last_norm_rows(const float* x, const int* rows, const float* w, float eps, int n, int width, void* act, int ld_act,
-                                  bool f32, cudaStream_t s) {
-    if (f32) last_norm_rows_kernel<float><<<n, 256, 0, s>>>(x, rows, w, eps, width, (float*)act, ld_act);
-    else last_norm_rows_kernel<__nv_bfloat16><<<n, 256, 0, s>>>(x, rows, w, eps, width, (__nv_bfloat16*)act, ld_act);
+cudaError_t launch_last_norm_rows(const float* x, const int* rows, const float* w, int kind, float eps, int n, int width, void* act,
+                                  int ld_act, bool f32, cudaStream_t s) {
+    if (f32) last_norm_rows_kernel<float><<<n, 256, 0, s>>>(x, rows, w, kind, eps, width, (float*)act, ld_act);
+    else last_norm_rows_kernel<__nv_bfloat16><<<n, 256, 0, s>>>(x, rows, w, kind, eps, width, (__nv_bfloat16*)act, ld_act);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_prenorm_rows(const PrenormRows& a, bool f32, cudaStream_t s) {
+    const size_t smem = (size_t)a.width * sizeof(float);
+    if (f32) prenorm_rows_kernel<float><<<a.n, 256, smem, s>>>(a);
+    else prenorm_rows_kernel<__nv_bfloat16><<<a.n, 256, smem, s>>>(a);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_head_norm_rows(int heads, int vdim, float eps, const float* norm, const float* gate, int ldg, int gate_kind, int n,
+                                  const float* o, void* act, int ld_act, bool f32, cudaStream_t s) {
+    const int grid = (n * heads + 7) / 8;
+    if (f32) head_norm_rows_kernel<float><<<grid, 256, 0, s>>>(heads, vdim, eps, norm, gate, ldg, gate_kind, n, o, (float*)act, ld_act);
+    else head_norm_rows_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(heads, vdim, eps, norm, gate, ldg, gate_kind, n, o, (__nv_bfloat16*)act, ld_act);
     return cudaGetLastError();
 }
 
@@ -493,10 +584,7 @@ cudaError_t launch_mem_rows(const MatMem& mem, const ProjCols& c, const float* p
     const size_t elems = (size_t)mem.heads * mem.dim * (mem.vdim + 1);
     mem_scan_kernel<<<(unsigned)((elems + 255) / 256), 256, 0, s>>>(mem, pos0, n, chunks, w);
     mem_out_kernel<<<dim3(chunks, mem.heads, vt), 256, 0, s>>>(mem, c.mq, c.mk, c.mv, proj, ldp, n, w);
-    const int grid = (n * mem.heads + 7) / 8;
-    if (f32) mem_norm_kernel<float><<<grid, 256, 0, s>>>(mem, c.mg, proj, ldp, n, w.o, (float*)act, ld_act);
-    else mem_norm_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(mem, c.mg, proj, ldp, n, w.o, (__nv_bfloat16*)act, ld_act);
-    return cudaGetLastError();
+    return launch_head_norm_rows(mem.heads, mem.vdim, mem.eps, mem.norm, proj + c.mg, ldp, GATE_SIGMOID, n, w.o, act, ld_act, f32, s);
 }
 
 }  // namespace mg

@@ -1,0 +1,267 @@
+// Mixture of experts: the choice (the largest router logits, weights by a softmax over them, fp32), and the chosen
+// experts.  One token streams the chosen experts' rows where they lie; a prompt's tokens are grouped by expert
+// into row tiles of 128, each tile one expert's, and go through grouped products (gemm_tc, or launch_gemm_f32).
+#include <algorithm>
+
+#include "layered_ops.cuh"
+
+namespace mg {
+
+namespace {
+
+constexpr int kThreads = 256;
+
+// One warp: the `top` largest of z[0..experts) in falling order (lower index first among equals) and the softmax
+// over them.  z is shared memory and is overwritten; sel and wt are shared memory too.  Whatever z holds,
+// the chosen indices are distinct and valid.
+__device__ __forceinline__ void choose(float* z, int experts, int top, int* sel, float* wt, int lane) {
+    unsigned taken = 0;                     // of this lane's entries lane, lane + 32, ...
+    float first = 0.f, sum = 0.f;
+    for (int k = 0; k < top; k++) {
+        int bi = -1;
+        float bv = 0.f;
+        for (int i = lane, q = 0; i < experts; i += 32, q++) {
+            const float v = z[i];
+            if (!((taken >> q) & 1u) && (bi < 0 || v > bv)) { bi = i; bv = v; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const int oi = __shfl_xor_sync(MG_FULL_MASK, bi, o);
+            const float ov = __shfl_xor_sync(MG_FULL_MASK, bv, o);
+            if (oi >= 0 && (bi < 0 || ov > bv || (!(bv > ov) && oi < bi))) { bi = oi; bv = ov; }
+        }
+        bi = __shfl_sync(MG_FULL_MASK, bi, 0);          // one answer, also where comparisons have none
+        bv = __shfl_sync(MG_FULL_MASK, bv, 0);
+        if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
+        if (k == 0) first = bv;
+        const float e = expf(bv - first);
+        sum += e;
+        if (lane == 0) { sel[k] = bi; wt[k] = e; }
+    }
+    __syncwarp();
+    for (int k = lane; k < top; k += 32) wt[k] /= sum;
+    __syncwarp();
+}
+static_assert(kMaxExperts <= 32 * 32, "a lane marks its entries in 32 bits");
+
+// Choice of one token, by the whole CTA (every CTA for itself).  zs: `experts` floats.
+__device__ __forceinline__ void choose_cta(const Moe& m, const float* router, float* zs, int* sel, float* wt) {
+    for (int i = threadIdx.x; i < m.experts; i += blockDim.x) zs[i] = router[i] + m.bias[i];
+    __syncthreads();
+    if (threadIdx.x < 32) choose(zs, m.experts, m.top, sel, wt, threadIdx.x);
+    __syncthreads();
+}
+
+// mid[k][row] = silu(gate row . h) * (up row . h) of the chosen experts: a warp per (expert, row).
+__global__ void __launch_bounds__(kThreads) moe_up_kernel(const MoeStep a) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ int sel[kMaxTop];
+    __shared__ float wt[kMaxTop];
+    const Moe& m = a.moe;
+    float* hs = smem;                       // [ldw]
+    float* zs = smem + m.ldw;               // [experts]
+    pdl_launch_dependents();
+    pdl_wait();
+    for (int i = threadIdx.x; i < m.ldw; i += kThreads) hs[i] = i < m.width ? a.h[i] : 0.f;
+    choose_cta(m, a.router, zs, sel, wt);
+    const int lane = threadIdx.x & 31, nw = gridDim.x * (kThreads / 32), chunks = m.ldw / 8, items = m.top * m.ff;
+    for (int it = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5); it < items; it += nw) {
+        const int k = it / m.ff;
+        const size_t row = (size_t)sel[k] * m.ff + (it - k * m.ff);
+        const uint4* g = reinterpret_cast<const uint4*>(m.gate + row * m.ldw * 2);
+        const uint4* u = reinterpret_cast<const uint4*>(m.up + row * m.ldw * 2);
+        float sg = 0.f, su = 0.f;
+        for (int c0 = 0; c0 < chunks; c0 += 128) {
+            uint4 wg[4], wu[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const int c = c0 + i * 32 + lane;
+                wg[i] = c < chunks ? ld_stream16(g + c) : make_uint4(0u, 0u, 0u, 0u);
+                wu[i] = c < chunks ? ld_stream16(u + c) : make_uint4(0u, 0u, 0u, 0u);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const int c = c0 + i * 32 + lane;
+                if (c < chunks) {
+                    const float4 x[2] = {*reinterpret_cast<const float4*>(hs + c * 8), *reinterpret_cast<const float4*>(hs + c * 8 + 4)};
+                    sg += Chunk<FMT_BF16>::dot(wg[i], x);
+                    su += Chunk<FMT_BF16>::dot(wu[i], x);
+                }
+            }
+        }
+        sg = warp_sum(sg);
+        su = warp_sum(su);
+        if (lane == 0) a.mid[it] = silu(sg) * su;
+    }
+}
+
+// out[row] = sum over the chosen experts of weight * (down row . mid) + gate * (shared down row . its mid): the
+// factors go into the staged vectors, a warp per output row.
+template <int R>
+__global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeStep a) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ int sel[kMaxTop];
+    __shared__ float wt[kMaxTop];
+    const Moe& m = a.moe;
+    float* xs = smem;                                   // [top * ffs + shared_ffs]
+    float* zs = smem + m.top * m.ffs + m.shared_ffs;    // [experts]
+    const int lane = threadIdx.x & 31;
+    pdl_launch_dependents();
+    pdl_wait();
+    choose_cta(m, a.router, zs, sel, wt);
+    for (int k = 0; k < m.top; k++)
+        for (int i = threadIdx.x; i < m.ffs; i += kThreads) xs[k * m.ffs + i] = i < m.ff ? a.mid[k * m.ff + i] * wt[k] : 0.f;
+    if (m.shared_ff) {
+        const float sg = sigmoid(a.router[m.sg_col()]);
+        const float *g = a.router + m.sg_col() + 1, *u = g + m.shared_ff;
+        for (int i = threadIdx.x; i < m.shared_ffs; i += kThreads) xs[m.top * m.ffs + i] = i < m.shared_ff ? silu(g[i]) * u[i] * sg : 0.f;
+    }
+    __syncthreads();
+    const int nw = gridDim.x * (kThreads / 32);
+    for (int r0 = (blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5)) * R; r0 < m.width; r0 += nw * R) {
+        float acc[R] = {};
+        for (int k = 0; k < m.top + (m.shared_ff ? 1 : 0); k++) {
+            const bool sh = k == m.top;
+            const int ld = sh ? m.shared_ffs : m.ffs, chunks = ld / 8;
+            const uint8_t* w = sh ? m.shared_down : m.down + (size_t)sel[k] * m.width * ld * 2;
+            const float* x0 = xs + k * m.ffs;
+            const uint4* row[R];
+#pragma unroll
+            for (int r = 0; r < R; r++) row[r] = reinterpret_cast<const uint4*>(w + (size_t)min(r0 + r, m.width - 1) * ld * 2);
+            for (int c0 = 0; c0 < chunks; c0 += 128) {
+                uint4 ww[R][4];
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+#pragma unroll
+                    for (int r = 0; r < R; r++) {
+                        const int c = c0 + i * 32 + lane;
+                        ww[r][i] = c < chunks ? ld_stream16(row[r] + c) : make_uint4(0u, 0u, 0u, 0u);
+                    }
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    const int c = c0 + i * 32 + lane;
+                    if (c < chunks) {
+                        const float4 x[2] = {*reinterpret_cast<const float4*>(x0 + c * 8), *reinterpret_cast<const float4*>(x0 + c * 8 + 4)};
+#pragma unroll
+                        for (int r = 0; r < R; r++) acc[r] += Chunk<FMT_BF16>::dot(ww[r][i], x);
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const float v = warp_sum(acc[r]);
+            if (lane == 0 && r0 + r < m.width) a.out[r0 + r] = v;
+        }
+    }
+}
+
+// ---- prompts ----
+
+// A warp per token: choice, and the token's place among those of its expert.
+__global__ void __launch_bounds__(kThreads) moe_choose_kernel(const Moe m, const float* router, int ldr, int n, MoeRows w) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ int sel[kThreads / 32][kMaxTop];
+    __shared__ float wt[kThreads / 32][kMaxTop];
+    const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * (kThreads / 32) + wid;
+    if (t >= n) return;
+    float* z = smem + wid * m.experts;
+    for (int i = lane; i < m.experts; i += 32) z[i] = router[(size_t)t * ldr + i] + m.bias[i];
+    __syncwarp();
+    choose(z, m.experts, m.top, sel[wid], wt[wid], lane);
+    for (int k = lane; k < m.top; k += 32) {
+        const int e = sel[wid][k];
+        w.sel[(size_t)t * m.top + k] = e;
+        w.weight[(size_t)t * m.top + k] = wt[wid][k];
+        w.slot[(size_t)t * m.top + k] = atomicAdd(w.count + e, 1);      // which place a token gets does not change its result
+    }
+}
+
+// One CTA: first row of every expert (whole tiles of 128), the expert of every tile; clears the counts.
+__global__ void __launch_bounds__(1024) moe_plan_kernel(const Moe m, MoeRows w) {
+    __shared__ int tiles[kMaxExperts], first[kMaxExperts + 1];
+    for (int e = threadIdx.x; e < m.experts; e += blockDim.x) {
+        tiles[e] = (w.count[e] + 127) / 128;
+        w.count[e] = 0;
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int at = 0;
+        for (int e = 0; e < m.experts; e++) { first[e] = at; at += tiles[e]; }
+        first[m.experts] = at;
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < m.experts; e += blockDim.x) {
+        w.first[e] = first[e] * 128;
+        for (int i = first[e]; i < first[e + 1] && i < w.tiles; i++) w.group[i] = e;
+    }
+    for (int i = first[m.experts] + threadIdx.x; i < w.tiles; i += blockDim.x) w.group[i] = -1;
+}
+
+// A CTA per token: its row to its place in every chosen expert's group; slot becomes the grouped row.
+__global__ void __launch_bounds__(128) moe_gather_kernel(const Moe m, const uint4* act, int units, MoeRows w) {
+    const size_t t = blockIdx.x;
+    for (int k = 0; k < m.top; k++) {
+        const size_t at = t * m.top + k;
+        const int row = w.first[w.sel[at]] + w.slot[at];
+        uint4* dst = static_cast<uint4*>(w.x) + (size_t)row * units;
+        for (int i = threadIdx.x; i < units; i += 128) dst[i] = act[t * units + i];
+    }
+}
+
+__global__ void __launch_bounds__(kThreads) moe_combine_kernel(const Moe m, const float* router, int ldr, MoeRows w, float* z) {
+    __shared__ float wt[kMaxTop];
+    __shared__ int row[kMaxTop];
+    const size_t t = blockIdx.x;
+    for (int k = threadIdx.x; k < m.top; k += kThreads) {
+        wt[k] = w.weight[t * m.top + k];
+        row[k] = w.first[w.sel[t * m.top + k]] + w.slot[t * m.top + k];
+    }
+    __syncthreads();
+    const float sg = m.shared_ff ? sigmoid(router[t * ldr + m.sg_col()]) : 0.f;
+    float* out = z + t * m.width;
+    for (int i = threadIdx.x; i < m.width; i += kThreads) {
+        float v = m.shared_ff ? sg * out[i] : 0.f;
+#pragma unroll 4
+        for (int k = 0; k < m.top; k++) v = fmaf(wt[k], w.y[(size_t)row[k] * m.width + i], v);
+        out[i] = v;
+    }
+}
+
+constexpr int kDownRows = 2;
+
+}  // namespace
+
+size_t moe_step_smem(const Moe& m) {
+    return (size_t)(std::max(m.ldw, m.top * m.ffs + m.shared_ffs) + m.experts) * sizeof(float);
+}
+
+cudaError_t moe_step_attrs(size_t bytes) {
+    cudaError_t c = cudaFuncSetAttribute((const void*)moe_up_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+    return c != cudaSuccess ? c : cudaFuncSetAttribute((const void*)moe_down_kernel<kDownRows>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+}
+
+cudaError_t launch_moe_up(const MoeStep& a, int sms, bool pdl, cudaStream_t s) {
+    const int grid = std::min((a.moe.top * a.moe.ff + 7) / 8, 2 * sms);
+    return launch_pdl(moe_up_kernel, grid, kThreads, (size_t)(a.moe.ldw + a.moe.experts) * sizeof(float), pdl, s, a);
+}
+
+cudaError_t launch_moe_down(const MoeStep& a, int sms, bool pdl, cudaStream_t s) {
+    const Moe& m = a.moe;
+    const int grid = std::min((m.width + 8 * kDownRows - 1) / (8 * kDownRows), 2 * sms);
+    return launch_pdl(moe_down_kernel<kDownRows>, grid, kThreads, (size_t)(m.top * m.ffs + m.shared_ffs + m.experts) * sizeof(float), pdl, s, a);
+}
+
+cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s) {
+    moe_choose_kernel<<<(n + 7) / 8, kThreads, (size_t)8 * m.experts * sizeof(float), s>>>(m, router, ldr, n, w);
+    moe_plan_kernel<<<1, 1024, 0, s>>>(m, w);
+    moe_gather_kernel<<<n, 128, 0, s>>>(m, (const uint4*)act, m.ldw * (f32 ? 4 : 2) / 16, w);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, cudaStream_t s) {
+    moe_combine_kernel<<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
+    return cudaGetLastError();
+}
+
+}  // namespace mg

@@ -11,9 +11,11 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
+import numpy as np
+
 from .configs import CONFIGS, ModelConfig
-from .layered import (MATH, EMBED, FINAL_NORM, HEAD, LAYER_SLOTS, SLOTS, GateAttention, LayeredConfig, LayeredInference,
-                      MatrixMemory, ParallelLayer, slot_shapes)
+from .layered import (MATH, NORM_LAYER, POS_NONE, GateAttention, LatentAttention, LayeredConfig, LayeredInference, Loop,
+                      MatrixMemory, MixtureOfExperts, ParallelLayer, PrenormLayer, Wkv, slot_shapes)
 from .safetensors import SafeTensors
 
 
@@ -25,7 +27,8 @@ class ConfigError(ValueError):
 class Architecture:
     name: str
     family: str                                     # library family that serves it (build.FAMILIES)
-    read_config: Callable[[dict], object]           # config.json -> configuration
+    # config.json, and a function that gives a tensor's shape -> configuration
+    read_config: Callable[[dict, Callable[[str], tuple[int, ...]]], object]
     load_weights: Callable[[object, SafeTensors], None]
 
 
@@ -96,7 +99,83 @@ def mitotar_weights(engine: LayeredInference, st: SafeTensors) -> None:
         engine.SetWeightBF16(idx, bits)
 
 
-register(Architecture("Mitotar", "layered", mitotar_config, mitotar_weights))
+register(Architecture("Mitotar", "layered", lambda j, shape: mitotar_config(j), mitotar_weights))
+
+
+# ---- Kuzipel --------------------------------------------------------------------------------------
+
+def kuzipel_config(j: dict, shape: Callable[[str], tuple[int, ...]]) -> LayeredConfig:
+    """The rank of a recurrent layer's decay is known from its tensor only."""
+    layers = []
+    for i, l in enumerate(_get(j, "layers", "config")):
+        where = f"layer {i}"
+        kind, m = _get(l, "type", where), _get(l, "mixer", where)
+        if kind == "latent_attention":
+            rot = _get(m, "rot", where)
+            rot_dim = int(_get(m, "rot_dim", where))
+            if rot.get("dims", rot_dim) != rot_dim or rot_dim < 2 or rot_dim % 2:
+                raise ConfigError(f"{where}: the rotated part has rot_dim {rot_dim} dimensions, rot.dims {rot.get('dims')} of them rotated")
+            dim = int(_get(m, "dim", where))
+            mixer = LatentAttention(heads=int(_get(m, "heads", where)), dim=dim, rot_dim=rot_dim, vdim=int(m.get("vdim", dim)),
+                                    q_rank=int(_get(m, "q_rank", where)), kv_rank=int(_get(m, "kv_rank", where)),
+                                    scale=float(_get(m, "scale", where)), rot_base=float(_get(rot, "base", where)))
+        elif kind == "wkv":
+            mixer = Wkv(heads=int(_get(m, "heads", where)), dim=int(_get(m, "dim", where)), decay_rank=int(shape(f"l{i}.mix.w1")[0]))
+        else:
+            raise ConfigError(f"{where}: mixer type {kind!r} is not known")
+        mlp = l.get("mlp")
+        moe = None
+        if mlp:
+            if mlp.get("kind", "moe") != "moe":
+                raise ConfigError(f"{where}: feed-forward kind {mlp['kind']!r} is not known")
+            router, shared = _get(mlp, "router", where), mlp.get("shared")
+            moe = MixtureOfExperts(experts=int(_get(router, "experts", where)), top=int(_get(router, "top", where)),
+                                   ff=int(_get(_get(mlp, "expert", where), "ff", where)), shared_ff=int(_get(shared, "ff", where)) if shared else 0)
+            if not 1 <= moe.top <= moe.experts:
+                raise ConfigError(f"{where}: {moe.top} of {moe.experts} experts cannot be chosen")
+        layers.append(PrenormLayer(mixer, moe))
+    loop = j.get("loop")
+    if loop:
+        loop = Loop(int(_get(loop, "start", "loop")), int(_get(loop, "stop", "loop")), int(_get(loop, "times", "loop")))
+        if not 0 <= loop.start < loop.stop <= len(layers) or loop.times < 1:
+            raise ConfigError(f"loop: layers {loop.start} to {loop.stop} of {len(layers)}, {loop.times} times")
+    return LayeredConfig(name="Kuzipel", width=int(_get(j, "width", "config")), vocab=int(_get(j, "vocab", "config")), layers=tuple(layers),
+                         norm_eps=float(_get(_get(j, "norm", "config"), "eps", "norm")), norm=NORM_LAYER, positions=POS_NONE,
+                         residual_mult=float(j.get("residual_mult", 1.0)), loop=loop or None)
+
+
+# slot -> tensor name under the layer's prefix; {e} stands for an expert
+KUZIPEL_TENSORS = {
+    "norm1": "norm1", "norm2": "norm2", "ls1": "ls1", "ls2": "ls2",
+    "la.dq": "mix.dq", "la.dq_norm": "mix.dq.norm", "la.uq": "mix.uq", "la.dkv": "mix.dkv", "la.dkv_norm": "mix.dkv.norm",
+    "la.uk": "mix.uk", "la.uv": "mix.uv", "la.o": "mix.o",
+    **{f"wkv.mu_{t}": f"mix.mu.{t}" for t in "rkvgw"},
+    **{f"wkv.{t}": f"mix.{t}" for t in ("r", "k", "v", "g", "w1", "w2", "w0", "u", "norm", "o")},
+    "moe.router": "mlp.router", "moe.bias": "mlp.router.b", "moe.gate": "mlp.e{e}.gate", "moe.up": "mlp.e{e}.up", "moe.down": "mlp.e{e}.down",
+    "shared.gate": "mlp.shared.gate", "shared.up": "mlp.shared.up", "shared.down": "mlp.shared.down", "shared.sg": "mlp.shared.sg",
+}
+KUZIPEL_GLOBALS = {"embed": "embed", "final_norm": "final.norm", "head": "head", "loop_in": "loop.in"}
+
+
+def kuzipel_tensors(cfg: LayeredConfig, slot_name: str, layer: int) -> list[str]:
+    """The tensors a slot holds, stacked one below the other."""
+    if layer < 0:
+        return [KUZIPEL_GLOBALS[slot_name]]
+    t = f"l{layer}.{KUZIPEL_TENSORS[slot_name]}"
+    return [t.format(e=e) for e in range(cfg.layers[layer].moe.experts)] if "{e}" in t else [t]
+
+
+def kuzipel_weights(engine: LayeredInference, st: SafeTensors) -> None:
+    for idx, name, layer, rows, cols in slot_shapes(engine.cfg):
+        names = kuzipel_tensors(engine.cfg, name, layer)
+        parts = [st.bf16_bits(t) for t in names]
+        for t, b in zip(names, parts):
+            if (b.shape != (rows // len(names), cols)) if rows else (b.size != cols):
+                raise ConfigError(f"{t}: shape {b.shape} does not fit the configuration ({rows // len(names)} x {cols})")
+        engine.SetWeightBF16(idx, parts[0] if len(parts) == 1 else np.concatenate(parts))
+
+
+register(Architecture("Kuzipel", "layered", kuzipel_config, kuzipel_weights))
 
 
 # ---- loading ----------------------------------------------------------------------------------------
@@ -109,7 +188,16 @@ def read_config(folder: str):
     if name not in ARCHITECTURES:
         raise ConfigError(f"{folder}: architecture {name!r} is not registered (known: {', '.join(sorted(ARCHITECTURES))})")
     arch = ARCHITECTURES[name]
-    return arch, arch.read_config(j)
+    weights: list[SafeTensors] = []
+
+    def shape(tensor: str) -> tuple[int, ...]:
+        if not weights:
+            weights.append(SafeTensors(os.path.join(folder, "model.safetensors")))
+        if tensor not in weights[0]:
+            raise ConfigError(f"{folder}: no tensor {tensor!r}")
+        return weights[0].shape(tensor)
+
+    return arch, arch.read_config(j, shape)
 
 
 def create_engine(cfg, device: int = 0):

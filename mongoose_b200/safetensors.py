@@ -35,6 +35,9 @@ class SafeTensors:
     def dtype(self, name: str) -> str:
         return self._index[name]["dtype"]
 
+    def shape(self, name: str) -> tuple[int, ...]:
+        return tuple(self._index[name]["shape"])
+
     def __getitem__(self, name: str) -> np.ndarray:
         if name not in self._index:
             raise KeyError(f"{self.path} holds no tensor {name!r}")

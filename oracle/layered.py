@@ -119,9 +119,8 @@ def feed_forward(h, w):
     return gelu_tanh(h @ w["up"].T) @ w["down"].T
 
 
-def forward(cfg: dict, weights: dict, tokens, layers_out: list | None = None) -> np.ndarray:
-    """Logits [n, vocab] of the whole sequence at once."""
-    w = {k: np.asarray(v, np.float64) for k, v in weights.items()}
+def parallel_layers(cfg, w, tokens, layers_out):
+    """The residual stream behind post-normed layers of two branches (Mitotar)."""
     eps, width = cfg["norm"]["eps"], cfg["width"]
     x = w["embed"][np.asarray(tokens)] + np.stack([sinusoid(p, width) for p in range(len(tokens))])
     for i, layer in enumerate(cfg["layers"]):
@@ -132,4 +131,139 @@ def forward(cfg: dict, weights: dict, tokens, layers_out: list | None = None) ->
             x = x + rms_norm(feed_forward(x, under(lw, "mlp.")), lw["norm2"], eps, around_zero=True)
         if layers_out is not None:
             layers_out.append(x.copy())
-    return rms_norm(x, w["final.norm"], eps, around_zero=True) @ w["head"].T
+    return rms_norm(x, w["final.norm"], eps, around_zero=True)
+
+
+# ---- Kuzipel ---------------------------------------------------------------------------------------
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def layer_norm(x, w, eps):
+    d = x - np.mean(x, axis=-1, keepdims=True)
+    return d / np.sqrt(np.mean(d * d, axis=-1, keepdims=True) + eps) * w
+
+
+def rotate(x, p, base):
+    """Rotary positions over the whole last axis, element i with element i + half; p one position per row."""
+    half = x.shape[-1] // 2
+    a = np.asarray(p, np.float64)[:, None] * base ** (-2.0 * np.arange(half) / (2 * half))
+    a = a.reshape(a.shape[0], *[1] * (x.ndim - 2), half)
+    u, v = x[..., :half], x[..., half:]
+    return np.concatenate([u * np.cos(a) - v * np.sin(a), v * np.cos(a) + u * np.sin(a)], axis=-1)
+
+
+def softmax(z):
+    e = np.exp(z - np.max(z, axis=-1, keepdims=True))
+    return e / np.sum(e, axis=-1, keepdims=True)
+
+
+def causal_softmax(s):
+    n = s.shape[-1]
+    return softmax(np.where(np.arange(n)[None] <= np.arange(n)[:, None], s, -np.inf))
+
+
+def latent_attention(h, w, p, eps):
+    """Queries, keys and values through low-rank latents; one rotated key part for all heads."""
+    n, H, D, R, C = h.shape[0], p["heads"], p["dim"], p["rot_dim"], p["kv_rank"]
+    pos = np.arange(n)
+    q = (rms_norm(h @ w["dq"].T, w["dq.norm"], eps) @ w["uq"].T).reshape(n, H, D + R)
+    down = h @ w["dkv"].T
+    c = rms_norm(down[:, :C], w["dkv.norm"], eps)
+    kr = rotate(down[:, C:], pos, p["rot"]["base"])
+    qr = rotate(q[..., D:], pos, p["rot"]["base"])
+    k = (c @ w["uk"].T).reshape(n, H, D)
+    v = (c @ w["uv"].T).reshape(n, H, p["vdim"])
+    out = np.empty((n, H, p["vdim"]))
+    for a in range(H):
+        out[:, a] = causal_softmax((q[:, a, :D] @ k[:, a].T + qr[:, a] @ kr.T) * p["scale"]) @ v[:, a]
+    return out.reshape(n, -1) @ w["o"].T
+
+
+def token_shift(h, mu):
+    """Each token's vector moved by mu towards the one before it (zeros before the first)."""
+    before = np.concatenate([np.zeros_like(h[:1]), h[:-1]])
+    return h + (before - h) * mu
+
+
+def channel_decay(z, w1, w2, w0):
+    return np.exp(-np.exp(np.tanh(z @ w1.T) @ w2.T + w0))
+
+
+def wkv_step(S, r, k, v, w, u):
+    """One token of one head.  S [key channel, value channel]."""
+    kv = np.outer(k, v)
+    o = (S + u[:, None] * kv).T @ r
+    return w[:, None] * S + kv, o
+
+
+def wkv(h, w, p, eps):
+    n, H, D = h.shape[0], p["heads"], p["dim"]
+    mixed = {t: token_shift(h, w["mu." + t]) for t in "rkvgw"}
+    r, k, v = ((mixed[t] @ w[t].T).reshape(n, H, D) for t in "rkv")
+    d = channel_decay(mixed["w"], w["w1"], w["w2"], w["w0"]).reshape(n, H, D)
+    u = w["u"].reshape(H, D)
+    out = np.empty((n, H, D))
+    for a in range(H):
+        S = np.zeros((D, D))
+        for t in range(n):
+            S, out[t, a] = wkv_step(S, r[t, a], k[t, a], v[t, a], d[t, a], u[a])
+    y = unit_rms(out, eps).reshape(n, H * D) * w["norm"] * silu(mixed["g"] @ w["g"].T)
+    return y @ w["o"].T
+
+
+def glu(h, w):
+    return (silu(h @ w["gate"].T) * (h @ w["up"].T)) @ w["down"].T
+
+
+def route(z, top):
+    """Weights [n, experts]: softmax over the `top` largest logits of each row, zero elsewhere."""
+    out = np.zeros_like(z)
+    for t in range(z.shape[0]):
+        chosen = np.argsort(-z[t], kind="stable")[:top]
+        out[t, chosen] = softmax(z[t, chosen])
+    return out
+
+
+def mixture(h, w, p):
+    g = route(h @ w["router"].T + w["router.b"], p["router"]["top"])
+    y = sum(g[:, [e]] * glu(h, under(w, f"e{e}.")) for e in range(p["router"]["experts"]))
+    return y + sigmoid(h @ w["shared.sg"].T) * glu(h, under(w, "shared."))
+
+
+def layer_runs(n_layers, loop):
+    """(layer, does a pass of the loop begin before it) in the order of computation."""
+    if not loop:
+        return [(i, False) for i in range(n_layers)]
+    a, b = loop["start"], loop["stop"]
+    body = [(i, i == a) for i in range(a, b)]
+    return [(i, False) for i in range(a)] + body * loop["times"] + [(i, False) for i in range(b, n_layers)]
+
+
+MIXERS = {"latent_attention": latent_attention, "wkv": wkv}
+
+
+def prenorm_layers(cfg, w, tokens, layers_out):
+    """The residual stream behind pre-normed layers with layer scale, some of them in a loop (Kuzipel)."""
+    eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
+    x0 = x = w["embed"][np.asarray(tokens)]
+    for i, begins in layer_runs(len(cfg["layers"]), cfg.get("loop")):
+        if begins:
+            x = np.concatenate([x, x0], axis=-1) @ w["loop.in"].T
+        layer, lw = cfg["layers"][i], under(w, f"l{i}.")
+        x = x + m * lw["ls1"] * MIXERS[layer["type"]](layer_norm(x, lw["norm1"], eps), under(lw, "mix."), layer["mixer"], eps)
+        if layer.get("mlp"):
+            x = x + m * lw["ls2"] * mixture(layer_norm(x, lw["norm2"], eps), under(lw, "mlp."), layer["mlp"])
+        if layers_out is not None:
+            layers_out.append(x.copy())
+    return layer_norm(x, w["final.norm"], eps)
+
+
+DESIGNS = {"Mitotar": parallel_layers, "Kuzipel": prenorm_layers}
+
+
+def forward(cfg: dict, weights: dict, tokens, layers_out: list | None = None) -> np.ndarray:
+    """Logits [n, vocab] of the whole sequence at once."""
+    w = {k: np.asarray(v, np.float64) for k, v in weights.items()}
+    return DESIGNS[cfg.get("architecture", "Mitotar")](cfg, w, tokens, layers_out) @ w["head"].T
