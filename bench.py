@@ -67,6 +67,10 @@ WORKLOADS = {
     "mitotar-0.5b": synthetic.LAYERED["mitotar-0.5b"],
     "mitotar-1.1b": synthetic.LAYERED["mitotar-1.1b"],
     "mitotar-7b-width-4l": synthetic.LAYERED["mitotar-7b-width-4l"],
+    # the same for random-init Kuzipel, beside Mitotar of equal width and depth
+    "kuzipel-0.5b": synthetic.LAYERED["kuzipel-0.5b"],
+    "kuzipel-1.1b": synthetic.LAYERED["kuzipel-1.1b"],
+    "kuzipel-7b-width-4l": synthetic.LAYERED["kuzipel-7b-width-4l"],
     # the single-op configuration: one Q8_0 dequant-matvec, W 4864 x 896 in raw 34-byte blocks
     "q8_0-matvec-4864x896": None,
 }
@@ -82,9 +86,9 @@ def parse_args():
     ap.add_argument("--workload", default="qwen2.5-0.5b-q8_0-b1", choices=sorted(WORKLOADS))
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN)
     ap.add_argument("--sequences", type=int, default=8, help="sequences of the *-seqs workload (full config: 64)")
-    ap.add_argument("--contexts", default="512,4000", help="positions before the timed decode steps of the mitotar-* workloads")
-    ap.add_argument("--prefill", type=int, default=2048, help="tokens of the timed prompt portion of the mitotar-* workloads")
-    ap.add_argument("--no-closest", action="store_true", help="skip the dense model beside a mitotar-* workload")
+    ap.add_argument("--contexts", default="512,4000", help="positions before the timed decode steps of the mitotar-* and kuzipel-* workloads")
+    ap.add_argument("--prefill", type=int, default=2048, help="tokens of the timed prompt portion of the mitotar-* and kuzipel-* workloads")
+    ap.add_argument("--no-closest", action="store_true", help="skip the dense model or Mitotar model beside a mitotar-* or kuzipel-* workload")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-e2e", action="store_true", help="skip the host-buffer leg (profiling runs)")
     ap.add_argument("--cpu-steps", type=int, default=0, help="steps of the CPU baseline sample (0 = auto)")
@@ -751,26 +755,18 @@ def timed_decode(torch, eng, context, tok, steps, warm, local_rank):
     return ev0.elapsed_time(ev1) / steps
 
 
-def run_layered_workload(args, cfg, local_rank):
-    """Prefill of one portion and greedy decode at several contexts, random-init weights.  A step is one
-    decode token at the first context; `closest` is the dense model of the same widths (Q8_0 on its
-    default path, prompts fed token by token as it does)."""
-    import torch
+def measure_layered(args, torch, cfg, local_rank, sampler, with_e2e):
+    """Prefill of one portion, greedy decode at several contexts, and steps through the public call."""
     from mongoose_b200 import layered
-    from mongoose_b200.fused_infer import CUDAFusedInference
-    if not torch.cuda.is_available():
-        raise SystemExit("bench.py needs a CUDA device: there is no CPU fallback for this path")
-    torch.cuda.set_device(local_rank)
     K, W, P = args.steps, max(args.warmup, 3), args.prefill
     contexts = [int(c) for c in args.contexts.split(",")]
     cfg = cfg.with_(max_seq=max(max(contexts) + W + K, P))
     eng = layered.LayeredInference(cfg, device=local_rank)
     synthetic.load_layered(eng, seed=0)
     toks = synthetic.prompt_ids(0, max(max(contexts), P), cfg.vocab)
-    peak, peak_src = measured_peak_gbs()
+    peak, _ = measured_peak_gbs()
     tf_peak, _ = measured_peak_tflops()
     stream = torch.cuda.ExternalStream(eng.stream, device=local_rank)
-    sampler = ClockSampler(local_rank)
     sampler.start()
 
     # ---- prefill: the portion from position 0, through the public call (token ids in, no logits out) ----
@@ -799,29 +795,56 @@ def run_layered_workload(args, cfg, local_rank):
     decode = []
     for c in contexts:
         eng.Forward(toks[:c], 0)
+        launches0 = eng.LaunchCount()
         sampler.begin()
         ms = timed_decode(torch, eng, c, int(toks[0]), K, W, local_rank)
         sampler.end()
         b = (layered.weight_bytes_per_token(cfg) + 2 * layered.state_bytes(cfg) +
              layered.cache_bytes_per_position(cfg) * (c + W + (K + 1) / 2.0))
         decode.append({"context": c, "value": 1e3 / ms, "unit": "tok/s", "ms_per_step": ms, "bytes_per_token": b,
-                       "GB/s": b / ms / 1e6, "frac_of_hbm": b / ms / 1e6 / peak})
+                       "GB/s": b / ms / 1e6, "frac_of_hbm": b / ms / 1e6 / peak, "launches": (eng.LaunchCount() - launches0) * K // (K + W)})
 
     # ---- end to end: token id in, logits out to the host, every step ----
-    eng.Forward(toks[:contexts[0]], 0)
-    logits = torch.empty(cfg.vocab, dtype=torch.float32).pin_memory()
-    for i in range(W):
-        eng.StepToken(int(toks[i]), contexts[0] + i, logits)
-    t0 = time.perf_counter()
-    for i in range(W, W + K):
-        eng.StepToken(int(toks[i % len(toks)]), contexts[0] + i, logits)
-    e2e = (time.perf_counter() - t0) / K
-    clocks = sampler.stop()
+    e2e = None
+    if with_e2e:
+        eng.Forward(toks[:contexts[0]], 0)
+        logits = torch.empty(cfg.vocab, dtype=torch.float32).pin_memory()
+        for i in range(W):
+            eng.StepToken(int(toks[i]), contexts[0] + i, logits)
+        t0 = time.perf_counter()
+        for i in range(W, W + K):
+            eng.StepToken(int(toks[i % len(toks)]), contexts[0] + i, logits)
+        e2e = (time.perf_counter() - t0) / K
     eng.close()
+    return prefill, decode, e2e
 
+
+def run_layered_workload(args, cfg, local_rank):
+    """Prefill of one portion and greedy decode at several contexts, random-init weights.  A step is one
+    decode token at the first context; `closest` is the dense model of the same widths (Q8_0 on its
+    default path, prompts fed token by token as it does), for Kuzipel the Mitotar model of the same widths."""
+    import torch
+    from mongoose_b200 import layered
+    from mongoose_b200.fused_infer import CUDAFusedInference
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: there is no CPU fallback for this path")
+    torch.cuda.set_device(local_rank)
+    K, W = args.steps, max(args.warmup, 3)
+    contexts = [int(c) for c in args.contexts.split(",")]
+    peak, peak_src = measured_peak_gbs()
+    sampler = ClockSampler(local_rank)
+    prefill, decode, e2e = measure_layered(args, torch, cfg, local_rank, sampler, True)
+    clocks = sampler.stop()
+
+    design, size = args.workload.split("-", 1)
     closest = None
-    if not args.no_closest:
-        d = {"mitotar-0.5b": mc.QWEN25_05B, "mitotar-1.1b": mc.TINYLLAMA_11B, "mitotar-7b-width-4l": TP_LEG_CFG}[args.workload]
+    if not args.no_closest and design == "kuzipel":
+        like = synthetic.LAYERED["mitotar-" + size]
+        sampler = ClockSampler(local_rank)
+        p, d, _ = measure_layered(args, torch, like.with_(layers=like.layers[:1] * len(cfg.runs())), local_rank, sampler, False)
+        closest = {"model": like.name, "layers": len(cfg.runs()), "format": "bf16", "prefill": p, "decode": d, "clocks": sampler.stop()}
+    elif not args.no_closest:
+        d = {"0.5b": mc.QWEN25_05B, "1.1b": mc.TINYLLAMA_11B, "7b-width-4l": TP_LEG_CFG}[size]
         d = d.with_(max_seq=contexts[0] + W + K)
         eng = CUDAFusedInference(d, device=local_rank)
         synthetic.load_engine(eng, d, seed=0)
@@ -845,13 +868,13 @@ def run_layered_workload(args, cfg, local_rank):
         "metric": "decode_tokens_per_s", "value": decode[0]["value"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
         "ms_per_step": decode[0]["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
         "data": "synthetic",
-        "config": {"workload": args.workload, "width": cfg.width, "layers": cfg.n_layers, "vocab": cfg.vocab, "batch": 1,
+        "config": {"workload": args.workload, "width": cfg.width, "layers": len(cfg.runs()), "vocab": cfg.vocab, "batch": 1,
                    "context": contexts[0], "l2": "inputs larger than L2 (weights streamed per token: %d MB)" % (layered.weight_bytes_per_token(cfg) // 2 ** 20),
                    "timing": "CUDA events on the engine stream"},
         "prefill": prefill, "decode": decode, "closest": closest,
         "e2e": {"value": 1.0 / e2e, "unit": "tok/s", "h2d_bytes_per_step": 8, "d2h_bytes_per_step": cfg.vocab * 4 + 4,
                 "api": "StepToken(token, pos, logitsOut) with a pinned host buffer"},
-        "peak_source": peak_src, "clocks": clocks}), flush=True)
+        "gpu_launches": decode[0]["launches"], "peak_source": peak_src, "clocks": clocks}), flush=True)
 
 
 def main():

@@ -50,17 +50,6 @@ struct Geo {
     static constexpr int bytes = body + 1024 + 256 + talk_bytes + (2 * HP + bn * HP) * 4;
 };
 
-__device__ __forceinline__ unsigned long long pack2(float a, float b) {
-    return (unsigned long long)__float_as_uint(a) | ((unsigned long long)__float_as_uint(b) << 32);
-}
-__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-    unsigned long long d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ float lo(unsigned long long v) { return __uint_as_float((unsigned)v); }
-__device__ __forceinline__ float hi(unsigned long long v) { return __uint_as_float((unsigned)(v >> 32)); }
-
 // 1 / (1 + 2^t)
 __device__ __forceinline__ float sigmoid_of_exp2(float t) {
     float e, r;

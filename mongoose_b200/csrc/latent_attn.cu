@@ -129,21 +129,26 @@ __global__ void __launch_bounds__(kThreads) latent_attend_kernel(const LatentSte
     const Attend<KT> sm(A, a.group, a.tile, smem);
     const int row = A.row(), chunks = row / CN, tile = a.tile, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const KT* cache = static_cast<const KT*>(A.cache);
-    auto load = [&](int buf, int j) {               // rows past the range are zero
+    auto load = [&](int buf, int j) {               // a warp per row; rows past the range are zero
         KT* dst = sm.k + (size_t)buf * tile * sm.ks;
-        for (int i = threadIdx.x; i < tile * chunks; i += kThreads) {
-            const int p = i / chunks, c = i - p * chunks;
-            if (j + p < j1) cp_async16(dst + p * sm.ks + c * CN, cache + (size_t)(j + p) * row + c * CN);
-            else *reinterpret_cast<uint4*>(dst + p * sm.ks + c * CN) = make_uint4(0u, 0u, 0u, 0u);
-        }
+        for (int p = wid; p < tile; p += kThreads / 32)
+            for (int c = lane; c < chunks; c += 32) {
+                if (j + p < j1) cp_async16(dst + p * sm.ks + c * CN, cache + (size_t)(j + p) * row + c * CN);
+                else *reinterpret_cast<uint4*>(dst + p * sm.ks + c * CN) = make_uint4(0u, 0u, 0u, 0u);
+            }
     };
+    const float* qa = a.qa + ((size_t)t * A.heads + h0) * row;
+    for (int h = wid; h < G; h += kThreads / 32)
+        for (int c = lane * 4; c < row; c += 128) cp_async16(sm.q + h * sm.qs + c, qa + (size_t)h * row + c);
     load(0, j0);
     cp_async_commit();
-    const float* qa = a.qa + ((size_t)t * A.heads + h0) * row;
-    for (int i = threadIdx.x; i < G * row; i += kThreads) sm.q[i / row * sm.qs + i % row] = qa[i];
     for (int i = threadIdx.x; i < sm.g4; i += kThreads) { sm.m[i] = -INFINITY; sm.l[i] = 0.f; sm.fix[i] = 1.f; }
     for (int i = threadIdx.x; i < tile * sm.g4; i += kThreads) sm.w[i] = 0.f;
     const int pairs = A.rank_s / 2, sets = sm.g4 / 4 * pairs;
+    const int gh = (G + 1) / 2, units = gh * (tile / 2);
+    int LS = 1;
+    while (LS < 32 && 2 * LS * units <= kThreads) LS *= 2;
+    const int sub = threadIdx.x & (LS - 1);
     float acc[EP][4][2] = {};
     int buf = 0;
     for (int j = j0; j < j1; j += tile, buf ^= 1) {
@@ -153,15 +158,16 @@ __global__ void __launch_bounds__(kThreads) latent_attend_kernel(const LatentSte
         __syncthreads();
         const KT* K = sm.k + (size_t)buf * tile * sm.ks;
         const int keys = min(tile, j1 - j);
-        // scores: two heads x two rows per thread, neighbouring threads on neighbouring heads
-        const int gh = (G + 1) / 2, units = gh * (tile / 2);
-        for (int u = threadIdx.x; u < units; u += kThreads) {
-            const int p = u / gh * 2, h = (u - u / gh * gh) * 2, hb = min(h + 1, G - 1);
+        // scores: LS lanes share two heads x two rows
+        for (int u0 = 0; u0 < units; u0 += kThreads / LS) {
+            const int u = u0 + threadIdx.x / LS;
+            const bool in = u < units;
+            const int p = in ? u / gh * 2 : 0, h = in ? (u - u / gh * gh) * 2 : 0, hb = min(h + 1, G - 1);
             const KT *ka = K + p * sm.ks, *kb = ka + sm.ks;
             const float *qa0 = sm.q + h * sm.qs, *qb0 = sm.q + hb * sm.qs;
             float s[2][2] = {};
 #pragma unroll 2
-            for (int c = 0; c < chunks; c++) {
+            for (int c = in ? sub : chunks; c < chunks; c += LS) {
                 float x[CN], y[CN];
                 Chunk16<KT>::load(ka + c * CN, x);
                 Chunk16<KT>::load(kb + c * CN, y);
@@ -178,11 +184,19 @@ __global__ void __launch_bounds__(kThreads) latent_attend_kernel(const LatentSte
                     }
                 }
             }
-            sm.w[p * sm.g4 + h] = s[0][0];
-            sm.w[(p + 1) * sm.g4 + h] = s[0][1];
-            if (h + 1 < G) {
-                sm.w[p * sm.g4 + h + 1] = s[1][0];
-                sm.w[(p + 1) * sm.g4 + h + 1] = s[1][1];
+            for (int o = LS / 2; o > 0; o >>= 1) {
+                s[0][0] += __shfl_xor_sync(MG_FULL_MASK, s[0][0], o);
+                s[0][1] += __shfl_xor_sync(MG_FULL_MASK, s[0][1], o);
+                s[1][0] += __shfl_xor_sync(MG_FULL_MASK, s[1][0], o);
+                s[1][1] += __shfl_xor_sync(MG_FULL_MASK, s[1][1], o);
+            }
+            if (in && sub == 0) {
+                sm.w[p * sm.g4 + h] = s[0][0];
+                sm.w[(p + 1) * sm.g4 + h] = s[0][1];
+                if (h + 1 < G) {
+                    sm.w[p * sm.g4 + h + 1] = s[1][0];
+                    sm.w[(p + 1) * sm.g4 + h + 1] = s[1][1];
+                }
             }
         }
         __syncthreads();
@@ -245,14 +259,16 @@ __global__ void __launch_bounds__(kThreads) latent_attend_kernel(const LatentSte
 }
 
 constexpr int kValueRows = 32;      // value dimensions per CTA, four per warp
+constexpr int kValueGroups = 8;     // groups of threads that share the ranges, at most
 
 // CTA (head, 32 value dimensions) of one token: joins the ranges, then U_v times the weighted sum of latents.
 template <typename OT>
 __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentStep a) {
     extern __shared__ __align__(16) float smem[];
+    __shared__ float red[40];
     const LatentAttn& A = a.at;
-    float* o = smem;                                // [ld], zero from rank_s on
-    float* f = smem + A.ld;                         // [splits]
+    float* o = smem;                                // [groups][ld], zero from rank_s on
+    float* f = smem + kValueGroups * A.ld;          // [splits]
     const int slices = (A.vdim + kValueRows - 1) / kValueRows, t = blockIdx.y;
     const int h = blockIdx.x / slices, v0 = (blockIdx.x - h * slices) * kValueRows;
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
@@ -274,29 +290,47 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentStep
     int j0, j1;
     const int active = key_split(len, a.splits, a.tile, 0, &j0, &j1);
     const float2* ml = a.ml + (size_t)t * a.splits * A.heads + h;
-    if (wid == 0) {
-        float mx = -INFINITY, sum = 0.f;
-        for (int s = lane; s < active; s += 32) mx = fmaxf(mx, ml[(size_t)s * A.heads].x);
-        mx = warp_max(mx);
-        for (int s = lane; s < active; s += 32) {
-            const float2 p = ml[(size_t)s * A.heads];
-            const float e = expf(p.x - mx);
-            f[s] = e;
-            sum += e * p.y;
-        }
-        sum = warp_sum(sum);
-        __syncwarp();
-        for (int s = lane; s < active; s += 32) f[s] /= sum;
-    }
-    __syncthreads();
+    // four latent values per thread, the ranges dealt out to `rows` groups of threads
     const float* part = a.part + ((size_t)t * a.splits * A.heads + h) * A.rank_s;
     const size_t stride = (size_t)A.heads * A.rank_s;
-    for (int i = threadIdx.x; i < A.ld; i += kThreads) {
-        float v = 0.f;
-        if (i < A.rank_s) {
-#pragma unroll 8
-            for (int s = 0; s < active; s++) v = fmaf(f[s], part[s * stride + i], v);
+    const int quads = A.ld / 4, rows = min(kThreads / min(quads, kThreads), kValueGroups), grp = threadIdx.x / min(quads, kThreads);
+    {   // factors of the ranges
+        float mx = -INFINITY, sum = 0.f;
+        const float2 mine = (int)threadIdx.x < active ? ml[(size_t)threadIdx.x * A.heads] : make_float2(-INFINITY, 0.f);
+        for (int s = threadIdx.x; s < active; s += kThreads) mx = fmaxf(mx, s < kThreads ? mine.x : ml[(size_t)s * A.heads].x);
+        mx = block_max(mx, red);
+        for (int s = threadIdx.x; s < active; s += kThreads) {
+            const float2 p = s < kThreads ? mine : ml[(size_t)s * A.heads];
+            f[s] = expf(p.x - mx);
+            sum += f[s] * p.y;
         }
+        const float inv = 1.0f / block_sum(sum, red);
+        for (int s = threadIdx.x; s < active; s += kThreads) f[s] *= inv;
+    }
+    __syncthreads();
+    if (grp < rows)
+        for (int i = (threadIdx.x - grp * min(quads, kThreads)) * 4; i < A.ld; i += kThreads * 4) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < A.rank_s) {
+                constexpr int N = 16;               // ranges in flight
+                for (int s0 = grp; s0 < active; s0 += N * rows) {
+                    float4 p[N];
+#pragma unroll
+                    for (int q = 0; q < N; q++)
+                        p[q] = s0 + q * rows < active ? *reinterpret_cast<const float4*>(part + (s0 + q * rows) * stride + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                    for (int q = 0; q < N; q++) {
+                        const float w = s0 + q * rows < active ? f[s0 + q * rows] : 0.f;
+                        v.x = fmaf(w, p[q].x, v.x); v.y = fmaf(w, p[q].y, v.y); v.z = fmaf(w, p[q].z, v.z); v.w = fmaf(w, p[q].w, v.w);
+                    }
+                }
+            }
+            *reinterpret_cast<float4*>(o + grp * A.ld + i) = v;
+        }
+    __syncthreads();
+    for (int i = threadIdx.x; rows > 1 && i < A.ld; i += kThreads) {
+        float v = o[i];
+        for (int g = 1; g < rows; g++) v += o[g * A.ld + i];
         o[i] = v;
     }
     __syncthreads();
@@ -404,7 +438,12 @@ cudaError_t launch_latent_attend(const LatentStep& a, bool f32_cache, bool pdl, 
 
 cudaError_t launch_latent_value(const LatentStep& a, bool f32_out, bool pdl, cudaStream_t s) {
     const dim3 grid(a.at.heads * ((a.at.vdim + kValueRows - 1) / kValueRows), a.tokens);
-    const size_t smem = (size_t)(a.at.ld + a.splits) * sizeof(float);
+    const size_t smem = (size_t)(kValueGroups * a.at.ld + a.splits) * sizeof(float);
+    if (smem > 48 * 1024) {
+        cudaError_t c = cudaFuncSetAttribute(f32_out ? (const void*)latent_value_kernel<float> : (const void*)latent_value_kernel<__nv_bfloat16>,
+                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (c != cudaSuccess) return c;
+    }
     return f32_out ? launch_pdl(latent_value_kernel<float>, grid, kThreads, smem, pdl, s, a)
                    : launch_pdl(latent_value_kernel<__nv_bfloat16>, grid, kThreads, smem, pdl, s, a);
 }

@@ -178,8 +178,9 @@ cudaError_t launch_wkv_rows(const Wkv& wk, const float* proj, int ldp, const flo
 struct MoeStep {
     Moe moe;
     const float* router;        // one router row
-    const float* h;             // [width] normed
-    float* mid;                 // [top * ff] of the chosen experts
+    const float* h;             // [ldw] normed, zero from width on
+    int* sel;                   // [top] the choice, made by launch_moe_up's kernel
+    float* mid;                 // [top * ffs + shared_ffs] inner vectors of the chosen experts and the shared one
     float* out;                 // [width]
 };
 size_t moe_step_smem(const Moe& m);
@@ -194,13 +195,13 @@ struct MoeRows {                // workspace of a portion
     int* group;                 // [tiles] expert of every 128 grouped rows, -1: none
     int tiles;
     void* x;                    // [tiles * 128][ldw] grouped inputs
-    float* y;                   // [tiles * 128][width]
+    void* y;                    // [tiles * 128][width] grouped outputs, bf16 or fp32
 };
 inline int moe_tiles(const Moe& m, int n) { return (int)(((long long)n * m.top + 127) / 128) + m.experts; }
 // choice, grouping and the grouped inputs
 cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s);
 // z = weighted sum of the grouped rows (+ z times the shared expert's gate)
-cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, cudaStream_t s);
+cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, bool f32, cudaStream_t s);
 
 // ---- portions of a prompt (layered_prefill.cu) -----------------------------------------------------
 // `act` buffers hold bf16 or fp32 (f32 = true) rows padded to a multiple of 64 with zeros.

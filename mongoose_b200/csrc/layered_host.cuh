@@ -79,6 +79,7 @@ struct Layered {
     // one token
     float *row = nullptr, *part = nullptr, *attn = nullptr, *mem_raw = nullptr, *mem_y = nullptr, *y[2] = {}, *z = nullptr, *mid = nullptr;
     float *x0 = nullptr, *hn = nullptr, *q1 = nullptr, *rt = nullptr, *emid = nullptr;
+    int* esel = nullptr;
     float *qa = nullptr, *lpart = nullptr;      // latent attention: folded queries, partial sums (one token, or all rows)
     float2* ml = nullptr;
     // portions
@@ -187,7 +188,7 @@ int layered_buffers(Layered& m, F take) {
             get(&l.shared_down, (size_t)(e.shared_ff ? W : 0) * e.shared_ffs, 2);
             const size_t nt = moe_tiles(e, T), rows = nt * 128;
             rt = std::max(rt, (size_t)l.router_rows()); rtr = std::max(rtr, (size_t)pad_to(e.experts + 1, 4));
-            emid = std::max(emid, (size_t)e.top * e.ff);
+            emid = std::max(emid, (size_t)e.top * e.ffs + e.shared_ffs);
             xmid = std::max(xmid, std::max(rows * e.ffs, (size_t)T * e.shared_ffs));
             moe = std::max(moe, rows); tiles = std::max(tiles, nt); top = std::max(top, (size_t)e.top); experts = std::max(experts, (size_t)e.experts);
         }
@@ -213,7 +214,7 @@ int layered_buffers(Layered& m, F take) {
     if (c.positions == MG_POS_SINUSOID) get(&m.pos_tab, (size_t)c.max_seq * W, 4);
     get(&m.row, m.np, 4); get(&m.part, part, 4); get(&m.attn, kat, 4);
     get(&m.mem_raw, kmem, 4); get(&m.mem_y, kmem, 4); get(&m.y[0], W, 4); get(&m.y[1], W, 4); get(&m.z, W, 4); get(&m.mid, ff, 4);
-    get(&m.hn, any_pre ? W : 0, 4); get(&m.q1, q1, 4); get(&m.rt, rt, 4); get(&m.emid, emid, 4);
+    get(&m.hn, any_pre ? kw : 0, 4); get(&m.q1, q1, 4); get(&m.rt, rt, 4); get(&m.emid, emid, 4);
     get(&m.qa, qa, 4); get(&m.lpart, lpart, 4); get(&m.ml, ml, 8);
     get(&m.status, 1, 4); get(&m.tokens, T, 4); get(&m.want, T, 4);
     get(&m.x, (size_t)T * W, 4); get(&m.P, (size_t)T * m.np, 4);
@@ -228,7 +229,8 @@ int layered_buffers(Layered& m, F take) {
     get(&m.rtr, (size_t)T * rtr, 4); get(&m.xmid, xmid, as); get(&m.glu, m.f32 ? xmid : 0, 4);
     get(&m.moe.sel, (size_t)T * top, 4); get(&m.moe.slot, (size_t)T * top, 4); get(&m.moe.weight, (size_t)T * top, 4);
     get(&m.moe.count, experts, 4); get(&m.moe.first, experts ? experts + 1 : 0, 4); get(&m.moe.group, tiles, 4);
-    get(&m.moe.x, moe * kw, as); get(&m.moe.y, moe * W, 4);
+    get(&m.moe.x, moe * kw, as); get(&m.moe.y, moe * W, as);
+    get(&m.esel, top, 4);
     get(&m.mw.b, (size_t)mh * T, 8); get(&m.mw.ig, (size_t)mh * T, 4); get(&m.mw.mm, (size_t)mh * T, 4); get(&m.mw.m0, mh, 4);
     get(&m.mw.g, (size_t)mh * ((T + kMemChunk - 1) / kMemChunk), 4);
     get(&m.mw.U, u, 4); get(&m.mw.nU, nu, 4); get(&m.mw.o, (size_t)T * kmem, 4);
@@ -693,7 +695,7 @@ int enqueue_layered_step(mg_engine* e, cudaStream_t s, int ls, int le, int mode,
         a.w[0] = WeightView{l.router, nullptr}; a.rows[0] = l.router_rows(); a.out = m.rt;
         if ((rc = phase(a, EPI_STORE))) return rc;
         MoeStep t{};
-        t.moe = l.moe; t.router = m.rt; t.h = m.hn; t.mid = m.emid; t.out = m.z;
+        t.moe = l.moe; t.router = m.rt; t.h = m.hn; t.sel = m.esel; t.mid = m.emid; t.out = m.z;
         MG_CUDA(e, launch_moe_up(t, e->num_sms, e->use_pdl, s));
         MG_CUDA(e, launch_moe_down(t, e->num_sms, e->use_pdl, s));
         e->capture_kernels += 2;
@@ -785,9 +787,9 @@ int layered_matmul_batch(mg_engine* e, const void* act, long long stride, int ac
 }
 
 // One gated feed-forward, or with `group` those of stacked experts, each tile of 128 rows its own: z = down(silu(gate
-// act) * (up act)).  ld, ffs: padded row lengths; `count` matrices are stacked.
+// act) * (up act)), fp32 or like activations.  ld, ffs: padded row lengths; `count` matrices are stacked.
 int layered_glu(mg_engine* e, const void* act, int act_rows, int ld, const uint8_t* gate, const uint8_t* up, const uint8_t* down, int ff, int ffs,
-                int count, const int* group, float* z, int n) {
+                int count, const int* group, void* z, bool z_act, int n) {
     Layered& m = *e->lm;
     const int W = m.c.width;
     e->launches += m.f32 ? 3 : 2;
@@ -799,7 +801,7 @@ int layered_glu(mg_engine* e, const void* act, int act_rows, int ld, const uint8
         g.W = up; g.out = (float*)m.xmid; g.epi = F32_SILU_MUL; g.aux = m.glu;
         MG_CUDA(e, launch_gemm_f32(g, e->stream));
         g = GemmF32{};
-        g.A = (const float*)m.xmid; g.lda = ffs; g.W = down; g.ldw = ffs; g.out = z; g.ldc = W; g.n = n; g.rows = W; g.K = ffs;
+        g.A = (const float*)m.xmid; g.lda = ffs; g.W = down; g.ldw = ffs; g.out = (float*)z; g.ldc = W; g.n = n; g.rows = W; g.K = ffs;
         g.group = group; g.group_stride = (long long)W * ffs;
         MG_CUDA(e, launch_gemm_f32(g, e->stream));
         return MG_OK;
@@ -811,7 +813,7 @@ int layered_glu(mg_engine* e, const void* act, int act_rows, int ld, const uint8
         !make_tile_map(&g.b, gate, ld, ff, count, ld, (long long)ff * ld, 64) || !make_tile_map(&g.b2, up, ld, ff, count, ld, (long long)ff * ld, 64))
         return fail(e, MG_ERR_CUDA, "tensor map of a %d x %d feed-forward failed", ff, ld);
     MG_CUDA(e, launch_gemm_tc(g, e->stream));
-    g.bn = W > 64 ? 128 : 64; g.n = W; g.k = ffs; g.out = z; g.ldc = W; g.mode = GEMM_F32;
+    g.bn = W > 64 ? 128 : 64; g.n = W; g.k = ffs; g.out = z; g.ldc = W; g.mode = z_act ? GEMM_BF16 : GEMM_F32;
     if (!make_tile_map(&g.a, m.xmid, ffs, act_rows, 1, ffs, (long long)act_rows * ffs, 128) ||
         !make_tile_map(&g.b, down, ffs, W, count, ffs, (long long)W * ffs, g.bn))
         return fail(e, MG_ERR_CUDA, "tensor map of a %d x %d feed-forward failed", W, ffs);
@@ -901,10 +903,10 @@ int moe_rows(mg_engine* e, LayerWeights& l, int n) {
     int rc;
     if ((rc = layered_matmul(e, m.act, m.max_rows, m.kw, l.router, m.rtr, ldr, n, cols, false))) return rc;
     MG_CUDA(e, launch_moe_route(x, m.rtr, ldr, n, m.act, m.f32, w, s));
-    if ((rc = layered_glu(e, w.x, w.tiles * 128, m.kw, l.e_gate, l.e_up, l.e_down, x.ff, x.ffs, x.experts, w.group, w.y, w.tiles * 128))) return rc;
+    if ((rc = layered_glu(e, w.x, w.tiles * 128, m.kw, l.e_gate, l.e_up, l.e_down, x.ff, x.ffs, x.experts, w.group, w.y, true, w.tiles * 128))) return rc;
     if (x.shared_ff && (rc = layered_glu(e, m.act, m.max_rows, m.kw, l.router_row(x.sg_col() + 1), l.router_row(x.sg_col() + 1 + x.shared_ff),
-                                         l.shared_down, x.shared_ff, x.shared_ffs, 1, nullptr, m.zr, n))) return rc;
-    MG_CUDA(e, launch_moe_combine(x, m.rtr, ldr, n, w, m.zr, s));
+                                         l.shared_down, x.shared_ff, x.shared_ffs, 1, nullptr, m.zr, false, n))) return rc;
+    MG_CUDA(e, launch_moe_combine(x, m.rtr, ldr, n, w, m.zr, m.f32, s));
     e->launches += 4;
     return MG_OK;
 }

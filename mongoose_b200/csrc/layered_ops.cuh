@@ -20,6 +20,40 @@ __device__ __forceinline__ float2 pair_f32(const __nv_bfloat16* p) {
     const uint32_t w = *reinterpret_cast<const uint32_t*>(p);
     return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u));
 }
+// V values at once (V = 4: the address is a multiple of 16 bytes, of 8 for bf16)
+template <int V>
+__device__ __forceinline__ void load_values(const float* p, float (&o)[V]) {
+    if constexpr (V == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+    } else {
+        o[0] = *p;
+    }
+}
+template <int V>
+__device__ __forceinline__ void load_values(const __nv_bfloat16* p, float (&o)[V]) {
+    if constexpr (V == 4) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        o[0] = __uint_as_float(v.x << 16); o[1] = __uint_as_float(v.x & 0xffff0000u);
+        o[2] = __uint_as_float(v.y << 16); o[3] = __uint_as_float(v.y & 0xffff0000u);
+    } else {
+        o[0] = __bfloat162float(*p);
+    }
+}
+template <int V>
+__device__ __forceinline__ void store_values(const float (&v)[V], float* p) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else *p = v[0];
+}
+template <int V>
+__device__ __forceinline__ void store_values(const float (&v)[V], __nv_bfloat16* p) {
+    if constexpr (V == 4) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    } else {
+        *p = __float2bfloat16_rn(v[0]);
+    }
+}
 // 16 bytes of keys as floats
 template <typename KT>
 struct Chunk16;
@@ -163,6 +197,33 @@ inline size_t attn_smem(const GateAttn& at, int nq, int kt_bytes, int most, int*
     }
     return 0;
 }
+
+// Maximum over a whole CTA; every thread gets it.  `red` as for block_sum.
+__device__ __forceinline__ float block_max(float v, float* red) {
+    v = warp_max(v);
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+    __syncthreads();
+    if (lane == 0) red[wid] = v;
+    __syncthreads();
+    return warp_max(lane < nw ? red[lane] : -INFINITY);
+}
+
+// Two fp32 operations at once.
+__device__ __forceinline__ unsigned long long pack2(float a, float b) {
+    return (unsigned long long)__float_as_uint(a) | ((unsigned long long)__float_as_uint(b) << 32);
+}
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ float lo(unsigned long long v) { return __uint_as_float((unsigned)v); }
+__device__ __forceinline__ float hi(unsigned long long v) { return __uint_as_float((unsigned)(v >> 32)); }
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");

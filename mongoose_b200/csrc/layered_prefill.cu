@@ -152,21 +152,26 @@ __global__ void __launch_bounds__(256) post_rows_kernel(float* x, const float* z
     }
 }
 
-// Mean and 1 / sqrt(spread + eps) of a row for a norm of the given kind; get(i) is the thread's own element i.
-template <typename F>
-__device__ __forceinline__ float2 row_norm(F get, int kind, float eps, int width, float* red) {
+// Mean and 1 / sqrt(spread + eps) of row y for a norm of the given kind; a thread reads V values at a time, those
+// it would write in a loop of the same shape.
+template <int V>
+__device__ __forceinline__ float2 row_norm(const float* y, int kind, float eps, int width, float* red) {
     const float inv = 1.0f / (float)width;
     float s = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = get(i);
-        s += kind == NORM_LAYER ? v : v * v;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float v[V];
+        load_values<V>(y + i, v);
+#pragma unroll
+        for (int q = 0; q < V; q++) s += kind == NORM_LAYER ? v[q] : v[q] * v[q];
     }
     s = block_sum(s, red) * inv;
     if (kind != NORM_LAYER) return make_float2(0.f, 1.0f / sqrtf(s + eps));
     float d = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = get(i) - s;
-        d = fmaf(v, v, d);
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float v[V];
+        load_values<V>(y + i, v);
+#pragma unroll
+        for (int q = 0; q < V; q++) d = fmaf(v[q] - s, v[q] - s, d);
     }
     return make_float2(s, 1.0f / sqrtf(block_sum(d, red) * inv + eps));
 }
@@ -176,45 +181,48 @@ __global__ void __launch_bounds__(256) last_norm_rows_kernel(const float* x, con
                                                              AT* act, int ld_act) {
     __shared__ float red[40];
     const float* a = x + (size_t)rows[blockIdx.x] * width;
-    const float2 n = row_norm([&](int i) { return a[i]; }, kind, eps, width, red);
+    const float2 n = row_norm<1>(a, kind, eps, width, red);
     const float one = kind == NORM_RMS_AROUND_ZERO ? 1.0f : 0.0f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) from_f32((a[i] - n.x) * n.y * (one + w[i]), act + (size_t)blockIdx.x * ld_act + i);
 }
 
-template <typename AT>
+template <typename AT, int V>
 __global__ void __launch_bounds__(256) prenorm_rows_kernel(const PrenormRows a) {
     extern __shared__ __align__(16) float y[];
     __shared__ float red[40];
-    const int W = a.width;
+    const int W = a.width, step = 256 * V;
     const size_t r = blockIdx.x;
     float* x = a.x + r * W;
     AT* act = static_cast<AT*>(a.act) + r * a.ld_act;
-    for (int i = threadIdx.x; i < W; i += blockDim.x) {
-        float v = x[i];
+    for (int i = threadIdx.x * V; i < W; i += step) {
+        float v[V];
+        load_values<V>(x + i, v);
         if (a.z) {
-            v += a.mult * (a.ls[i] * a.z[r * W + i]);
-            x[i] = v;
+            float z[V], ls[V];
+            load_values<V>(a.z + r * W + i, z);
+            load_values<V>(a.ls + i, ls);
+#pragma unroll
+            for (int q = 0; q < V; q++) v[q] += a.mult * (ls[q] * z[q]);
+            store_values<V>(v, x + i);
         }
-        y[i] = v;
-    }
-    if (a.cat) {
-        for (int i = threadIdx.x; i < W; i += blockDim.x) {
-            from_f32(y[i], act + i);
-            from_f32(a.cat[r * W + i], act + W + i);
+        if (a.norm_w) store_values<V>(v, y + i);
+        else if (a.act) store_values<V>(v, act + i);
+        if (a.cat) {
+            load_values<V>(a.cat + r * W + i, v);
+            store_values<V>(v, act + W + i);
         }
-        return;
     }
-    if (!a.norm_w) {
-        if (a.act)
-            for (int i = threadIdx.x; i < W; i += blockDim.x) from_f32(y[i], act + i);
-        return;
-    }
-    const float2 n = row_norm([&](int i) { return y[i]; }, a.kind, a.eps, W, red);
+    if (!a.norm_w) return;
+    const float2 n = row_norm<V>(y, a.kind, a.eps, W, red);
     const float one = a.kind == NORM_RMS_AROUND_ZERO ? 1.0f : 0.0f;
-    for (int i = threadIdx.x; i < W; i += blockDim.x) {
-        const float v = (y[i] - n.x) * n.y * (one + a.norm_w[i]);
-        if (a.h) a.h[r * W + i] = v;
-        else from_f32(v, act + i);
+    for (int i = threadIdx.x * V; i < W; i += step) {
+        float v[V], w[V];
+        load_values<V>(y + i, v);
+        load_values<V>(a.norm_w + i, w);
+#pragma unroll
+        for (int q = 0; q < V; q++) v[q] = (v[q] - n.x) * n.y * (one + w[q]);
+        if (a.h) store_values<V>(v, a.h + r * W + i);
+        else store_values<V>(v, act + i);
     }
 }
 
@@ -493,6 +501,29 @@ __global__ void __launch_bounds__(256) head_norm_rows_kernel(int heads, int vdim
     }
 }
 
+// The same with a quad of values per lane and `lanes` lanes (a power of two) per head: head sizes that are whole
+// quads, up to 128.
+template <typename AT>
+__global__ void __launch_bounds__(256) head_norm_quads_kernel(int heads, int vdim, int lanes, float eps, const float* norm, const float* gate,
+                                                              int ldg, int gate_kind, int n, const float* o, AT* act, int ld_act) {
+    const int unit = (blockIdx.x * 256 + threadIdx.x) / lanes, sub = threadIdx.x & (lanes - 1);
+    const int t = unit / heads, h = unit - t * heads, c = h * vdim + sub * 4;
+    const bool in = t < n && sub * 4 < vdim;
+    float v[4] = {}, g[4], w[4];
+    if (in) {
+        load_values<4>(o + (size_t)t * heads * vdim + c, v);
+        load_values<4>(gate + (size_t)t * ldg + c, g);
+        load_values<4>(norm + c, w);
+    }
+    float ss = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+    for (int m = lanes / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(MG_FULL_MASK, ss, m);
+    const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
+    if (!in) return;
+#pragma unroll
+    for (int q = 0; q < 4; q++) v[q] *= r * w[q] * (gate_kind == GATE_SILU ? silu(g[q]) : sigmoid(g[q]));
+    store_values<4>(v, act + (size_t)t * ld_act + c);
+}
+
 template <typename KT, int NQ>
 cudaError_t attn_rows_for(const GateAttn& at, const void* qh, int pos0, int n, void* out, int ld_out, cudaStream_t s) {
     int tile;
@@ -563,17 +594,31 @@ cudaError_t launch_last_norm_rows(const float* x, const int* rows, const float* 
 
 cudaError_t launch_prenorm_rows(const PrenormRows& a, bool f32, cudaStream_t s) {
     const size_t smem = (size_t)a.width * sizeof(float);
-    if (f32) prenorm_rows_kernel<float><<<a.n, 256, smem, s>>>(a);
-    else prenorm_rows_kernel<__nv_bfloat16><<<a.n, 256, smem, s>>>(a);
+    const bool quads = a.width % 4 == 0;
+    if (f32 && quads) prenorm_rows_kernel<float, 4><<<a.n, 256, smem, s>>>(a);
+    else if (f32) prenorm_rows_kernel<float, 1><<<a.n, 256, smem, s>>>(a);
+    else if (quads) prenorm_rows_kernel<__nv_bfloat16, 4><<<a.n, 256, smem, s>>>(a);
+    else prenorm_rows_kernel<__nv_bfloat16, 1><<<a.n, 256, smem, s>>>(a);
+    return cudaGetLastError();
+}
+
+template <typename AT>
+static cudaError_t head_norm_for(int heads, int vdim, float eps, const float* norm, const float* gate, int ldg, int gate_kind, int n, const float* o,
+                                 AT* act, int ld_act, cudaStream_t s) {
+    const bool quads = vdim % 4 == 0 && vdim <= 128 && ldg % 4 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0;
+    int lanes = 1;
+    while (lanes * 4 < vdim) lanes *= 2;
+    if (quads)
+        head_norm_quads_kernel<AT><<<(int)(((long long)n * heads * lanes + 255) / 256), 256, 0, s>>>(heads, vdim, lanes, eps, norm, gate, ldg, gate_kind, n, o, act, ld_act);
+    else
+        head_norm_rows_kernel<AT><<<(n * heads + 7) / 8, 256, 0, s>>>(heads, vdim, eps, norm, gate, ldg, gate_kind, n, o, act, ld_act);
     return cudaGetLastError();
 }
 
 cudaError_t launch_head_norm_rows(int heads, int vdim, float eps, const float* norm, const float* gate, int ldg, int gate_kind, int n,
                                   const float* o, void* act, int ld_act, bool f32, cudaStream_t s) {
-    const int grid = (n * heads + 7) / 8;
-    if (f32) head_norm_rows_kernel<float><<<grid, 256, 0, s>>>(heads, vdim, eps, norm, gate, ldg, gate_kind, n, o, (float*)act, ld_act);
-    else head_norm_rows_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(heads, vdim, eps, norm, gate, ldg, gate_kind, n, o, (__nv_bfloat16*)act, ld_act);
-    return cudaGetLastError();
+    return f32 ? head_norm_for(heads, vdim, eps, norm, gate, ldg, gate_kind, n, o, (float*)act, ld_act, s)
+               : head_norm_for(heads, vdim, eps, norm, gate, ldg, gate_kind, n, o, (__nv_bfloat16*)act, ld_act, s);
 }
 
 cudaError_t launch_mem_rows(const MatMem& mem, const ProjCols& c, const float* proj, int ldp, int pos0, int n, const MemRows& w, void* act,

@@ -11,30 +11,31 @@ namespace {
 
 constexpr int kThreads = 256;
 
-// One warp: the `top` largest of z[0..experts) in falling order (lower index first among equals) and the softmax
-// over them.  z is shared memory and is overwritten; sel and wt are shared memory too.  Whatever z holds,
-// the chosen indices are distinct and valid.
-__device__ __forceinline__ void choose(float* z, int experts, int top, int* sel, float* wt, int lane) {
+// Order of floats as unsigned integers.
+__device__ __forceinline__ unsigned ordered(float v) {
+    const unsigned u = __float_as_uint(v);
+    return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+
+// One warp: the `top` largest of z[0..experts) in falling order and the softmax over them.  z, sel and wt are shared
+// memory.  Whatever z holds, the chosen indices are distinct and valid.
+__device__ __forceinline__ void choose(const float* z, int experts, int top, int* sel, float* wt, int lane) {
     unsigned taken = 0;                     // of this lane's entries lane, lane + 32, ...
     float first = 0.f, sum = 0.f;
     for (int k = 0; k < top; k++) {
         int bi = -1;
-        float bv = 0.f;
+        unsigned bv = 0;
         for (int i = lane, q = 0; i < experts; i += 32, q++) {
-            const float v = z[i];
+            const unsigned v = ordered(z[i]);
             if (!((taken >> q) & 1u) && (bi < 0 || v > bv)) { bi = i; bv = v; }
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const int oi = __shfl_xor_sync(MG_FULL_MASK, bi, o);
-            const float ov = __shfl_xor_sync(MG_FULL_MASK, bv, o);
-            if (oi >= 0 && (bi < 0 || ov > bv || (!(bv > ov) && oi < bi))) { bi = oi; bv = ov; }
-        }
-        bi = __shfl_sync(MG_FULL_MASK, bi, 0);          // one answer, also where comparisons have none
-        bv = __shfl_sync(MG_FULL_MASK, bv, 0);
+        const unsigned best = __reduce_max_sync(MG_FULL_MASK, bi < 0 ? 0u : bv);
+        const int from = __ffs(__ballot_sync(MG_FULL_MASK, bi >= 0 && bv == best)) - 1;
+        bi = __shfl_sync(MG_FULL_MASK, bi, from);
         if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
-        if (k == 0) first = bv;
-        const float e = expf(bv - first);
+        const float v = z[bi];
+        if (k == 0) first = v;
+        const float e = expf(v - first);
         sum += e;
         if (lane == 0) { sel[k] = bi; wt[k] = e; }
     }
@@ -52,7 +53,8 @@ __device__ __forceinline__ void choose_cta(const Moe& m, const float* router, fl
     __syncthreads();
 }
 
-// mid[k][row] = silu(gate row . h) * (up row . h) of the chosen experts: a warp per (expert, row).
+// The vector that the down matrices read: per chosen expert silu(gate row . h) * (up row . h) times its weight, then the
+// shared expert's inner vector times its gate; parts are padded like the matrices' rows.  A warp per (expert, row).
 __global__ void __launch_bounds__(kThreads) moe_up_kernel(const MoeStep a) {
     extern __shared__ __align__(16) float smem[];
     __shared__ int sel[kMaxTop];
@@ -62,12 +64,17 @@ __global__ void __launch_bounds__(kThreads) moe_up_kernel(const MoeStep a) {
     float* zs = smem + m.ldw;               // [experts]
     pdl_launch_dependents();
     pdl_wait();
-    for (int i = threadIdx.x; i < m.ldw; i += kThreads) hs[i] = i < m.width ? a.h[i] : 0.f;
+    for (int i = threadIdx.x * 4; i < m.ldw; i += kThreads * 4) cp_async16(hs + i, a.h + i);
+    cp_async_commit();
     choose_cta(m, a.router, zs, sel, wt);
+    if (blockIdx.x == 0)
+        for (int k = threadIdx.x; k < m.top; k += kThreads) a.sel[k] = sel[k];
+    cp_async_wait<0>();
+    __syncthreads();
     const int lane = threadIdx.x & 31, nw = gridDim.x * (kThreads / 32), chunks = m.ldw / 8, items = m.top * m.ff;
     for (int it = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5); it < items; it += nw) {
-        const int k = it / m.ff;
-        const size_t row = (size_t)sel[k] * m.ff + (it - k * m.ff);
+        const int k = it / m.ff, f = it - k * m.ff;
+        const size_t row = (size_t)sel[k] * m.ff + f;
         const uint4* g = reinterpret_cast<const uint4*>(m.gate + row * m.ldw * 2);
         const uint4* u = reinterpret_cast<const uint4*>(m.up + row * m.ldw * 2);
         float sg = 0.f, su = 0.f;
@@ -91,67 +98,82 @@ __global__ void __launch_bounds__(kThreads) moe_up_kernel(const MoeStep a) {
         }
         sg = warp_sum(sg);
         su = warp_sum(su);
-        if (lane == 0) a.mid[it] = silu(sg) * su;
+        if (lane == 0) a.mid[k * m.ffs + f] = silu(sg) * su * wt[k];
+    }
+    if (m.shared_ff) {
+        const float *g = a.router + m.sg_col() + 1, *u = g + m.shared_ff;
+        for (int i = blockIdx.x * kThreads + threadIdx.x; i < m.shared_ff; i += gridDim.x * kThreads)
+            a.mid[m.top * m.ffs + i] = silu(g[i]) * u[i] * sigmoid(a.router[m.sg_col()]);
     }
 }
 
-// out[row] = sum over the chosen experts of weight * (down row . mid) + gate * (shared down row . its mid): the
-// factors go into the staged vectors, a warp per output row.
+// out = the chosen experts' down matrices and the shared one, side by side, times that vector.  A CTA takes R rows at
+// a time, its warps share their columns, and the first rows' weights are on the way before the vector is there.
 template <int R>
 __global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeStep a) {
     extern __shared__ __align__(16) float smem[];
+    __shared__ float part[2][kThreads / 32][R];
     __shared__ int sel[kMaxTop];
-    __shared__ float wt[kMaxTop];
+    constexpr int AHEAD = 3;
     const Moe& m = a.moe;
     float* xs = smem;                                   // [top * ffs + shared_ffs]
-    float* zs = smem + m.top * m.ffs + m.shared_ffs;    // [experts]
-    const int lane = threadIdx.x & 31;
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
+    const int per = m.ffs / 8, own = m.top * per, chunks = own + m.shared_ffs / 8;
     pdl_launch_dependents();
     pdl_wait();
-    choose_cta(m, a.router, zs, sel, wt);
-    for (int k = 0; k < m.top; k++)
-        for (int i = threadIdx.x; i < m.ffs; i += kThreads) xs[k * m.ffs + i] = i < m.ff ? a.mid[k * m.ff + i] * wt[k] : 0.f;
-    if (m.shared_ff) {
-        const float sg = sigmoid(a.router[m.sg_col()]);
-        const float *g = a.router + m.sg_col() + 1, *u = g + m.shared_ff;
-        for (int i = threadIdx.x; i < m.shared_ffs; i += kThreads) xs[m.top * m.ffs + i] = i < m.shared_ff ? silu(g[i]) * u[i] * sg : 0.f;
-    }
+    for (int i = threadIdx.x * 4; i < chunks * 8; i += kThreads * 4) cp_async16(xs + i, a.mid + i);
+    cp_async_commit();
+    for (int k = threadIdx.x; k < m.top; k += kThreads) sel[k] = a.sel[k];
     __syncthreads();
-    const int nw = gridDim.x * (kThreads / 32);
-    for (int r0 = (blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5)) * R; r0 < m.width; r0 += nw * R) {
+    auto load = [&](int c, int r0, uint4 (&w)[R]) {
+        const int k = c / per;
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const size_t row = min(r0 + r, m.width - 1);
+            w[r] = c >= chunks ? make_uint4(0u, 0u, 0u, 0u)
+                 : c < own ? ld_stream16(m.down + (((size_t)sel[k] * m.width + row) * per + (c - k * per)) * 16)
+                           : ld_stream16(m.shared_down + (row * (m.shared_ffs / 8) + (c - own)) * 16);
+        }
+    };
+    uint4 w[AHEAD][R];
+    int r0 = blockIdx.x * R;
+#pragma unroll
+    for (int i = 0; i < AHEAD; i++) load(threadIdx.x + i * kThreads, r0, w[i]);
+    cp_async_wait<0>();
+    __syncthreads();
+    for (int buf = 0; r0 < m.width; r0 += gridDim.x * R, buf ^= 1) {
         float acc[R] = {};
-        for (int k = 0; k < m.top + (m.shared_ff ? 1 : 0); k++) {
-            const bool sh = k == m.top;
-            const int ld = sh ? m.shared_ffs : m.ffs, chunks = ld / 8;
-            const uint8_t* w = sh ? m.shared_down : m.down + (size_t)sel[k] * m.width * ld * 2;
-            const float* x0 = xs + k * m.ffs;
-            const uint4* row[R];
+        auto use = [&](int c, const uint4 (&v)[R]) {
+            if (c < chunks) {
+                const float4 x[2] = {*reinterpret_cast<const float4*>(xs + c * 8), *reinterpret_cast<const float4*>(xs + c * 8 + 4)};
 #pragma unroll
-            for (int r = 0; r < R; r++) row[r] = reinterpret_cast<const uint4*>(w + (size_t)min(r0 + r, m.width - 1) * ld * 2);
-            for (int c0 = 0; c0 < chunks; c0 += 128) {
-                uint4 ww[R][4];
-#pragma unroll
-                for (int i = 0; i < 4; i++)
-#pragma unroll
-                    for (int r = 0; r < R; r++) {
-                        const int c = c0 + i * 32 + lane;
-                        ww[r][i] = c < chunks ? ld_stream16(row[r] + c) : make_uint4(0u, 0u, 0u, 0u);
-                    }
-#pragma unroll
-                for (int i = 0; i < 4; i++) {
-                    const int c = c0 + i * 32 + lane;
-                    if (c < chunks) {
-                        const float4 x[2] = {*reinterpret_cast<const float4*>(x0 + c * 8), *reinterpret_cast<const float4*>(x0 + c * 8 + 4)};
-#pragma unroll
-                        for (int r = 0; r < R; r++) acc[r] += Chunk<FMT_BF16>::dot(ww[r][i], x);
-                    }
-                }
+                for (int r = 0; r < R; r++) acc[r] += Chunk<FMT_BF16>::dot(v[r], x);
             }
+        };
+        const int next = r0 + gridDim.x * R;
+#pragma unroll
+        for (int i = 0; i < AHEAD; i++) use(threadIdx.x + i * kThreads, w[i]);
+        for (int c = threadIdx.x + AHEAD * kThreads; c < chunks; c += AHEAD * kThreads) {
+#pragma unroll
+            for (int i = 0; i < AHEAD; i++) load(c + i * kThreads, r0, w[i]);
+#pragma unroll
+            for (int i = 0; i < AHEAD; i++) use(c + i * kThreads, w[i]);
+        }
+        if (next < m.width) {
+#pragma unroll
+            for (int i = 0; i < AHEAD; i++) load(threadIdx.x + i * kThreads, next, w[i]);
         }
 #pragma unroll
         for (int r = 0; r < R; r++) {
             const float v = warp_sum(acc[r]);
-            if (lane == 0 && r0 + r < m.width) a.out[r0 + r] = v;
+            if (lane == 0) part[buf][wid][r] = v;
+        }
+        __syncthreads();
+        if (threadIdx.x < R && r0 + threadIdx.x < m.width) {
+            float v = 0.f;
+#pragma unroll
+            for (int q = 0; q < kThreads / 32; q++) v += part[buf][q][threadIdx.x];
+            a.out[r0 + threadIdx.x] = v;
         }
     }
 }
@@ -209,6 +231,7 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const Moe m, const uint
     }
 }
 
+template <typename AT, int V>
 __global__ void __launch_bounds__(kThreads) moe_combine_kernel(const Moe m, const float* router, int ldr, MoeRows w, float* z) {
     __shared__ float wt[kMaxTop];
     __shared__ int row[kMaxTop];
@@ -218,23 +241,32 @@ __global__ void __launch_bounds__(kThreads) moe_combine_kernel(const Moe m, cons
         row[k] = w.first[w.sel[t * m.top + k]] + w.slot[t * m.top + k];
     }
     __syncthreads();
+    const AT* y = static_cast<const AT*>(w.y);
     const float sg = m.shared_ff ? sigmoid(router[t * ldr + m.sg_col()]) : 0.f;
     float* out = z + t * m.width;
-    for (int i = threadIdx.x; i < m.width; i += kThreads) {
-        float v = m.shared_ff ? sg * out[i] : 0.f;
+    for (int i = threadIdx.x * V; i < m.width; i += kThreads * V) {
+        float v[V] = {};
+        if (m.shared_ff) {
+            load_values<V>(out + i, v);
+#pragma unroll
+            for (int q = 0; q < V; q++) v[q] *= sg;
+        }
 #pragma unroll 4
-        for (int k = 0; k < m.top; k++) v = fmaf(wt[k], w.y[(size_t)row[k] * m.width + i], v);
-        out[i] = v;
+        for (int k = 0; k < m.top; k++) {
+            float e[V];
+            load_values<V>(y + (size_t)row[k] * m.width + i, e);
+#pragma unroll
+            for (int q = 0; q < V; q++) v[q] = fmaf(wt[k], e[q], v[q]);
+        }
+        store_values<V>(v, out + i);
     }
 }
 
-constexpr int kDownRows = 2;
+constexpr int kDownRows = 4;
 
 }  // namespace
 
-size_t moe_step_smem(const Moe& m) {
-    return (size_t)(std::max(m.ldw, m.top * m.ffs + m.shared_ffs) + m.experts) * sizeof(float);
-}
+size_t moe_step_smem(const Moe& m) { return (size_t)std::max(m.ldw + m.experts, m.top * m.ffs + m.shared_ffs) * sizeof(float); }
 
 cudaError_t moe_step_attrs(size_t bytes) {
     cudaError_t c = cudaFuncSetAttribute((const void*)moe_up_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
@@ -248,8 +280,10 @@ cudaError_t launch_moe_up(const MoeStep& a, int sms, bool pdl, cudaStream_t s) {
 
 cudaError_t launch_moe_down(const MoeStep& a, int sms, bool pdl, cudaStream_t s) {
     const Moe& m = a.moe;
-    const int grid = std::min((m.width + 8 * kDownRows - 1) / (8 * kDownRows), 2 * sms);
-    return launch_pdl(moe_down_kernel<kDownRows>, grid, kThreads, (size_t)(m.top * m.ffs + m.shared_ffs + m.experts) * sizeof(float), pdl, s, a);
+    const size_t smem = (size_t)(m.top * m.ffs + m.shared_ffs) * sizeof(float);
+    const int per_sm = std::max(1, std::min(2, (int)(220 * 1024 / (smem + 2048))));     // CTAs that share an SM
+    const int grid = std::min((m.width + kDownRows - 1) / kDownRows, per_sm * sms);
+    return launch_pdl(moe_down_kernel<kDownRows>, grid, kThreads, smem, pdl, s, a);
 }
 
 cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s) {
@@ -259,8 +293,12 @@ cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int n, 
     return cudaGetLastError();
 }
 
-cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, cudaStream_t s) {
-    moe_combine_kernel<<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
+cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, bool f32, cudaStream_t s) {
+    const bool quads = m.width % 4 == 0;
+    if (f32 && quads) moe_combine_kernel<float, 4><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
+    else if (f32) moe_combine_kernel<float, 1><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
+    else if (quads) moe_combine_kernel<__nv_bfloat16, 4><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
+    else moe_combine_kernel<__nv_bfloat16, 1><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
     return cudaGetLastError();
 }
 

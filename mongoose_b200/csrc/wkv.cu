@@ -9,7 +9,7 @@ namespace mg {
 namespace {
 
 constexpr int kStepThreads = 256;
-constexpr int kStepRows = 16;       // rows of the state a warp holds at a time
+constexpr int kStepRows = 8;        // rows of the state a warp holds at a time, two columns per lane
 
 // One token: a CTA per head, lanes over value channels, warps over key channels.
 __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvStep a) {
@@ -21,17 +21,28 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvStep a)
     float* part = inner + rk;               // [warps][D]
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     constexpr int nw = kStepThreads / 32;
+    // weights first: they wait for nothing
+    const int sub = threadIdx.x & 3, d_of = threadIdx.x >> 2;
+    constexpr int kAhead = 2;
+    uint4 w2[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; i++) {
+        const int c = (sub + 4 * i) * 8;
+        w2[i] = d_of < D && c < rk ? __ldg(reinterpret_cast<const uint4*>(M.w2 + (size_t)(c0 + d_of) * M.ld2 + c)) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    const float w0 = d_of < D ? M.w0[c0 + d_of] : 0.f;
     for (int i = threadIdx.x; i < D; i += kStepThreads) u[i] = M.u[c0 + i];
     pdl_launch_dependents();
     pdl_wait();
     const bool fresh = a.st->pos == 0;
     float* S = M.S + (size_t)blockIdx.x * D * D;
-    float s0[kStepRows];
+    float s0[kStepRows][2];
     auto load_rows = [&](int k0, int col) {
 #pragma unroll
         for (int i = 0; i < kStepRows; i++) {
             const int d = k0 + wid + i * nw;
-            s0[i] = !fresh && col < D && d < D ? S[(size_t)d * D + col] : 0.f;
+            s0[i][0] = !fresh && col < D && d < D ? S[(size_t)d * D + col] : 0.f;
+            s0[i][1] = !fresh && col + 32 < D && d < D ? S[(size_t)d * D + col + 32] : 0.f;
         }
     };
     load_rows(0, lane);
@@ -39,41 +50,50 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvStep a)
     for (int i = threadIdx.x; i < rk; i += kStepThreads) inner[i] = i < M.rank ? tanhf(a.row[4 * (size_t)n + i]) : 0.f;
     __syncthreads();
     // decays: four threads per channel
-    const int sub = threadIdx.x & 3;
     for (int d0 = 0; d0 < D; d0 += kStepThreads / 4) {
-        const int d = d0 + (threadIdx.x >> 2);
+        const int d = d0 + d_of;
         float z = 0.f;
         if (d < D) {
             const __nv_bfloat16* wp = M.w2 + (size_t)(c0 + d) * M.ld2;
-            for (int c = sub * 8; c < rk; c += 32) {
-                float x[8];
-                Chunk16<__nv_bfloat16>::load(wp + c, x);
 #pragma unroll
-                for (int i = 0; i < 8; i++) z = fmaf(x[i], inner[c + i], z);
+            for (int i = 0; i < kAhead; i++) {
+                const int c = (sub + 4 * i) * 8;
+                if (c < rk) {
+                    if (d0 > 0) w2[i] = __ldg(reinterpret_cast<const uint4*>(wp + c));
+                    const float4 x[2] = {*reinterpret_cast<const float4*>(inner + c), *reinterpret_cast<const float4*>(inner + c + 4)};
+                    z += Chunk<FMT_BF16>::dot(w2[i], x);
+                }
+            }
+            for (int c = (sub + 4 * kAhead) * 8; c < rk; c += 32) {
+                const float4 x[2] = {*reinterpret_cast<const float4*>(inner + c), *reinterpret_cast<const float4*>(inner + c + 4)};
+                z += Chunk<FMT_BF16>::dot(__ldg(reinterpret_cast<const uint4*>(wp + c)), x);
             }
         }
         z += __shfl_xor_sync(MG_FULL_MASK, z, 1);
         z += __shfl_xor_sync(MG_FULL_MASK, z, 2);
-        if (sub == 0 && d < D) w[d] = expf(-expf(z + M.w0[c0 + d]));
+        if (sub == 0 && d < D) w[d] = expf(-expf(z + (d0 > 0 ? M.w0[c0 + d] : w0)));
     }
     __syncthreads();
-    for (int v0 = 0; v0 < D; v0 += 32) {
+    for (int v0 = 0; v0 < D; v0 += 64) {
         const int col = v0 + lane;
-        const float vv = col < D ? v[col] : 0.f;
-        float o = 0.f;
+        const float va = col < D ? v[col] : 0.f, vb = col + 32 < D ? v[col + 32] : 0.f;
+        float oa = 0.f, ob = 0.f;
         for (int k0 = 0; k0 < D; k0 += kStepRows * nw) {
             if (v0 > 0 || k0 > 0) load_rows(k0, col);
 #pragma unroll
             for (int i = 0; i < kStepRows; i++) {
                 const int d = k0 + wid + i * nw;
                 if (d < D) {
-                    const float kv = k[d] * vv;
-                    o = fmaf(fmaf(u[d], kv, s0[i]), r[d], o);
-                    if (col < D) S[(size_t)d * D + col] = fmaf(w[d], s0[i], kv);
+                    const float ka = k[d] * va, kb = k[d] * vb;
+                    oa = fmaf(fmaf(u[d], ka, s0[i][0]), r[d], oa);
+                    ob = fmaf(fmaf(u[d], kb, s0[i][1]), r[d], ob);
+                    if (col < D) S[(size_t)d * D + col] = fmaf(w[d], s0[i][0], ka);
+                    if (col + 32 < D) S[(size_t)d * D + col + 32] = fmaf(w[d], s0[i][1], kb);
                 }
             }
         }
-        if (col < D) part[wid * D + col] = o;
+        if (col < D) part[wid * D + col] = oa;
+        if (col + 32 < D) part[wid * D + col + 32] = ob;
     }
     __syncthreads();
     float ss = 0.f;
@@ -89,7 +109,8 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvStep a)
         a.y[c0 + i] = part[i] * inv * M.norm[c0 + i] * silu(a.row[3 * (size_t)n + c0 + i]);
 }
 
-template <typename AT>
+// V values per thread and step (4 where rows are whole quads).
+template <typename AT, int V>
 __global__ void __launch_bounds__(256) wkv_mix_kernel(const float* h, const float* prev, const float* m0, const float* m1, const float* m2,
                                                       const float* m3, const float* m4, int pos0, int width, AT* act, int ld_act,
                                                       long long stride) {
@@ -98,74 +119,118 @@ __global__ void __launch_bounds__(256) wkv_mix_kernel(const float* h, const floa
     const float* before = t > 0 ? cur - width : prev + (size_t)(pos0 & 1) * width;
     const bool none = t == 0 && pos0 == 0;
     const float* mu[5] = {m0, m1, m2, m3, m4};
-    for (int i = threadIdx.x; i < width; i += 256) {
-        const float x = cur[i], d = (none ? 0.f : before[i]) - x;
+    for (int i = threadIdx.x * V; i < width; i += 256 * V) {
+        float x[V], d[V];
+        load_values<V>(cur + i, x);
+        if (none) {
 #pragma unroll
-        for (int j = 0; j < 5; j++) from_f32(fmaf(d, mu[j][i], x), act + j * stride + (size_t)t * ld_act + i);
+            for (int q = 0; q < V; q++) d[q] = 0.f;
+        } else {
+            load_values<V>(before + i, d);
+        }
+#pragma unroll
+        for (int j = 0; j < 5; j++) {
+            float m[V];
+            load_values<V>(mu[j] + i, m);
+#pragma unroll
+            for (int q = 0; q < V; q++) m[q] = fmaf(d[q] - x[q], m[q], x[q]);
+            store_values<V>(m, act + j * stride + (size_t)t * ld_act + i);
+        }
     }
 }
 
 // ---- prompts ----
-constexpr int kScanThreads = 128;
+constexpr int kScanWarps = 8, kScanThreads = kScanWarps * 32;
+constexpr int kScanCols = 2;        // value channels per warp
+constexpr int kScanGroup = 8;       // tokens whose sums are reduced together
 
-// KS lanes share a column of the state, KPT key channels each: lane j holds channels 4 (j + q KS) .. + 3.  Tokens
-// come through shared memory in tiles; sums over key channels of KS tokens are reduced at once, which leaves
-// lane j with token j's output.
-template <int KPT, int KS>
-struct Scan {
-    static constexpr int cols = kScanThreads / KS;      // value channels per CTA
-    static constexpr int rows = KPT * KS;               // key channels, padded
-};
+// A lane's N neighbouring key channels as pairs (quads 32 lanes apart where N > 4).
+template <int N>
+__device__ __forceinline__ void lds_pairs(const float* p, int lane, unsigned long long (&o)[N / 2]) {
+    if constexpr (N == 2) {
+        o[0] = *reinterpret_cast<const unsigned long long*>(p + 2 * lane);
+    } else {
+#pragma unroll
+        for (int q = 0; q < N / 4; q++) {
+            const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p + 4 * (lane + 32 * q));
+            o[2 * q] = v.x; o[2 * q + 1] = v.y;
+        }
+    }
+}
+template <int KPT>
+__device__ __forceinline__ int scan_channel(int lane, int i) { return KPT == 2 ? 2 * lane + i : 4 * (lane + i / 4 * 32) + i % 4; }
 
-// A token in shared memory: r, k, w padded to `rows`, then the CTA's value channels.
-template <int KPT, int KS>
+// A warp owns two columns of a head's state, its lanes KPT key channels each, two at a time in packed arithmetic.
+// Tokens come through shared memory in tiles: r, k, w padded to 32 KPT channels, then the CTA's value channels.
+// A sum over key channels is one over lanes; those of eight tokens x two columns are reduced at once by halving
+// exchanges, which leave lanes 2 i and 2 i + 1 with token i / 2 and column i % 2.
+template <int KPT>
 __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const Wkv M, const float* proj, int ldp, const float* decay, int pos0, int n,
                                                                 int tile, float* out) {
     extern __shared__ __align__(16) float smem[];
-    using G = Scan<KPT, KS>;
-    constexpr int Q = KPT / 4;
-    const int D = M.dim, nh = M.heads * D, h = blockIdx.x, v0 = blockIdx.y * G::cols;
-    const int sub = threadIdx.x % KS, col = threadIdx.x / KS, v = v0 + col;
-    constexpr int per = 3 * G::rows + (G::cols + 3) / 4 * 4;
-    const int cols = min(G::cols, D - v0);
+    constexpr int rows = 32 * KPT, per = 3 * rows + kScanWarps * kScanCols, P = KPT / 2, NO = kScanGroup * kScanCols;
+    const int D = M.dim, nh = M.heads * D, h = blockIdx.x, v0 = blockIdx.y * kScanWarps * kScanCols;
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, vw = v0 + wid * kScanCols;
+    const int cols = min(kScanWarps * kScanCols, D - v0);
     // the padding is zero and stays so
     for (int i = threadIdx.x; i < 2 * tile * per; i += kScanThreads) smem[i] = 0.f;
     __syncthreads();
     const bool wide = ((D | ldp) & 3) == 0;
-    auto load = [&](int buf, int t0) {
+    auto load = [&](int buf, int t0) {              // a warp per token
         const int T = min(tile, n - t0);
-        float* dst = smem + (size_t)buf * tile * per;
-        const int step = wide ? 4 : 1, units = D / step;
-        for (int i = threadIdx.x; i < T * units; i += kScanThreads) {
-            const int t = i / units, c = (i - t * units) * step;
-            const float* row = proj + (size_t)(t0 + t) * ldp + h * D + c;
-            const float* dw = decay + (size_t)(t0 + t) * nh + h * D + c;
-            float* to = dst + t * per + c;
+        for (int t = wid; t < T; t += kScanWarps) {
+            float* to = smem + ((size_t)buf * tile + t) * per;
+            const float* row = proj + (size_t)(t0 + t) * ldp + h * D;
+            const float* dw = decay + (size_t)(t0 + t) * nh + h * D;
             if (wide) {
-                cp_async16(to, row);
-                cp_async16(to + G::rows, row + nh);
-                cp_async16(to + 2 * G::rows, dw);
+                for (int c = lane * 4; c < D; c += 128) {
+                    cp_async16(to + c, row + c);
+                    cp_async16(to + rows + c, row + nh + c);
+                    cp_async16(to + 2 * rows + c, dw + c);
+                }
             } else {
-                cp_async4(to, row);
-                cp_async4(to + G::rows, row + nh);
-                cp_async4(to + 2 * G::rows, dw);
+                for (int c = lane; c < D; c += 32) {
+                    cp_async4(to + c, row + c);
+                    cp_async4(to + rows + c, row + nh + c);
+                    cp_async4(to + 2 * rows + c, dw + c);
+                }
             }
-        }
-        for (int i = threadIdx.x; i < T * cols; i += kScanThreads) {
-            const int t = i / cols, c = i - t * cols;
-            cp_async4(dst + t * per + 3 * G::rows + c, proj + (size_t)(t0 + t) * ldp + 2 * (size_t)nh + h * D + v0 + c);
+            for (int c = lane; c < cols; c += 32) cp_async4(to + 3 * rows + c, row + 2 * (size_t)nh + v0 + c);
         }
     };
     load(0, 0);
     cp_async_commit();
-    float S[KPT], u[KPT];
+    unsigned long long S[kScanCols][P], u[P];
 #pragma unroll
-    for (int i = 0; i < KPT; i++) {
-        const int d = 4 * (sub + i / 4 * KS) + i % 4;
-        const bool in = d < D && v < D;
-        u[i] = d < D ? M.u[h * D + d] : 0.f;
-        S[i] = in && pos0 > 0 ? M.S[((size_t)h * D + d) * D + v] : 0.f;
+    for (int i = 0; i < P; i++) {
+        const int d = scan_channel<KPT>(lane, 2 * i);       // and the next
+        u[i] = pack2(d < D ? M.u[h * D + d] : 0.f, d + 1 < D ? M.u[h * D + d + 1] : 0.f);
+#pragma unroll
+        for (int c = 0; c < kScanCols; c++) {
+            const float* s = M.S + ((size_t)h * D + d) * D + vw + c;
+            const bool in = vw + c < D && pos0 > 0;
+            S[c][i] = pack2(in && d < D ? s[0] : 0.f, in && d + 1 < D ? s[D] : 0.f);
+        }
     }
+    auto token = [&](const float* p, float* o) {
+        unsigned long long r[P], k[P], w[P];
+        lds_pairs<KPT>(p, lane, r);
+        lds_pairs<KPT>(p + rows, lane, k);
+        lds_pairs<KPT>(p + 2 * rows, lane, w);
+        const float2 v2 = *reinterpret_cast<const float2*>(p + 3 * rows + wid * kScanCols);
+        const unsigned long long v[kScanCols] = {pack2(v2.x, v2.x), pack2(v2.y, v2.y)};
+#pragma unroll
+        for (int c = 0; c < kScanCols; c++) {
+            unsigned long long sum = 0ull;
+#pragma unroll
+            for (int i = 0; i < P; i++) {
+                const unsigned long long kv = mul2(k[i], v[c]);
+                sum = fma2(fma2(u[i], kv, S[c][i]), r[i], sum);
+                S[c][i] = fma2(w[i], S[c][i], kv);
+            }
+            o[c] = lo(sum) + hi(sum);
+        }
+    };
     int buf = 0;
     for (int t0 = 0; t0 < n; t0 += tile, buf ^= 1) {
         if (t0 + tile < n) load(buf ^ 1, t0 + tile);
@@ -174,59 +239,60 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const Wkv M, con
         __syncthreads();
         const float* base = smem + (size_t)buf * tile * per;
         const int T = min(tile, n - t0);
-        for (int g = 0; g < T; g += KS) {
-            float o[KS];
+        for (int g = 0; g < T; g += kScanGroup) {
+            float o[NO];
+            if (g + kScanGroup <= T) {
 #pragma unroll
-            for (int j = 0; j < KS; j++) {
-                o[j] = 0.f;
-                if (g + j < T) {
-                    const float* p = base + (g + j) * per + 4 * sub;
-                    const float vv = base[(g + j) * per + 3 * G::rows + col];
+                for (int j = 0; j < kScanGroup; j++) token(base + (g + j) * per, o + j * kScanCols);
+            } else {
 #pragma unroll
-                    for (int q = 0; q < Q; q++) {
-                        const float4 r4 = *reinterpret_cast<const float4*>(p + 4 * q * KS), k4 = *reinterpret_cast<const float4*>(p + G::rows + 4 * q * KS),
-                                     w4 = *reinterpret_cast<const float4*>(p + 2 * G::rows + 4 * q * KS);
-                        const float rr[4] = {r4.x, r4.y, r4.z, r4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, ww[4] = {w4.x, w4.y, w4.z, w4.w};
-#pragma unroll
-                        for (int i = 0; i < 4; i++) {
-                            const float kv = kk[i] * vv;
-                            o[j] = fmaf(fmaf(u[4 * q + i], kv, S[4 * q + i]), rr[i], o[j]);
-                            S[4 * q + i] = fmaf(ww[i], S[4 * q + i], kv);
-                        }
-                    }
-                }
+                for (int j = 0; j < kScanGroup; j++)
+                    if (g + j < T) token(base + (g + j) * per, o + j * kScanCols);
             }
-            // halves exchange until lane `sub` holds token `sub`'s sum
 #pragma unroll
-            for (int m = KS / 2; m > 0; m >>= 1) {
-                const bool up = (sub & m) != 0;
+            for (int m = NO / 2; m > 0; m >>= 1) {
+                const bool up = (lane & (2 * m)) != 0;
 #pragma unroll
                 for (int j = 0; j < m; j++) {
                     const float give = up ? o[j] : o[j + m], keep = up ? o[j + m] : o[j];
-                    o[j] = keep + __shfl_xor_sync(MG_FULL_MASK, give, m);
+                    o[j] = keep + __shfl_xor_sync(MG_FULL_MASK, give, 2 * m);
                 }
             }
-            if (g + sub < T && v < D) out[(size_t)(t0 + g + sub) * nh + h * D + v] = o[0];
+            o[0] += __shfl_xor_sync(MG_FULL_MASK, o[0], 1);
+            const int t = g + (lane >> 2), v = vw + ((lane >> 1) & 1);
+            if ((lane & 1) == 0 && t < T && v < D) out[(size_t)(t0 + t) * nh + h * D + v] = o[0];
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int i = 0; i < KPT; i++) {
-        const int d = 4 * (sub + i / 4 * KS) + i % 4;
-        if (d < D && v < D) M.S[((size_t)h * D + d) * D + v] = S[i];
+    for (int i = 0; i < P; i++) {
+        const int d = scan_channel<KPT>(lane, 2 * i);
+#pragma unroll
+        for (int c = 0; c < kScanCols; c++) {
+            float* s = M.S + ((size_t)h * D + d) * D + vw + c;
+            if (vw + c < D && d < D) s[0] = lo(S[c][i]);
+            if (vw + c < D && d + 1 < D) s[D] = hi(S[c][i]);
+        }
     }
 }
 
-template <int KPT, int KS>
+template <int KPT>
 cudaError_t scan_for(const Wkv& wk, const float* proj, int ldp, const float* decay, int pos0, int n, float* out, cudaStream_t s) {
-    using G = Scan<KPT, KS>;
-    constexpr int per = 3 * G::rows + (G::cols + 3) / 4 * 4;
-    int tile = 32;
-    while (tile > KS && 2 * (size_t)tile * per * sizeof(float) > 100 * 1024) tile /= 2;
-    const size_t smem = 2 * (size_t)tile * per * sizeof(float);
-    static cudaError_t attr = cudaFuncSetAttribute((const void*)wkv_scan_kernel<KPT, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    constexpr int per = 3 * 32 * KPT + kScanWarps * kScanCols, tile = KPT <= 4 ? 32 : KPT == 8 ? 16 : 8;
+    constexpr size_t smem = 2 * (size_t)tile * per * sizeof(float);
+    static_assert(tile % kScanGroup == 0 && smem <= 227 * 1024, "a tile holds whole groups");
+    static cudaError_t attr = cudaFuncSetAttribute((const void*)wkv_scan_kernel<KPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (attr != cudaSuccess) return attr;
-    wkv_scan_kernel<KPT, KS><<<dim3(wk.heads, (wk.dim + G::cols - 1) / G::cols), kScanThreads, smem, s>>>(wk, proj, ldp, decay, pos0, n, tile, out);
+    wkv_scan_kernel<KPT><<<dim3(wk.heads, (wk.dim + kScanWarps * kScanCols - 1) / (kScanWarps * kScanCols)), kScanThreads, smem, s>>>(
+        wk, proj, ldp, decay, pos0, n, tile, out);
+    return cudaGetLastError();
+}
+
+template <typename AT>
+cudaError_t mix_for(const float* h, const float* prev, const float* const mu[5], int pos0, int n, int width, AT* act, int ld_act, long long stride,
+                    cudaStream_t s) {
+    if (width % 4 == 0) wkv_mix_kernel<AT, 4><<<n, 256, 0, s>>>(h, prev, mu[0], mu[1], mu[2], mu[3], mu[4], pos0, width, act, ld_act, stride);
+    else wkv_mix_kernel<AT, 1><<<n, 256, 0, s>>>(h, prev, mu[0], mu[1], mu[2], mu[3], mu[4], pos0, width, act, ld_act, stride);
     return cudaGetLastError();
 }
 
@@ -240,19 +306,17 @@ cudaError_t launch_wkv_step(const WkvStep& a, bool pdl, cudaStream_t s) {
 
 cudaError_t launch_wkv_mix(const float* h, const float* prev, const float* const mu[5], int pos0, int n, int width, void* act, int ld_act,
                            long long act_stride, bool f32, cudaStream_t s) {
-    if (f32) wkv_mix_kernel<float><<<n, 256, 0, s>>>(h, prev, mu[0], mu[1], mu[2], mu[3], mu[4], pos0, width, (float*)act, ld_act, act_stride);
-    else wkv_mix_kernel<__nv_bfloat16><<<n, 256, 0, s>>>(h, prev, mu[0], mu[1], mu[2], mu[3], mu[4], pos0, width, (__nv_bfloat16*)act, ld_act, act_stride);
-    return cudaGetLastError();
+    return f32 ? mix_for(h, prev, mu, pos0, n, width, (float*)act, ld_act, act_stride, s)
+               : mix_for(h, prev, mu, pos0, n, width, (__nv_bfloat16*)act, ld_act, act_stride, s);
 }
 
 bool wkv_rows_fits(const Wkv& wk) { return wk.dim <= 512; }
 
 cudaError_t launch_wkv_rows(const Wkv& wk, const float* proj, int ldp, const float* decay, int pos0, int n, float* out, cudaStream_t s) {
-    if (wk.dim <= 32) return scan_for<8, 4>(wk, proj, ldp, decay, pos0, n, out, s);
-    if (wk.dim <= 64) return scan_for<8, 8>(wk, proj, ldp, decay, pos0, n, out, s);
-    if (wk.dim <= 128) return scan_for<8, 16>(wk, proj, ldp, decay, pos0, n, out, s);
-    if (wk.dim <= 256) return scan_for<16, 16>(wk, proj, ldp, decay, pos0, n, out, s);
-    if (wk.dim <= 512) return scan_for<32, 16>(wk, proj, ldp, decay, pos0, n, out, s);
+    if (wk.dim <= 64) return scan_for<2>(wk, proj, ldp, decay, pos0, n, out, s);
+    if (wk.dim <= 128) return scan_for<4>(wk, proj, ldp, decay, pos0, n, out, s);
+    if (wk.dim <= 256) return scan_for<8>(wk, proj, ldp, decay, pos0, n, out, s);
+    if (wk.dim <= 512) return scan_for<16>(wk, proj, ldp, decay, pos0, n, out, s);
     return cudaErrorInvalidValue;
 }
 

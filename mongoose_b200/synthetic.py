@@ -11,7 +11,8 @@ from __future__ import annotations
 import numpy as np
 
 from . import configs as mc
-from .layered import GateAttention, LayeredConfig, MatrixMemory, ParallelLayer, slot_shapes
+from .layered import (NORM_LAYER, POS_NONE, GateAttention, LatentAttention, LayeredConfig, Loop, MatrixMemory, MixtureOfExperts,
+                      ParallelLayer, PrenormLayer, Wkv, slot_shapes)
 from .safetensors import to_bf16_bits
 
 
@@ -91,19 +92,36 @@ def mitotar_like(name: str, width: int, n_layers: int, ffn: int, vocab: int, hea
     return LayeredConfig(name=name, width=width, vocab=vocab, layers=(layer,) * n_layers, norm_eps=1e-6, max_seq=max_seq)
 
 
-# layer widths of the dense configurations of the same name
+def kuzipel_like(name: str, width: int, n_layers: int, vocab: int, attn: LatentAttention, wkv: Wkv, moe: MixtureOfExperts,
+                 max_seq: int) -> LayeredConfig:
+    """`n_layers` layer runs: one attention layer, then two recurrent ones, and so on, the first recurrent one twice."""
+    layers = tuple(PrenormLayer(wkv if i % 3 else attn, moe) for i in range(n_layers - 1))
+    return LayeredConfig(name=name, width=width, vocab=vocab, layers=layers, norm_eps=1e-5, max_seq=max_seq, norm=NORM_LAYER,
+                         positions=POS_NONE, residual_mult=0.5, loop=Loop(1, 2, 2))
+
+
+def latent_like(heads: int, dim: int, rot_dim: int, q_rank: int, kv_rank: int) -> LatentAttention:
+    return LatentAttention(heads, dim, rot_dim, dim, q_rank, kv_rank, (dim + rot_dim) ** -0.5, 10000.0)
+
+
+# layer widths of the dense configurations of the same name; a token's experts together are as wide as their feed-forward
 LAYERED = {c.name: c for c in (
     mitotar_like("mitotar-tiny", 96, 2, 160, 300, 4, 2, 24, 3, 20, 256),
     mitotar_like("mitotar-0.5b", 896, 24, 4864, 151936, 14, 2, 64, 4, 128, 4096),
     mitotar_like("mitotar-1.1b", 2048, 22, 5632, 32000, 32, 4, 64, 8, 128, 4096),
     mitotar_like("mitotar-7b-width-4l", 3584, 4, 18944, 16000, 28, 4, 128, 8, 256, 4096),
+    kuzipel_like("kuzipel-tiny", 96, 5, 300, latent_like(3, 24, 8, 40, 56), Wkv(4, 20, 12), MixtureOfExperts(5, 2, 40, 72), 256),
+    kuzipel_like("kuzipel-0.5b", 896, 24, 151936, latent_like(14, 64, 32, 384, 256), Wkv(14, 64, 64), MixtureOfExperts(16, 4, 608, 2432), 4096),
+    kuzipel_like("kuzipel-1.1b", 2048, 22, 32000, latent_like(16, 128, 64, 768, 512), Wkv(32, 64, 64), MixtureOfExperts(16, 4, 704, 2816), 4096),
+    kuzipel_like("kuzipel-7b-width-4l", 3584, 4, 16000, latent_like(28, 128, 64, 1536, 512), Wkv(56, 64, 64),
+                 MixtureOfExperts(16, 4, 2368, 9472), 4096),
 )}
 
 
 def layered_tensors(cfg: LayeredConfig, seed: int = 0):
     """Yield (slot, name, layer, fp32 tensor) of a random-init model: matrices N(0, 1 / fan-in), head mixing
     near the identity, norm weights and biases jittered around their neutral value."""
-    around_zero = {"norm1", "norm2", "final_norm", "at.bias", "mem.i_bias"}
+    around_zero = {"at.bias", "mem.i_bias", "moe.bias"} | ({"norm1", "norm2", "final_norm"} if cfg.norm != NORM_LAYER else set())
     for idx, name, layer, rows, cols in slot_shapes(cfg):
         rng = np.random.default_rng([seed, idx])
         if rows:
@@ -113,7 +131,7 @@ def layered_tensors(cfg: LayeredConfig, seed: int = 0):
             n = cfg.layers[layer].attn.heads
             w = (np.eye(n) + 0.3 * n ** -0.5 * rng.standard_normal((n, n))).astype(np.float32).reshape(-1)
         else:
-            neutral = 0.0 if name in around_zero else 3.0 if name == "mem.f_bias" else 1.0
+            neutral = 0.0 if name in around_zero else 3.0 if name == "mem.f_bias" else -2.0 if name == "wkv.w0" else 0.5 if "mu_" in name else 1.0
             w = (neutral + 0.2 * rng.standard_normal(cols)).astype(np.float32)
         yield idx, name, layer, w
 
