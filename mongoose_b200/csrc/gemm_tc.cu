@@ -1,7 +1,8 @@
 // out = A B^T for bf16 A [m][k] and B [n][k], fp32 accumulation: one 128 x BN tile per CTA.  Warp 0 streams both
 // operands with TMA into a ring of 64-column stages, one thread of warp 1 issues tcgen05.mma into TMEM,
 // warps 2-5 read the accumulator back and store it row by row through shared memory.  Two CTAs share an
-// SM, so one's epilogue runs under the other's products.
+// SM, so one's epilogue runs under the other's products; where there are fewer tiles than SMs, a CTA has the
+// SM to itself and a ring deep enough to cover the latency of its copies.
 #include "gemm_tc.h"
 #include "layered_ops.cuh"
 #include "umma.cuh"
@@ -11,7 +12,8 @@ namespace mg {
 namespace {
 
 constexpr int kThreads = 192;
-constexpr int kStages = 3;
+constexpr int kShallow = 3;
+constexpr int deep(int bn) { return bn == 64 ? 8 : 6; }
 
 // gelu for results that are rounded to bf16: tanh from one fast exponential
 __device__ __forceinline__ float gelu_tanh_fast(float z) {
@@ -21,17 +23,17 @@ __device__ __forceinline__ float gelu_tanh_fast(float z) {
 
 __device__ __forceinline__ float silu_fast(float z) { return z * __fdividef(1.0f, 1.0f + __expf(-z)); }
 
-template <int BN>
+template <int BN, int kStages>
 struct Smem {
     static constexpr int a_bytes = 128 * 128, b_bytes = BN * 128, stage = a_bytes + b_bytes;
     static constexpr int bytes = kStages * stage + 1024 + 256;      // + alignment + barriers
 };
 
-template <int BN>
-__global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_constant__ GemmTC g) {
+template <int BN, int kStages>
+__global__ void __launch_bounds__(kThreads, kStages == kShallow ? 2 : 1) gemm_tc_kernel(const __grid_constant__ GemmTC g) {
     extern __shared__ uint8_t raw[];
     uint8_t* base = reinterpret_cast<uint8_t*>(((uintptr_t)raw + 1023) & ~(uintptr_t)1023);
-    uint64_t* full = reinterpret_cast<uint64_t*>(base + kStages * Smem<BN>::stage);
+    uint64_t* full = reinterpret_cast<uint64_t*>(base + kStages * Smem<BN, kStages>::stage);
     uint64_t* empty = full + kStages;
     uint64_t* done = empty + kStages;
     uint32_t* tmem_base = reinterpret_cast<uint32_t*>(done + 1);
@@ -67,11 +69,11 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
             for (int i = 0; i < kt; i++) {
                 const int s = i % kStages, use = i / kStages;
                 if (use > 0 && !bar_wait(empty + s, (use - 1) & 1, g.status)) break;
-                bar_expect(full + s, Smem<BN>::stage);
-                uint8_t* st = base + s * Smem<BN>::stage;
+                bar_expect(full + s, Smem<BN, kStages>::stage);
+                uint8_t* st = base + s * Smem<BN, kStages>::stage;
                 tma_load_3d(st, &g.a, i * 64, row0, z, full + s);
-                tma_load_3d(st + Smem<BN>::a_bytes, &g.b, i * 64, col0, zb, full + s);
-                if (dual) tma_load_3d(st + Smem<BN>::a_bytes + 64 * 128, &g.b2, i * 64, col0, zb, full + s);
+                tma_load_3d(st + Smem<BN, kStages>::a_bytes, &g.b, (g.b_steps ? i % g.b_steps : i) * 64, col0, zb, full + s);
+                if (dual) tma_load_3d(st + Smem<BN, kStages>::a_bytes + 64 * 128, &g.b2, i * 64, col0, zb, full + s);
                 issued = i + 1;
             }
             // no copy may be in flight when the CTA leaves
@@ -86,7 +88,7 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
                 ok = bar_wait(full + s, (i / kStages) & 1, g.status);
                 if (!ok) break;
                 tc_fence_after();
-                const uint64_t da = tile_desc(base + s * Smem<BN>::stage), db = tile_desc(base + s * Smem<BN>::stage + Smem<BN>::a_bytes);
+                const uint64_t da = tile_desc(base + s * Smem<BN, kStages>::stage), db = tile_desc(base + s * Smem<BN, kStages>::stage + Smem<BN, kStages>::a_bytes);
 #pragma unroll
                 for (int k = 0; k < 4; k++) mma_bf16(acc, da + 2 * k, db + 2 * k, mma_desc(BN), i > 0 || k > 0);
                 mma_commit(empty + s);
@@ -113,13 +115,16 @@ __global__ void __launch_bounds__(kThreads, 2) gemm_tc_kernel(const __grid_const
 #pragma unroll
                 for (int i = 0; i < 32; i++) tile[lane * 33 + i] = v[i];
                 __syncwarp();
-                if (g.mode == GEMM_F32) {
+                if (g.mode == GEMM_F32 || g.mode == GEMM_DECAY_F32) {
                     const int col = col0 + c + lane;
                     float* out = static_cast<float*>(g.out) + z * g.batch_c + col;
+                    const float bias = g.mode == GEMM_DECAY_F32 && col < g.n ? g.bias[col] : 0.f;
 #pragma unroll 8
                     for (int r = 0; r < 32; r++) {
                         const int row = row0 + quarter * 32 + r;
-                        if (row < g.m && col < g.n) out[row * g.ldc] = tile[r * 33 + lane];
+                        float x = tile[r * 33 + lane];
+                        if (g.mode == GEMM_DECAY_F32) x = expf(-expf(x + bias));
+                        if (row < g.m && col < g.n) out[row * g.ldc] = x;
                     }
                 } else {                            // two columns per lane, two rows at a time
                     const int col = col0 + c + 2 * (lane & 15);
@@ -171,13 +176,29 @@ bool encode(CUtensorMap* map, const void* base, const cuuint64_t dims[3], const 
                     CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
+template <int BN, int kStages>
+cudaError_t run(const GemmTC& g, dim3 grid, cudaStream_t s) {
+    constexpr int bytes = Smem<BN, kStages>::bytes;
+    static cudaError_t attr = cudaFuncSetAttribute((const void*)gemm_tc_kernel<BN, kStages>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (attr != cudaSuccess) return attr;
+    gemm_tc_kernel<BN, kStages><<<grid, kThreads, bytes, s>>>(g);
+    return cudaGetLastError();
+}
+
+int sm_count() {
+    static const int n = [] {
+        int dev = 0, v = 0;
+        return cudaGetDevice(&dev) == cudaSuccess && cudaDeviceGetAttribute(&v, cudaDevAttrMultiProcessorCount, dev) == cudaSuccess ? v : 0;
+    }();
+    return n;
+}
+
 template <int BN>
 cudaError_t run(const GemmTC& g, cudaStream_t s) {
-    static cudaError_t attr = cudaFuncSetAttribute((const void*)gemm_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<BN>::bytes);
-    if (attr != cudaSuccess) return attr;
     const int cols = g.mode == GEMM_SILU_BF16 ? 64 : BN;
-    gemm_tc_kernel<BN><<<dim3((g.n + cols - 1) / cols, (g.m + 127) / 128, g.batch), kThreads, Smem<BN>::bytes, s>>>(g);
-    return cudaGetLastError();
+    const dim3 grid((g.n + cols - 1) / cols, (g.m + 127) / 128, g.batch);
+    const bool few = (long long)grid.x * grid.y * grid.z <= sm_count() && g.k > kShallow * 64;
+    return few ? run<BN, deep(BN)>(g, grid, s) : run<BN, kShallow>(g, grid, s);
 }
 
 }  // namespace

@@ -7,7 +7,8 @@
 namespace mg {
 
 enum : int { GEMM_F32 = 0, GEMM_BF16 = 1, GEMM_GELU_BF16 = 2,
-             GEMM_SILU_BF16 = 3 };      // two matrices on one input: silu(A B^T) * (A B2^T)
+             GEMM_SILU_BF16 = 3,        // two matrices on one input: silu(A B^T) * (A B2^T)
+             GEMM_DECAY_F32 = 4 };      // exp(-exp(A B^T + bias))
 
 // A 3-D bf16 tensor [batch][rows][k] seen by TMA in boxes of box_rows x 64 columns (128-byte swizzle); the
 // part of a box outside the tensor reads as zero.  Strides in elements, multiples of 8.
@@ -22,6 +23,8 @@ struct GemmTC {
     CUtensorMap b2;         // GEMM_SILU_BF16: the second matrix, boxes of 64 rows
     int bn;                 // 64 or 128; GEMM_SILU_BF16: 128, n in steps of 64
     int m, n, k;            // out[m][n], k columns (rounded up to 64 inside)
+    int b_steps;            // > 0: b has this many steps of 64 columns, a several times as many: a = [a1 a2 ..] multiplies [b b ..]
+    const float* bias;      // [n], GEMM_DECAY_F32
     int batch, b_group;     // batch z multiplies a's batch z with b's batch z / b_group
     const int* group;       // not NULL: row tile y multiplies b's batch group[y]; -1: the tile is empty
     int causal_pos0;        // >= 0: row r only needs columns k <= causal_pos0 + r (the rest of a is zero)

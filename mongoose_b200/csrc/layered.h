@@ -170,6 +170,8 @@ size_t wkv_step_smem(const Wkv& wk);
 // act[j][r] = the mix of row r and the one before it (prev before the first) with mu[j]
 cudaError_t launch_wkv_mix(const float* h, const float* prev, const float* const mu[5], int pos0, int n, int width, void* act, int ld_act,
                            long long act_stride, bool f32, cudaStream_t s);
+// act[n][ld] = tanh of the decay's inner projection as two bf16 parts
+cudaError_t launch_wkv_inner(const float* inner, int ldp, int rank, int n, void* act, int ld, cudaStream_t s);
 bool wkv_rows_fits(const Wkv& wk);
 // proj rows as WkvStep's, decays [n][heads * dim]; out [n][heads * dim] raw outputs
 cudaError_t launch_wkv_rows(const Wkv& wk, const float* proj, int ldp, const float* decay, int pos0, int n, float* out, cudaStream_t s);

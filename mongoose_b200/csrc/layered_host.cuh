@@ -90,7 +90,7 @@ struct Layered {
     uint8_t *aw = nullptr, *vt = nullptr;   // tensor-core attention: mixed weights of a query block, transposed keys or values
     uint8_t* keys = nullptr;            // keys formed from latents
     float *x0r = nullptr, *hr = nullptr, *q32 = nullptr, *decay = nullptr, *wo = nullptr, *rtr = nullptr, *glu = nullptr;
-    uint8_t *cat = nullptr, *mix = nullptr, *cq = nullptr, *xmid = nullptr;
+    uint8_t *cat = nullptr, *mix = nullptr, *inner = nullptr, *cq = nullptr, *xmid = nullptr;
     MoeRows moe{};
     MemRows mw{};
     int np = 0;                         // widest projection row
@@ -111,7 +111,7 @@ int layered_buffers(Layered& m, F take) {
         if (!rc && count) rc = take((void**)p, count * elem);
     };
     size_t hd = 0, kat = 1, kmem = 0, ff = 0, mh = 0, u = 0, nu = 0, part = 0, aw = 0, vt = 0;
-    size_t q1 = 0, q32 = 0, qa = 0, lpart = 0, ml = 0, keys = 0, cq = 0, wkv = 0, rt = 0, rtr = 0, emid = 0, xmid = 0, moe = 0, tiles = 0, top = 0, experts = 0;
+    size_t q1 = 0, q32 = 0, qa = 0, lpart = 0, ml = 0, keys = 0, cq = 0, wkv = 0, ld2 = 0, rt = 0, rtr = 0, emid = 0, xmid = 0, moe = 0, tiles = 0, top = 0, experts = 0;
     bool any_post = false, any_pre = false;
     for (size_t i = 0; i < m.layers.size(); i++) {
         LayerWeights& l = m.layers[i];
@@ -177,7 +177,7 @@ int layered_buffers(Layered& m, F take) {
             for (float*& v : l.mu) get(&v, W, 4);
             get(&l.w2, (size_t)n * l.wk.ld2, 2);
             get(&l.w0, n, 4); get(&l.u, n, 4); get(&l.wkv_norm, n, 4);
-            wkv = std::max(wkv, (size_t)n);
+            wkv = std::max(wkv, (size_t)n); ld2 = std::max(ld2, (size_t)2 * l.wk.ld2);
         }
         if (l.moe.experts) {
             const Moe& e = l.moe;
@@ -225,7 +225,7 @@ int layered_buffers(Layered& m, F take) {
     get(&m.my, (size_t)T * kmem, as); get(&m.midr, (size_t)T * ff, as); get(&m.fin, (size_t)m.logit_rows * kw, as);
     get(&m.aw, aw, 2); get(&m.vt, vt, 2); get(&m.keys, keys, 2);
     get(&m.q32, q32, 4); get(&m.cq, (size_t)T * cq, as);
-    if (wkv) { get(&m.hr, (size_t)T * W, 4); get(&m.mix, (size_t)5 * T * kw, as); get(&m.decay, (size_t)T * wkv, 4); get(&m.wo, (size_t)T * wkv, 4); }
+    if (wkv) { get(&m.hr, (size_t)T * W, 4); get(&m.mix, (size_t)5 * T * kw, as); get(&m.decay, (size_t)T * wkv, 4); get(&m.wo, (size_t)T * wkv, 4); get(&m.inner, m.f32 ? 0 : (size_t)T * ld2, 2); }
     get(&m.rtr, (size_t)T * rtr, 4); get(&m.xmid, xmid, as); get(&m.glu, m.f32 ? xmid : 0, 4);
     get(&m.moe.sel, (size_t)T * top, 4); get(&m.moe.slot, (size_t)T * top, 4); get(&m.moe.weight, (size_t)T * top, 4);
     get(&m.moe.count, experts, 4); get(&m.moe.first, experts ? experts + 1 : 0, 4); get(&m.moe.group, tiles, 4);
@@ -882,10 +882,25 @@ int wkv_rows(mg_engine* e, const LayerRun& run, LayerWeights& l, int pos, int n)
     MG_CUDA(e, cudaMemcpyAsync(run.prev + (size_t)((pos + n) & 1) * W, m.hr + (size_t)(n - 1) * W, (size_t)W * 4, cudaMemcpyDeviceToDevice, s));
     if ((rc = layered_matmul_batch(e, m.mix, stride, m.max_rows, kw, l.proj, m.P, np, n, d, 4))) return rc;
     if ((rc = layered_matmul(e, m.mix + 4 * stride * (m.f32 ? 4 : 2), m.max_rows, kw, l.proj + (size_t)4 * d * kw * 2, m.P + (size_t)4 * d, np, n, wk.rank, false))) return rc;
-    GemmF32 g{};
-    g.A = m.P + (size_t)4 * d; g.lda = np; g.W = l.w2; g.ldw = wk.ld2; g.out = m.decay; g.ldc = d; g.n = n; g.rows = d; g.K = wk.rank;
-    g.epi = F32_DECAY; g.bias = l.w0;
-    MG_CUDA(e, launch_gemm_f32(g, s));
+    // decays: the inner vector stays 32-bit, on the tensor cores as a high and a low part
+    if (m.f32) {
+        GemmF32 g{};
+        g.A = m.P + (size_t)4 * d; g.lda = np; g.W = l.w2; g.ldw = wk.ld2; g.out = m.decay; g.ldc = d; g.n = n; g.rows = d; g.K = wk.rank;
+        g.epi = F32_DECAY; g.bias = l.w0;
+        MG_CUDA(e, launch_gemm_f32(g, s));
+    } else {
+        const int ld = 2 * wk.ld2;
+        MG_CUDA(e, launch_wkv_inner(m.P + (size_t)4 * d, np, wk.rank, n, m.inner, ld, s));
+        GemmTC g{};
+        g.bn = d > 64 ? 128 : 64;
+        if (!make_tile_map(&g.a, m.inner, ld, m.max_rows, 1, ld, (long long)m.max_rows * ld, 128) ||
+            !make_tile_map(&g.b, l.w2, wk.ld2, d, 1, wk.ld2, (long long)d * wk.ld2, g.bn))
+            return fail(e, MG_ERR_CUDA, "tensor map of a %d x %d product failed", d, ld);
+        g.m = n; g.n = d; g.k = ld; g.batch = 1; g.b_group = 1; g.causal_pos0 = -1; g.b_steps = wk.ld2 / 64;
+        g.out = m.decay; g.ldc = d; g.mode = GEMM_DECAY_F32; g.bias = l.w0; g.status = m.status;
+        MG_CUDA(e, launch_gemm_tc(g, s));
+        e->launches += 1;
+    }
     MG_CUDA(e, launch_wkv_rows(wk, m.P, np, m.decay, pos, n, m.wo, s));
     MG_CUDA(e, launch_head_norm_rows(wk.heads, wk.dim, wk.eps, wk.norm, m.P + (size_t)3 * d, np, GATE_SILU, n, m.wo, m.ao, ko, m.f32, s));
     e->launches += 4;

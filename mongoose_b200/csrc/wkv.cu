@@ -139,12 +139,26 @@ __global__ void __launch_bounds__(256) wkv_mix_kernel(const float* h, const floa
     }
 }
 
+// act[t] = [high, low]: tanh of the decay's inner projection as two bf16 parts (16 bits of mantissa together), each padded
+// to ld / 2, so that a product of bf16 operands keeps it.
+__global__ void __launch_bounds__(256) wkv_inner_kernel(const float* inner, int ldp, int rank, int n, __nv_bfloat16* act, int ld) {
+    const int i = blockIdx.x * 256 + threadIdx.x, t = i / rank, c = i - t * rank;
+    if (t >= n) return;
+    const float v = tanhf(inner[(size_t)t * ldp + c]);
+    const __nv_bfloat16 high = __float2bfloat16_rn(v);
+    act[(size_t)t * ld + c] = high;
+    act[(size_t)t * ld + ld / 2 + c] = __float2bfloat16_rn(v - __bfloat162float(high));
+}
+
 // ---- prompts ----
 constexpr int kScanWarps = 8, kScanThreads = kScanWarps * 32;
-constexpr int kScanCols = 2;        // value channels per warp
-constexpr int kScanGroup = 8;       // tokens whose sums are reduced together
+constexpr int kScanTile = 32;       // tokens of a tile in shared memory
+constexpr int kScanStages = 3;
 
-// A lane's N neighbouring key channels as pairs (quads 32 lanes apart where N > 4).
+constexpr int kScanCols = 2;        // value channels per warp
+constexpr int kScanGroup = 16;      // tokens whose sums are reduced together
+
+// A lane's N key channels as pairs: neighbouring ones, quads 32 lanes apart where N > 4.
 template <int N>
 __device__ __forceinline__ void lds_pairs(const float* p, int lane, unsigned long long (&o)[N / 2]) {
     if constexpr (N == 2) {
@@ -160,46 +174,63 @@ __device__ __forceinline__ void lds_pairs(const float* p, int lane, unsigned lon
 template <int KPT>
 __device__ __forceinline__ int scan_channel(int lane, int i) { return KPT == 2 ? 2 * lane + i : 4 * (lane + i / 4 * 32) + i % 4; }
 
-// A warp owns two columns of a head's state, its lanes KPT key channels each, two at a time in packed arithmetic.
-// Tokens come through shared memory in tiles: r, k, w padded to 32 KPT channels, then the CTA's value channels.
-// A sum over key channels is one over lanes; those of eight tokens x two columns are reduced at once by halving
-// exchanges, which leave lanes 2 i and 2 i + 1 with token i / 2 and column i % 2.
+// A warp owns kScanCols columns of a head's state (value channels), its lanes KPT key channels each, two at a time in
+// packed arithmetic.  Tokens come through shared memory in tiles: r, k, w padded to 32 KPT channels, then the
+// CTA's value channels.  A sum over key channels is one over lanes; those of several tokens are reduced at once
+// by halving exchanges, which spread tokens and columns over the lanes.
+template <int KPT>
+struct Scan {
+    static constexpr int cols = kScanCols * kScanWarps;     // value channels per CTA
+    static constexpr int rows = 32 * KPT, per = 3 * rows + cols, P = KPT / 2;
+    static constexpr size_t smem(int tile) { return kScanStages * (size_t)tile * per * sizeof(float); }
+    static constexpr int tile = smem(kScanTile) <= 200 * 1024 ? kScanTile : kScanTile / 2;
+    static_assert(tile % kScanGroup == 0 && smem(tile) <= 227 * 1024, "a tile holds whole groups");
+};
+
 template <int KPT>
 __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const Wkv M, const float* proj, int ldp, const float* decay, int pos0, int n,
-                                                                int tile, float* out) {
+                                                                float* out) {
     extern __shared__ __align__(16) float smem[];
-    constexpr int rows = 32 * KPT, per = 3 * rows + kScanWarps * kScanCols, P = KPT / 2, NO = kScanGroup * kScanCols;
-    const int D = M.dim, nh = M.heads * D, h = blockIdx.x, v0 = blockIdx.y * kScanWarps * kScanCols;
+    using G = Scan<KPT>;
+    constexpr int rows = G::rows, per = G::per, P = G::P, tile = G::tile, NO = kScanGroup * kScanCols;
+    const int D = M.dim, nh = M.heads * D, h = blockIdx.x, v0 = blockIdx.y * G::cols;
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, vw = v0 + wid * kScanCols;
-    const int cols = min(kScanWarps * kScanCols, D - v0);
+    const int cols = min(G::cols, D - v0);
     // the padding is zero and stays so
-    for (int i = threadIdx.x; i < 2 * tile * per; i += kScanThreads) smem[i] = 0.f;
+    for (int i = threadIdx.x; i < kScanStages * tile * per; i += kScanThreads) smem[i] = 0.f;
     __syncthreads();
-    const bool wide = ((D | ldp) & 3) == 0;
-    auto load = [&](int buf, int t0) {              // a warp per token
-        const int T = min(tile, n - t0);
-        for (int t = wid; t < T; t += kScanWarps) {
-            float* to = smem + ((size_t)buf * tile + t) * per;
-            const float* row = proj + (size_t)(t0 + t) * ldp + h * D;
-            const float* dw = decay + (size_t)(t0 + t) * nh + h * D;
-            if (wide) {
-                for (int c = lane * 4; c < D; c += 128) {
-                    cp_async16(to + c, row + c);
-                    cp_async16(to + rows + c, row + nh + c);
-                    cp_async16(to + 2 * rows + c, dw + c);
-                }
-            } else {
-                for (int c = lane; c < D; c += 32) {
-                    cp_async4(to + c, row + c);
-                    cp_async4(to + rows + c, row + nh + c);
-                    cp_async4(to + 2 * rows + c, dw + c);
-                }
-            }
-            for (int c = lane; c < cols; c += 32) cp_async4(to + 3 * rows + c, row + 2 * (size_t)nh + v0 + c);
-        }
+    // a thread copies piece `c` of every `step`-th token from `first` on; quads where rows are whole quads
+    const int wide = ((D | ldp) & 3) == 0 ? 4 : 1;
+    auto pieces = [&](int count, int& first, int& c, int& step) {
+        if (count > kScanThreads) count = kScanThreads;             // the rest in further rounds over c
+        step = kScanThreads / count;
+        first = threadIdx.x / count;
+        c = (threadIdx.x - first * count) * wide;
+        if (first >= step) first = tile;
     };
-    load(0, 0);
-    cp_async_commit();
+    int f1, c1, s1, f2, c2, s2;
+    pieces(D / wide, f1, c1, s1);
+    pieces(cols / wide, f2, c2, s2);
+    const float* row0 = proj + h * D;
+    const float* dec0 = decay + h * D;
+    auto load = [&](int i) {
+        const int t0 = i * tile, T = min(tile, n - t0);
+        float* dst = smem + (size_t)(i % kScanStages) * tile * per;
+        auto copy = [&](float* to, const float* from) {
+            if (wide == 4) cp_async16(to, from);
+            else cp_async4(to, from);
+        };
+        for (int t = f1; t < T; t += s1)
+            for (int c = c1; c < D; c += kScanThreads * wide) {
+                const float* row = row0 + (size_t)(t0 + t) * ldp + c;
+                copy(dst + t * per + c, row);
+                copy(dst + t * per + rows + c, row + nh);
+                copy(dst + t * per + 2 * rows + c, dec0 + (size_t)(t0 + t) * nh + c);
+            }
+        for (int t = f2; t < T; t += s2) copy(dst + t * per + 3 * rows + c2, row0 + (size_t)(t0 + t) * ldp + 2 * (size_t)nh + v0 + c2);
+        cp_async_commit();
+    };
+    for (int i = 0; i < kScanStages - 1; i++) load(i);
     unsigned long long S[kScanCols][P], u[P];
 #pragma unroll
     for (int i = 0; i < P; i++) {
@@ -212,55 +243,79 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const Wkv M, con
             S[c][i] = pack2(in && d < D ? s[0] : 0.f, in && d + 1 < D ? s[D] : 0.f);
         }
     }
-    auto token = [&](const float* p, float* o) {
+    struct Token {
         unsigned long long r[P], k[P], w[P];
-        lds_pairs<KPT>(p, lane, r);
-        lds_pairs<KPT>(p + rows, lane, k);
-        lds_pairs<KPT>(p + 2 * rows, lane, w);
-        const float2 v2 = *reinterpret_cast<const float2*>(p + 3 * rows + wid * kScanCols);
-        const unsigned long long v[kScanCols] = {pack2(v2.x, v2.x), pack2(v2.y, v2.y)};
+        float v[kScanCols];
+    };
+    auto fetch = [&](const float* p, Token& x) {
+        lds_pairs<KPT>(p, lane, x.r);
+        lds_pairs<KPT>(p + rows, lane, x.k);
+        lds_pairs<KPT>(p + 2 * rows, lane, x.w);
+        const float* v = p + 3 * rows + wid * kScanCols;
+#pragma unroll
+        for (int c = 0; c < kScanCols; c += 2) {
+            const float2 t = *reinterpret_cast<const float2*>(v + c);
+            x.v[c] = t.x; x.v[c + 1] = t.y;
+        }
+    };
+    auto step = [&](const Token& x, float* o) {
 #pragma unroll
         for (int c = 0; c < kScanCols; c++) {
+            const unsigned long long v = pack2(x.v[c], x.v[c]);
             unsigned long long sum = 0ull;
 #pragma unroll
             for (int i = 0; i < P; i++) {
-                const unsigned long long kv = mul2(k[i], v[c]);
-                sum = fma2(fma2(u[i], kv, S[c][i]), r[i], sum);
-                S[c][i] = fma2(w[i], S[c][i], kv);
+                const unsigned long long kv = mul2(x.k[i], v);
+                const unsigned long long t = fma2(u[i], kv, S[c][i]);
+                sum = i ? fma2(t, x.r[i], sum) : mul2(t, x.r[i]);
+                S[c][i] = fma2(x.w[i], S[c][i], kv);
             }
             o[c] = lo(sum) + hi(sum);
         }
     };
-    int buf = 0;
-    for (int t0 = 0; t0 < n; t0 += tile, buf ^= 1) {
-        if (t0 + tile < n) load(buf ^ 1, t0 + tile);
-        cp_async_commit();
-        cp_async_wait<1>();
+    const int tiles = (n + tile - 1) / tile;
+    for (int it = 0; it < tiles; it++) {
+        const int t0 = it * tile, T = min(tile, n - t0);
+        load(it + kScanStages - 1);
+        cp_async_wait<kScanStages - 1>();
         __syncthreads();
-        const float* base = smem + (size_t)buf * tile * per;
-        const int T = min(tile, n - t0);
+        const float* base = smem + (size_t)(it % kScanStages) * tile * per;
         for (int g = 0; g < T; g += kScanGroup) {
             float o[NO];
             if (g + kScanGroup <= T) {
+                constexpr int AHEAD = KPT == 2 ? 4 : 1;     // tokens held before they are needed
+                Token x[AHEAD];
 #pragma unroll
-                for (int j = 0; j < kScanGroup; j++) token(base + (g + j) * per, o + j * kScanCols);
+                for (int j = 0; j < AHEAD; j++) fetch(base + (g + j) * per, x[j]);
+#pragma unroll
+                for (int j = 0; j < kScanGroup; j++) {
+                    const Token now = x[j % AHEAD];
+                    if (j + AHEAD < kScanGroup) fetch(base + (g + j + AHEAD) * per, x[j % AHEAD]);
+                    step(now, o + j * kScanCols);
+                }
             } else {
 #pragma unroll
                 for (int j = 0; j < kScanGroup; j++)
-                    if (g + j < T) token(base + (g + j) * per, o + j * kScanCols);
+                    if (g + j < T) {
+                        Token x;
+                        fetch(base + (g + j) * per, x);
+                        step(x, o + j * kScanCols);
+                    }
             }
+            constexpr int L = 32 / NO;              // lanes that end with the same sum
 #pragma unroll
             for (int m = NO / 2; m > 0; m >>= 1) {
-                const bool up = (lane & (2 * m)) != 0;
+                const bool up = (lane & (L * m)) != 0;
 #pragma unroll
                 for (int j = 0; j < m; j++) {
                     const float give = up ? o[j] : o[j + m], keep = up ? o[j + m] : o[j];
-                    o[j] = keep + __shfl_xor_sync(MG_FULL_MASK, give, 2 * m);
+                    o[j] = keep + __shfl_xor_sync(MG_FULL_MASK, give, L * m);
                 }
             }
-            o[0] += __shfl_xor_sync(MG_FULL_MASK, o[0], 1);
-            const int t = g + (lane >> 2), v = vw + ((lane >> 1) & 1);
-            if ((lane & 1) == 0 && t < T && v < D) out[(size_t)(t0 + t) * nh + h * D + v] = o[0];
+#pragma unroll
+            for (int m = L / 2; m > 0; m >>= 1) o[0] += __shfl_xor_sync(MG_FULL_MASK, o[0], m);
+            const int t = g + lane / L / kScanCols, v = vw + lane / L % kScanCols;
+            if (lane % L == 0 && t < T && v < D) out[(size_t)(t0 + t) * nh + h * D + v] = o[0];
         }
         __syncthreads();
     }
@@ -278,13 +333,11 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const Wkv M, con
 
 template <int KPT>
 cudaError_t scan_for(const Wkv& wk, const float* proj, int ldp, const float* decay, int pos0, int n, float* out, cudaStream_t s) {
-    constexpr int per = 3 * 32 * KPT + kScanWarps * kScanCols, tile = KPT <= 4 ? 32 : KPT == 8 ? 16 : 8;
-    constexpr size_t smem = 2 * (size_t)tile * per * sizeof(float);
-    static_assert(tile % kScanGroup == 0 && smem <= 227 * 1024, "a tile holds whole groups");
+    using G = Scan<KPT>;
+    constexpr size_t smem = G::smem(G::tile);
     static cudaError_t attr = cudaFuncSetAttribute((const void*)wkv_scan_kernel<KPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (attr != cudaSuccess) return attr;
-    wkv_scan_kernel<KPT><<<dim3(wk.heads, (wk.dim + kScanWarps * kScanCols - 1) / (kScanWarps * kScanCols)), kScanThreads, smem, s>>>(
-        wk, proj, ldp, decay, pos0, n, tile, out);
+    wkv_scan_kernel<KPT><<<dim3(wk.heads, (wk.dim + G::cols - 1) / G::cols), kScanThreads, smem, s>>>(wk, proj, ldp, decay, pos0, n, out);
     return cudaGetLastError();
 }
 
@@ -310,13 +363,17 @@ cudaError_t launch_wkv_mix(const float* h, const float* prev, const float* const
                : mix_for(h, prev, mu, pos0, n, width, (__nv_bfloat16*)act, ld_act, act_stride, s);
 }
 
-bool wkv_rows_fits(const Wkv& wk) { return wk.dim <= 512; }
+cudaError_t launch_wkv_inner(const float* inner, int ldp, int rank, int n, void* act, int ld, cudaStream_t s) {
+    wkv_inner_kernel<<<(n * rank + 255) / 256, 256, 0, s>>>(inner, ldp, rank, n, (__nv_bfloat16*)act, ld);
+    return cudaGetLastError();
+}
+
+bool wkv_rows_fits(const Wkv& wk) { return wk.dim <= 256; }
 
 cudaError_t launch_wkv_rows(const Wkv& wk, const float* proj, int ldp, const float* decay, int pos0, int n, float* out, cudaStream_t s) {
     if (wk.dim <= 64) return scan_for<2>(wk, proj, ldp, decay, pos0, n, out, s);
     if (wk.dim <= 128) return scan_for<4>(wk, proj, ldp, decay, pos0, n, out, s);
     if (wk.dim <= 256) return scan_for<8>(wk, proj, ldp, decay, pos0, n, out, s);
-    if (wk.dim <= 512) return scan_for<16>(wk, proj, ldp, decay, pos0, n, out, s);
     return cudaErrorInvalidValue;
 }
 
