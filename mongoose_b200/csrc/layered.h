@@ -170,8 +170,8 @@ size_t wkv_step_smem(const Wkv& wk);
 // act[j][r] = the mix of row r and the one before it (prev before the first) with mu[j]
 cudaError_t launch_wkv_mix(const float* h, const float* prev, const float* const mu[5], int pos0, int n, int width, void* act, int ld_act,
                            long long act_stride, bool f32, cudaStream_t s);
-// act[n][ld] = tanh of the decay's inner projection as two bf16 parts
-cudaError_t launch_wkv_inner(const float* inner, int ldp, int rank, int n, void* act, int ld, cudaStream_t s);
+// act[n][ld] = tanh of the decay's inner projection (the sum of `slices` slabs [n][ldp]) as two bf16 parts
+cudaError_t launch_wkv_inner(const float* inner, int ldp, int slices, int rank, int n, void* act, int ld, cudaStream_t s);
 bool wkv_rows_fits(const Wkv& wk);
 // proj rows as WkvStep's, decays [n][heads * dim]; out [n][heads * dim] raw outputs
 cudaError_t launch_wkv_rows(const Wkv& wk, const float* proj, int ldp, const float* decay, int pos0, int n, float* out, cudaStream_t s);
@@ -192,6 +192,7 @@ cudaError_t launch_moe_down(const MoeStep& a, int sms, bool pdl, cudaStream_t s)
 struct MoeRows {                // workspace of a portion
     int *sel, *slot;            // [n][top] chosen expert, its row among the grouped rows
     float* weight;              // [n][top]
+    float* shared_gate;         // [n]
     int* count;                 // [experts], zero between calls
     int* first;                 // [experts + 1] first grouped row of an expert
     int* group;                 // [tiles] expert of every 128 grouped rows, -1: none
@@ -200,10 +201,11 @@ struct MoeRows {                // workspace of a portion
     void* y;                    // [tiles * 128][width] grouped outputs, bf16 or fp32
 };
 inline int moe_tiles(const Moe& m, int n) { return (int)(((long long)n * m.top + 127) / 128) + m.experts; }
-// choice, grouping and the grouped inputs
-cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s);
+// choice, grouping, the grouped inputs and the shared expert's gate; the router rows are the sum of `slices` slabs
+// [n][ldr]
+cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int slices, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s);
 // z = weighted sum of the grouped rows (+ z times the shared expert's gate)
-cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, bool f32, cudaStream_t s);
+cudaError_t launch_moe_combine(const Moe& m, int n, const MoeRows& w, float* z, bool f32, cudaStream_t s);
 
 // ---- portions of a prompt (layered_prefill.cu) -----------------------------------------------------
 // `act` buffers hold bf16 or fp32 (f32 = true) rows padded to a multiple of 64 with zeros.

@@ -89,7 +89,7 @@ struct Layered {
     uint8_t *act = nullptr, *qh = nullptr, *ao = nullptr, *my = nullptr, *midr = nullptr, *fin = nullptr;
     uint8_t *aw = nullptr, *vt = nullptr;   // tensor-core attention: mixed weights of a query block, transposed keys or values
     uint8_t* keys = nullptr;            // keys formed from latents
-    float *x0r = nullptr, *hr = nullptr, *q32 = nullptr, *decay = nullptr, *wo = nullptr, *rtr = nullptr, *glu = nullptr;
+    float *x0r = nullptr, *hr = nullptr, *q32 = nullptr, *decay = nullptr, *wo = nullptr, *rtr = nullptr, *glu = nullptr, *inner32 = nullptr;
     uint8_t *cat = nullptr, *mix = nullptr, *inner = nullptr, *cq = nullptr, *xmid = nullptr;
     MoeRows moe{};
     MemRows mw{};
@@ -98,6 +98,8 @@ struct Layered {
 };
 
 namespace {
+
+constexpr int kThinSlices = 8;      // slices of layered_matmul_thin, at most
 
 // Runs `take(pointer, bytes)` over every device buffer of the model, so that sizing the arena and
 // carving it are one list.
@@ -225,8 +227,8 @@ int layered_buffers(Layered& m, F take) {
     get(&m.my, (size_t)T * kmem, as); get(&m.midr, (size_t)T * ff, as); get(&m.fin, (size_t)m.logit_rows * kw, as);
     get(&m.aw, aw, 2); get(&m.vt, vt, 2); get(&m.keys, keys, 2);
     get(&m.q32, q32, 4); get(&m.cq, (size_t)T * cq, as);
-    if (wkv) { get(&m.hr, (size_t)T * W, 4); get(&m.mix, (size_t)5 * T * kw, as); get(&m.decay, (size_t)T * wkv, 4); get(&m.wo, (size_t)T * wkv, 4); get(&m.inner, m.f32 ? 0 : (size_t)T * ld2, 2); }
-    get(&m.rtr, (size_t)T * rtr, 4); get(&m.xmid, xmid, as); get(&m.glu, m.f32 ? xmid : 0, 4);
+    if (wkv) { get(&m.hr, (size_t)T * W, 4); get(&m.mix, (size_t)5 * T * kw, as); get(&m.decay, (size_t)T * wkv, 4); get(&m.wo, (size_t)T * wkv, 4); get(&m.inner, m.f32 ? 0 : (size_t)T * ld2, 2); get(&m.inner32, (size_t)kThinSlices * T * (ld2 / 2), 4); }
+    get(&m.rtr, (size_t)kThinSlices * T * rtr, 4); get(&m.moe.shared_gate, rtr ? T : 0, 4); get(&m.xmid, xmid, as); get(&m.glu, m.f32 ? xmid : 0, 4);
     get(&m.moe.sel, (size_t)T * top, 4); get(&m.moe.slot, (size_t)T * top, 4); get(&m.moe.weight, (size_t)T * top, 4);
     get(&m.moe.count, experts, 4); get(&m.moe.first, experts ? experts + 1 : 0, 4); get(&m.moe.group, tiles, 4);
     get(&m.moe.x, moe * kw, as); get(&m.moe.y, moe * W, as);
@@ -786,6 +788,26 @@ int layered_matmul_batch(mg_engine* e, const void* act, long long stride, int ac
     return MG_OK;
 }
 
+// The same for few columns, which too few CTAs would share: the columns of act are cut into slices whose products
+// land in out[slice][n][ldc], for the reader to add in order.  Returns the number of slices in *slices.
+int layered_matmul_thin(mg_engine* e, const void* act, int act_rows, int ld, const uint8_t* w, float* out, int ldc, int n, int rows, int* slices) {
+    Layered& m = *e->lm;
+    int S = m.f32 || rows > 64 ? 1 : kThinSlices;
+    while (ld / 64 % S) S /= 2;
+    *slices = S;
+    if (S == 1) return layered_matmul(e, act, act_rows, ld, w, out, ldc, n, rows, false);
+    e->launches += 1;
+    const int k = ld / S;
+    GemmTC g{};
+    g.bn = 64;
+    if (!make_tile_map(&g.a, act, k, act_rows, S, ld, k, 128) || !make_tile_map(&g.b, w, k, rows, S, ld, k, g.bn))
+        return fail(e, MG_ERR_CUDA, "tensor map of a %d x %d product in %d slices failed", rows, ld, S);
+    g.m = n; g.n = rows; g.k = k; g.batch = S; g.b_group = 1; g.causal_pos0 = -1;
+    g.out = out; g.ldc = ldc; g.batch_c = (long long)n * ldc; g.mode = GEMM_F32; g.status = m.status;
+    MG_CUDA(e, launch_gemm_tc(g, e->stream));
+    return MG_OK;
+}
+
 // One gated feed-forward, or with `group` those of stacked experts, each tile of 128 rows its own: z = down(silu(gate
 // act) * (up act)), fp32 or like activations.  ld, ffs: padded row lengths; `count` matrices are stacked.
 int layered_glu(mg_engine* e, const void* act, int act_rows, int ld, const uint8_t* gate, const uint8_t* up, const uint8_t* down, int ff, int ffs,
@@ -881,16 +903,18 @@ int wkv_rows(mg_engine* e, const LayerRun& run, LayerWeights& l, int pos, int n)
     MG_CUDA(e, launch_wkv_mix(m.hr, run.prev, l.mu, pos, n, W, m.mix, kw, stride, m.f32, s));
     MG_CUDA(e, cudaMemcpyAsync(run.prev + (size_t)((pos + n) & 1) * W, m.hr + (size_t)(n - 1) * W, (size_t)W * 4, cudaMemcpyDeviceToDevice, s));
     if ((rc = layered_matmul_batch(e, m.mix, stride, m.max_rows, kw, l.proj, m.P, np, n, d, 4))) return rc;
-    if ((rc = layered_matmul(e, m.mix + 4 * stride * (m.f32 ? 4 : 2), m.max_rows, kw, l.proj + (size_t)4 * d * kw * 2, m.P + (size_t)4 * d, np, n, wk.rank, false))) return rc;
+    int slices;
+    const int ldi = pad_to(wk.rank, 4);
+    if ((rc = layered_matmul_thin(e, m.mix + 4 * stride * (m.f32 ? 4 : 2), m.max_rows, kw, l.proj + (size_t)4 * d * kw * 2, m.inner32, ldi, n, wk.rank, &slices))) return rc;
     // decays: the inner vector stays 32-bit, on the tensor cores as a high and a low part
     if (m.f32) {
         GemmF32 g{};
-        g.A = m.P + (size_t)4 * d; g.lda = np; g.W = l.w2; g.ldw = wk.ld2; g.out = m.decay; g.ldc = d; g.n = n; g.rows = d; g.K = wk.rank;
+        g.A = m.inner32; g.lda = ldi; g.W = l.w2; g.ldw = wk.ld2; g.out = m.decay; g.ldc = d; g.n = n; g.rows = d; g.K = wk.rank;
         g.epi = F32_DECAY; g.bias = l.w0;
         MG_CUDA(e, launch_gemm_f32(g, s));
     } else {
         const int ld = 2 * wk.ld2;
-        MG_CUDA(e, launch_wkv_inner(m.P + (size_t)4 * d, np, wk.rank, n, m.inner, ld, s));
+        MG_CUDA(e, launch_wkv_inner(m.inner32, ldi, slices, wk.rank, n, m.inner, ld, s));
         GemmTC g{};
         g.bn = d > 64 ? 128 : 64;
         if (!make_tile_map(&g.a, m.inner, ld, m.max_rows, 1, ld, (long long)m.max_rows * ld, 128) ||
@@ -916,12 +940,13 @@ int moe_rows(mg_engine* e, LayerWeights& l, int n) {
     w.tiles = moe_tiles(x, n);
     cudaStream_t s = e->stream;
     int rc;
-    if ((rc = layered_matmul(e, m.act, m.max_rows, m.kw, l.router, m.rtr, ldr, n, cols, false))) return rc;
-    MG_CUDA(e, launch_moe_route(x, m.rtr, ldr, n, m.act, m.f32, w, s));
+    int slices;
+    if ((rc = layered_matmul_thin(e, m.act, m.max_rows, m.kw, l.router, m.rtr, ldr, n, cols, &slices))) return rc;
+    MG_CUDA(e, launch_moe_route(x, m.rtr, ldr, slices, n, m.act, m.f32, w, s));
     if ((rc = layered_glu(e, w.x, w.tiles * 128, m.kw, l.e_gate, l.e_up, l.e_down, x.ff, x.ffs, x.experts, w.group, w.y, true, w.tiles * 128))) return rc;
     if (x.shared_ff && (rc = layered_glu(e, m.act, m.max_rows, m.kw, l.router_row(x.sg_col() + 1), l.router_row(x.sg_col() + 1 + x.shared_ff),
                                          l.shared_down, x.shared_ff, x.shared_ffs, 1, nullptr, m.zr, false, n))) return rc;
-    MG_CUDA(e, launch_moe_combine(x, m.rtr, ldr, n, w, m.zr, m.f32, s));
+    MG_CUDA(e, launch_moe_combine(x, n, w, m.zr, m.f32, s));
     e->launches += 4;
     return MG_OK;
 }

@@ -181,14 +181,19 @@ __global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeStep a) {
 // ---- prompts ----
 
 // A warp per token: choice, and the token's place among those of its expert.
-__global__ void __launch_bounds__(kThreads) moe_choose_kernel(const Moe m, const float* router, int ldr, int n, MoeRows w) {
+__global__ void __launch_bounds__(kThreads) moe_choose_kernel(const Moe m, const float* router, int ldr, int slices, int n, MoeRows w) {
     extern __shared__ __align__(16) float smem[];
     __shared__ int sel[kThreads / 32][kMaxTop];
     __shared__ float wt[kThreads / 32][kMaxTop];
     const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * (kThreads / 32) + wid;
     if (t >= n) return;
     float* z = smem + wid * m.experts;
-    for (int i = lane; i < m.experts; i += 32) z[i] = router[(size_t)t * ldr + i] + m.bias[i];
+    for (int i = lane; i < m.experts + (m.shared_ff ? 1 : 0); i += 32) {
+        float v = 0.f;
+        for (int s = 0; s < slices; s++) v += router[((size_t)s * n + t) * ldr + i];
+        if (i < m.experts) z[i] = v + m.bias[i];
+        else w.shared_gate[t] = sigmoid(v);
+    }
     __syncwarp();
     choose(z, m.experts, m.top, sel[wid], wt[wid], lane);
     for (int k = lane; k < m.top; k += 32) {
@@ -232,7 +237,7 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const Moe m, const uint
 }
 
 template <typename AT, int V>
-__global__ void __launch_bounds__(kThreads) moe_combine_kernel(const Moe m, const float* router, int ldr, MoeRows w, float* z) {
+__global__ void __launch_bounds__(kThreads) moe_combine_kernel(const Moe m, MoeRows w, float* z) {
     __shared__ float wt[kMaxTop];
     __shared__ int row[kMaxTop];
     const size_t t = blockIdx.x;
@@ -242,7 +247,7 @@ __global__ void __launch_bounds__(kThreads) moe_combine_kernel(const Moe m, cons
     }
     __syncthreads();
     const AT* y = static_cast<const AT*>(w.y);
-    const float sg = m.shared_ff ? sigmoid(router[t * ldr + m.sg_col()]) : 0.f;
+    const float sg = m.shared_ff ? w.shared_gate[t] : 0.f;
     float* out = z + t * m.width;
     for (int i = threadIdx.x * V; i < m.width; i += kThreads * V) {
         float v[V] = {};
@@ -286,19 +291,19 @@ cudaError_t launch_moe_down(const MoeStep& a, int sms, bool pdl, cudaStream_t s)
     return launch_pdl(moe_down_kernel<kDownRows>, grid, kThreads, smem, pdl, s, a);
 }
 
-cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s) {
-    moe_choose_kernel<<<(n + 7) / 8, kThreads, (size_t)8 * m.experts * sizeof(float), s>>>(m, router, ldr, n, w);
+cudaError_t launch_moe_route(const Moe& m, const float* router, int ldr, int slices, int n, const void* act, bool f32, const MoeRows& w, cudaStream_t s) {
+    moe_choose_kernel<<<(n + 7) / 8, kThreads, (size_t)8 * m.experts * sizeof(float), s>>>(m, router, ldr, slices, n, w);
     moe_plan_kernel<<<1, 1024, 0, s>>>(m, w);
     moe_gather_kernel<<<n, 128, 0, s>>>(m, (const uint4*)act, m.ldw * (f32 ? 4 : 2) / 16, w);
     return cudaGetLastError();
 }
 
-cudaError_t launch_moe_combine(const Moe& m, const float* router, int ldr, int n, const MoeRows& w, float* z, bool f32, cudaStream_t s) {
+cudaError_t launch_moe_combine(const Moe& m, int n, const MoeRows& w, float* z, bool f32, cudaStream_t s) {
     const bool quads = m.width % 4 == 0;
-    if (f32 && quads) moe_combine_kernel<float, 4><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
-    else if (f32) moe_combine_kernel<float, 1><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
-    else if (quads) moe_combine_kernel<__nv_bfloat16, 4><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
-    else moe_combine_kernel<__nv_bfloat16, 1><<<n, kThreads, 0, s>>>(m, router, ldr, w, z);
+    if (f32 && quads) moe_combine_kernel<float, 4><<<n, kThreads, 0, s>>>(m, w, z);
+    else if (f32) moe_combine_kernel<float, 1><<<n, kThreads, 0, s>>>(m, w, z);
+    else if (quads) moe_combine_kernel<__nv_bfloat16, 4><<<n, kThreads, 0, s>>>(m, w, z);
+    else moe_combine_kernel<__nv_bfloat16, 1><<<n, kThreads, 0, s>>>(m, w, z);
     return cudaGetLastError();
 }
 

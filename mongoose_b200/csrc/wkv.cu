@@ -139,12 +139,14 @@ __global__ void __launch_bounds__(256) wkv_mix_kernel(const float* h, const floa
     }
 }
 
-// act[t] = [high, low]: tanh of the decay's inner projection as two bf16 parts (16 bits of mantissa together), each padded
-// to ld / 2, so that a product of bf16 operands keeps it.
-__global__ void __launch_bounds__(256) wkv_inner_kernel(const float* inner, int ldp, int rank, int n, __nv_bfloat16* act, int ld) {
+// act[t] = [high, low]: tanh of the decay's inner projection, the sum of `slices` slabs, as two bf16 parts (16 bits of
+// mantissa together), each padded to ld / 2, so that a product of bf16 operands keeps it.
+__global__ void __launch_bounds__(256) wkv_inner_kernel(const float* inner, int ldp, int slices, int rank, int n, __nv_bfloat16* act, int ld) {
     const int i = blockIdx.x * 256 + threadIdx.x, t = i / rank, c = i - t * rank;
     if (t >= n) return;
-    const float v = tanhf(inner[(size_t)t * ldp + c]);
+    float v = 0.f;
+    for (int s = 0; s < slices; s++) v += inner[((size_t)s * n + t) * ldp + c];
+    v = tanhf(v);
     const __nv_bfloat16 high = __float2bfloat16_rn(v);
     act[(size_t)t * ld + c] = high;
     act[(size_t)t * ld + ld / 2 + c] = __float2bfloat16_rn(v - __bfloat162float(high));
@@ -363,8 +365,8 @@ cudaError_t launch_wkv_mix(const float* h, const float* prev, const float* const
                : mix_for(h, prev, mu, pos0, n, width, (__nv_bfloat16*)act, ld_act, act_stride, s);
 }
 
-cudaError_t launch_wkv_inner(const float* inner, int ldp, int rank, int n, void* act, int ld, cudaStream_t s) {
-    wkv_inner_kernel<<<(n * rank + 255) / 256, 256, 0, s>>>(inner, ldp, rank, n, (__nv_bfloat16*)act, ld);
+cudaError_t launch_wkv_inner(const float* inner, int ldp, int slices, int rank, int n, void* act, int ld, cudaStream_t s) {
+    wkv_inner_kernel<<<(n * rank + 255) / 256, 256, 0, s>>>(inner, ldp, slices, rank, n, (__nv_bfloat16*)act, ld);
     return cudaGetLastError();
 }
 
